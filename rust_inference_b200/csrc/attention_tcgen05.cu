@@ -23,12 +23,12 @@
 // softmax computes its exponentials before it waits for P V of the page before (it needs that only
 // to overwrite P and to rescale O).  Two CTAs fit on an SM (96 KiB of shared memory, 256 TMEM columns).
 //
-// Two further forms of the score and the mask (template FORMS; the plain kernel is compiled without them and is what it
+// Further forms of the score, the mask and the denominator (template FORMS; the plain kernel is compiled without them and is what it
 // was): capped scores, s <- cap * tanh(s * scale / cap), formed by the softmax thread in the base-2 domain before the
 // maximum is taken (tanh(x) = 1 - 2 / (1 + 2^(2 x log2 e)), the hardware's exponential and division, relative error far
 // below the bf16 rounding of P); and, with a window, the sequence's first `keep_first` positions kept visible: the page
 // walk then starts with the pages before the window that hold kept positions, and the mask lets keys below keep_first
-// pass.
+// pass; a sink, one more term exp(sink_h) in the row's sum, added where the row is divided by it.
 //
 // All mbarrier waits are bounded; on a timeout the kernel records a code in the host-visible
 // status word and winds down.
@@ -97,7 +97,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
                        const int* __restrict__ seq_slot, const int* __restrict__ seq_start,
                        const int* __restrict__ cu_seqlens, int n_heads, int n_kv_heads, float scale_log2, int window,
                        float out_scale, __nv_bfloat16* __restrict__ out, int out_ld, uint32_t smem_bytes, int* status,
-                       float cap_log2, float scale_over_cap, int keep_first) {
+                       float cap_log2, float scale_over_cap, int keep_first, const float* __restrict__ sink) {
     constexpr int ATOMS = HD / 64;                       // 64-wide (128-byte) column tiles per row of head_dim
     constexpr int Q_BYTES = ATOMS * BM * 128;            // [atom][128 queries][64]
     constexpr int K_BYTES = ATOMS * BN * 128;            // one buffer: [atom][64 keys][64]
@@ -368,7 +368,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
         tc_fence_after();
         if (ok && !abort_flag) {
             wait_for_previous_kernels();          // `out` must not be written while an earlier kernel may read it
-            const float inv = out_scale / l;
+            // FORMS: a sink joins the row's sum as one more term exp(sink_h) without a value (2^x may overflow to infinity when
+            // the sink outweighs every score: the result is then 0, as it should be)
+            const float inv = out_scale / ((FORMS && sink != nullptr) ? l + fast_exp2(fmaf(sink[h], 1.4426950408889634f, -m_used)) : l);
             __nv_bfloat16* dst = out + (size_t)(tok0 + q0 + r) * out_ld + (size_t)h * HD;
 #pragma unroll 1
             for (int c = 0; c < HD; c += 16) {
@@ -404,7 +406,7 @@ template <int HD, bool FORMS>
 int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const int* page_table, int max_pages,
            const int* seq_slot, const int* seq_start, const int* cu_seqlens, int n_seqs, int max_new, int n_heads,
            int n_kv_heads, float scale, int window, float out_scale, void* out, int out_ld, int* status, cudaStream_t stream,
-           float softcap = 0.f, int keep_first = 0) {
+           float softcap = 0.f, int keep_first = 0, const float* sink = nullptr) {
     constexpr int ATOMS = HD / 64;
     // Q, two K and two V pages, P, the barriers; with head_dim 128 no room for alignment padding is left if
     // two CTAs are to share an SM (the kernel refuses, with a status code, a shared window that needs any)
@@ -420,7 +422,7 @@ int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, 
     cudaError_t e = launch_dependent(kernel, grid, dim3(THREADS), (size_t)SMEM, stream, mq, mk, mv, page_table, max_pages,
                                      seq_slot, seq_start, cu_seqlens, n_heads, n_kv_heads, scale_log2, window,
                                      out_scale, (__nv_bfloat16*)out, out_ld, (uint32_t)SMEM, status,
-                                     softcap * 1.4426950408889634f, softcap > 0.f ? scale / softcap : 0.f, keep_first);
+                                     softcap * 1.4426950408889634f, softcap > 0.f ? scale / softcap : 0.f, keep_first, sink);
     return check_launch(e, "attention_tcgen05");
 }
 
@@ -466,12 +468,13 @@ RI_API int ri_attention_tcgen05_prefill(const void* map_q, const void* map_k, co
 }
 
 // The same with capped scores (softcap > 0: s <- softcap tanh(s scale / softcap)) and, with a window (> 0 only: the last
-// so many keys), the sequence's first keep_first positions kept visible beyond it.
+// so many keys), the sequence's first keep_first positions kept visible beyond it; sink (float32 [n_heads] or null): one
+// more term exp(sink_h) in the denominator of head h's softmax.
 RI_API int ri_attention_tcgen05_prefill_forms(const void* map_q, const void* map_k, const void* map_v, const int* page_table,
                                               int max_pages, const int* seq_slot, const int* seq_start,
                                               const int* cu_seqlens, void* out, int out_ld, int n_seqs, int max_new,
                                               int n_heads, int n_kv_heads, int hd, int page_size, float scale, int window,
-                                              float out_scale, float softcap, int keep_first, int* status,
+                                              float out_scale, float softcap, int keep_first, const float* sink, int* status,
                                               cudaStream_t stream) {
     if (n_seqs <= 0 || max_new <= 0) return 0;
     if (!ri_attention_tcgen05_supports(hd, page_size, n_heads, n_kv_heads, 8, out_ld))
@@ -486,9 +489,9 @@ RI_API int ri_attention_tcgen05_prefill_forms(const void* map_q, const void* map
     const CUtensorMap& mv = *reinterpret_cast<const CUtensorMap*>(map_v);
     if (hd == 64)
         return launch<64, true>(mq, mk, mv, page_table, max_pages, seq_slot, seq_start, cu_seqlens, n_seqs, max_new, n_heads,
-                                n_kv_heads, scale, window, out_scale, out, out_ld, status, stream, softcap, keep_first);
+                                n_kv_heads, scale, window, out_scale, out, out_ld, status, stream, softcap, keep_first, sink);
     return launch<128, true>(mq, mk, mv, page_table, max_pages, seq_slot, seq_start, cu_seqlens, n_seqs, max_new, n_heads,
-                             n_kv_heads, scale, window, out_scale, out, out_ld, status, stream, softcap, keep_first);
+                             n_kv_heads, scale, window, out_scale, out, out_ld, status, stream, softcap, keep_first, sink);
 }
 
 RI_DEFINE_LAST_ERROR()

@@ -117,29 +117,35 @@ __device__ __forceinline__ GateForm load_gate_form(const float* p) {
     return f;
 }
 
-// A learned activation of one argument (epilogue 4 of the contractions, and a kernel of its own):
-//   act(z) = a_p z^2 + z / 2 for z > 0,   a_n (e^z - 1 - z) + z / 2 otherwise,   a_p = softplus(p),  a_n = 1/2 + softplus(q),
-// p and q two floats in device memory.  Continuous at 0 with slope 1/2 on both sides; expm1f keeps e^z - 1 for small z.
-struct ActForm { float ap, an; };
-__device__ __forceinline__ ActForm load_act_form(const float* pq) {
-    const float p = pq[0], q = pq[1];
+// An activation of one argument (epilogue 4 of the contractions, and a kernel of its own):
+//   act(z) = a_p z^2 + l z for z > 0,   a_n (e^z - 1 - z) + l z otherwise.
+// Four floats {p, q, l, fixed} in device memory.  fixed = 0: a learned form, a_p = softplus(p), a_n = 1/2 + softplus(q)
+// (with l = 1/2 continuous at 0 with slope 1/2 on both sides; expm1f keeps e^z - 1 for small z).  fixed = 1: a_p = p and
+// a_n = q as they are; {1, 0, 0, 1} is the square of relu.
+struct ActForm { float ap, an, lin; };
+__device__ __forceinline__ ActForm load_act_form(const float* form) {
+    const float p = form[0], q = form[1];
+    const bool fixed = form[3] != 0.f;
     ActForm f;
-    f.ap = p > 20.f ? p : log1pf(expf(p));
-    f.an = 0.5f + (q > 20.f ? q : log1pf(expf(q)));
+    f.ap = fixed ? p : (p > 20.f ? p : log1pf(expf(p)));
+    f.an = fixed ? q : 0.5f + (q > 20.f ? q : log1pf(expf(q)));
+    f.lin = form[2];
     return f;
 }
 __device__ __forceinline__ float act_f32(float z, const ActForm& f) {
-    return z > 0.f ? fmaf(f.ap * z, z, 0.5f * z) : fmaf(f.an, expm1f(z) - z, 0.5f * z);
+    if (z > 0.f) return fmaf(f.ap * z, z, f.lin * z);
+    return f.an == 0.f ? f.lin * z : fmaf(f.an, expm1f(z) - z, f.lin * z);
 }
 
 // The same for a result that is rounded to bfloat16 right away: e^z - 1 - z from five terms of its series above -1/4
 // (relative error below 2e-5 there) and from the hardware's base-2 exponential below (4e-6), instead of expm1f, whose
 // instructions would outlast the tensor cores' part of a tile.
 __device__ __forceinline__ float act_quick_f32(float z, const ActForm& f) {
-    if (z > 0.f) return fmaf(f.ap * z, z, 0.5f * z);
+    if (z > 0.f) return fmaf(f.ap * z, z, f.lin * z);
+    if (f.an == 0.f) return f.lin * z;
     const float series = z * z * fmaf(z, fmaf(z, fmaf(z, 1.f / 120.f, 1.f / 24.f), 1.f / 6.f), 0.5f);
     const float t = z > -0.25f ? series : __expf(z) - 1.f - z;
-    return fmaf(f.an, t, 0.5f * z);
+    return fmaf(f.an, t, f.lin * z);
 }
 
 // The reference's SiLU, stable on both sides (math.rs:137-146).

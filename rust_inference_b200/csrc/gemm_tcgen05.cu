@@ -31,8 +31,9 @@
 //                                                      fed by the same X tile.  This epilogue takes no bias: its
 //                                                      `bias` argument, when not null, points to the three
 //                                                      constants of another gate form (`GateForm`, common.cuh)
-//   4  out<bf16> = act(acc)                           a learned activation of one argument (`ActForm`, common.cuh);
-//                                                      `bias` points to its two constants
+//   4  out<bf16> = act(acc)                           an activation of one argument (`ActForm`, common.cuh);
+//                                                      `bias` points to its four constants
+//   5  out<f32>  = silu(acc) for the first C features, acc for the rest: C is the float `bias` points to
 //
 // Every wait on an mbarrier is bounded.  A wait that runs out stores a code in the
 // host-visible status word, the CTA stops issuing work, waits (bounded) for its own
@@ -67,6 +68,8 @@ __host__ __device__ constexpr uint32_t make_idesc(int tn) {
 // x e^x / (1 + e^x) (math.rs:137-146); the fast exponential and division are exact to a few ulp of
 // float32, far below bf16's 8 bits.
 __device__ __forceinline__ float silu_to_bf16(float x) { return __fdividef(x, 1.f + __expf(-x)); }
+// The same kept in float32 (relative error near 1e-6).
+__device__ __forceinline__ float silu_quick(float x) { return __fdividef(x, 1.f + __expf(-x)); }
 // The gated epilogue in its general form (`GateForm`), with the same fast exponential and division.
 __device__ __forceinline__ float gated_to_bf16(float g, float u, const GateForm& f) {
     g = fminf(g, f.limit);
@@ -77,7 +80,9 @@ __device__ __forceinline__ float gated_to_bf16(float g, float u, const GateForm&
 template <int MODE>
 __device__ __forceinline__ void store_result(void* out_, size_t o, float acc, float bias, float acc2, const GateForm& gf,
                                              const ActForm& af) {
-    if (MODE == 4) {
+    if (MODE == 5) {
+        reinterpret_cast<float*>(out_)[o] = bias != 0.f ? silu_quick(acc) : acc;      // `bias`: whether the feature is one of the first C
+    } else if (MODE == 4) {
         reinterpret_cast<__nv_bfloat16*>(out_)[o] = __float2bfloat16_rn(act_quick_f32(acc, af));
     } else if (MODE == 0) {
         reinterpret_cast<__nv_bfloat16*>(out_)[o] = __float2bfloat16_rn(acc + bias);
@@ -291,9 +296,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
             if (!landed || abort_flag) break;
             const int f = f0 + lane_base + lane;
             const bool f_ok = f < n_feat;
-            const float b = (MODE != 3 && MODE != 4 && bias != nullptr && f_ok) ? bias[f] : 0.f;
+            const float b = MODE == 5 ? (f < (int)bias[0] ? 1.f : 0.f)
+                                      : (MODE != 3 && MODE != 4 && bias != nullptr && f_ok) ? bias[f] : 0.f;
             const GateForm gf = load_gate_form(MODE == 3 ? bias : nullptr);
-            const ActForm af = MODE == 4 ? load_act_form(bias) : ActForm{0.f, 0.f};
+            const ActForm af = MODE == 4 ? load_act_form(bias) : ActForm{0.f, 0.f, 0.f};
             const uint32_t trow = tmem_base + ((uint32_t)lane_base << 16) + (uint32_t)(buf * ACC_COLS);
 #pragma unroll 1
             for (int c0 = 0; c0 < tn; c0 += 16) {
@@ -361,7 +367,8 @@ __device__ __forceinline__ void tm_write_tile(uint32_t trow, int t, bool t_ok, i
                                               bool pieces = false) {     // MODE 2: other work items add to the same tile
     constexpr int FEATS = DUAL ? TM_ROWS / 2 : TM_ROWS;
     const GateForm gf = load_gate_form(MODE == 3 ? bias : nullptr);     // the gated epilogue's constants come in `bias`
-    const ActForm af = MODE == 4 ? load_act_form(bias) : ActForm{0.f, 0.f};     // so do the activation's
+    const ActForm af = MODE == 4 ? load_act_form(bias) : ActForm{0.f, 0.f, 0.f};     // so do the activation's
+    const int silu_feats = MODE == 5 ? (int)bias[0] : 0;
 #pragma unroll 1
     for (int c0 = 0; c0 < FEATS; c0 += 16) {
         if (f0 + c0 >= n_feat) break;                       // uniform over the warp
@@ -379,6 +386,7 @@ __device__ __forceinline__ void tm_write_tile(uint32_t trow, int t, bool t_ok, i
             if (MODE == 3) r[j] = gated_to_bf16(a, __uint_as_float(u[j]), gf);
             else if (MODE == 4) r[j] = act_quick_f32(a, af);
             else if (MODE == 2) r[j] = a;
+            else if (MODE == 5) r[j] = f0 + c0 + j < silu_feats ? silu_quick(a) : a;
             else r[j] = a + ((bias != nullptr && f0 + c0 + j < n_feat) ? bias[f0 + c0 + j] : 0.f);
         }
         if (whole) {
@@ -412,7 +420,7 @@ __device__ __forceinline__ void tm_write_tile(uint32_t trow, int t, bool t_ok, i
             for (int j = 0; j < 16; ++j)
                 if (f0 + c0 + j < n_feat) {
                     if (MODE == 0 || MODE == 3 || MODE == 4) reinterpret_cast<__nv_bfloat16*>(out_)[o0 + j] = __float2bfloat16_rn(r[j]);
-                    else if (MODE == 1) reinterpret_cast<float*>(out_)[o0 + j] = r[j];
+                    else if (MODE == 1 || MODE == 5) reinterpret_cast<float*>(out_)[o0 + j] = r[j];
                     else if (pieces) atomicAdd(reinterpret_cast<float*>(out_) + o0 + j, r[j]);
                     else reinterpret_cast<float*>(out_)[o0 + j] += r[j];
                 }
@@ -1087,8 +1095,9 @@ RI_API int ri_gemm_tcgen05(const void* map_x, const void* map_w, const void* map
                            int mode, int n_tok, int n_feat, int K, int split_k, int* status, cudaStream_t stream) {
     if (n_tok <= 0 || n_feat <= 0) return 0;
     if (K <= 0 || K % 8) return fail("gemm_tcgen05: K = %d must be a positive multiple of 8 (16-byte rows for TMA)", K);
-    if (mode < 0 || mode > 4) return fail("gemm_tcgen05: unknown epilogue mode %d", mode);
-    if (mode == 4 && bias == nullptr) return fail("gemm_tcgen05: the activation epilogue needs its two constants");
+    if (mode < 0 || mode > 5) return fail("gemm_tcgen05: unknown epilogue mode %d", mode);
+    if (mode == 4 && bias == nullptr) return fail("gemm_tcgen05: the activation epilogue needs its constants");
+    if (mode == 5 && bias == nullptr) return fail("gemm_tcgen05: the partly activated epilogue needs its number of features");
     if (mode == 3 && map_w2 == nullptr) return fail("gemm_tcgen05: the SiLU-gate epilogue needs a second matrix");
     if (mode == 2 && bias != nullptr) return fail("gemm_tcgen05: the residual epilogue takes no bias");
     if (mode != 2 && split_k > 1) return fail("gemm_tcgen05: only the residual epilogue can split K");
@@ -1107,6 +1116,7 @@ RI_API int ri_gemm_tcgen05(const void* map_x, const void* map_w, const void* map
             case 1: return launch_pair<false, 1>(mw, mw2, mx, bias, out, n_tok, n_feat, K, 1, status, stream);
             case 2: return launch_pair<false, 2>(mw, mw2, mx, bias, out, n_tok, n_feat, K, split_k, status, stream);
             case 4: return launch_pair<false, 4>(mw, mw2, mx, bias, out, n_tok, n_feat, K, 1, status, stream);
+            case 5: return launch_pair<false, 5>(mw, mw2, mx, bias, out, n_tok, n_feat, K, 1, status, stream);
             default: return launch_pair<true, 3>(mw, mw2, mx, bias, out, n_tok, n_feat, K, 1, status, stream);
         }
     }
@@ -1116,6 +1126,7 @@ RI_API int ri_gemm_tcgen05(const void* map_x, const void* map_w, const void* map
         case 1: return pick_tile<false, 1>(tn, mw, mw2, mx, bias, out, n_tok, n_feat, K, split_k, status, stream);
         case 2: return pick_tile<false, 2>(tn, mw, mw2, mx, bias, out, n_tok, n_feat, K, split_k, status, stream);
         case 4: return pick_tile<false, 4>(tn, mw, mw2, mx, bias, out, n_tok, n_feat, K, split_k, status, stream);
+        case 5: return pick_tile<false, 5>(tn, mw, mw2, mx, bias, out, n_tok, n_feat, K, split_k, status, stream);
         default: return pick_tile<true, 3>(tn, mw, mw2, mx, bias, out, n_tok, n_feat, K, split_k, status, stream);
     }
 }

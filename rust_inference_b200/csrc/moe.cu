@@ -7,7 +7,8 @@
 //             ranking, whatever the sign of their c); the `top` candidates with the highest c are
 //             taken, with weights s / (sum of the taken s + 1e-20).
 //             Optionally one more number per token: sigmoid(w_gate . h), the gate of a shared expert.
-//             Another form (`form` bit 0): s = softmax(W_router h) over all experts instead of the sigmoid; and
+//             Other forms: (`form` bit 0) s = softmax(W_router h) over all experts instead of the sigmoid; (bit 2) a
+//             group ranks by its largest c alone; no correction (a null pointer: c = s); and
 //             (bit 1) the weights are the taken s as they are, not divided by their sum.
 //   arrange   the (token, choice) pairs listed expert by expert, cut into tiles of rows that belong
 //             to one expert
@@ -96,7 +97,7 @@ moe_route_kernel(const T* x, const float* __restrict__ router, const float* __re
         const float s = sigmoid_f32(a);
         if (e < experts) {
             smem[k * stride + e] = (form & 1) ? a : s;           // softmax: the logit, turned into a score below
-            smem[k * stride + experts + e] = s + correction[e];
+            smem[k * stride + experts + e] = correction != nullptr ? s + correction[e] : s;
         } else {
             gate_out[tok0 + k] = s;
         }
@@ -163,12 +164,12 @@ moe_route_kernel(const T* x, const float* __restrict__ router, const float* __re
         for (int e = lane; e < experts; e += 32) {
             const float s = expf(score[e] - mx) / sum;
             score[e] = s;
-            choice[e] = s + correction[e];
+            choice[e] = correction != nullptr ? s + correction[e] : s;
         }
         __syncwarp();
     }
 
-    // groups: top-2 sum of c per group; all but the `keep` highest leave the ranking
+    // groups: top-2 sum of c (or its maximum) per group; all but the `keep` highest leave the ranking
     const int size = experts / groups;
     if (keep < groups) {
         for (int g = lane; g < groups; g += 32) {
@@ -177,7 +178,7 @@ moe_route_kernel(const T* x, const float* __restrict__ router, const float* __re
                 const float c = choice[g * size + k];
                 if (c > a) { b = a; a = c; } else if (c > b) { b = c; }
             }
-            gscore[g] = size > 1 ? a + b : a;
+            gscore[g] = size > 1 && !(form & 4) ? a + b : a;
         }
         __syncwarp();
         // `keep` rounds of taking the best remaining group; a taken group is marked with +inf
@@ -401,7 +402,8 @@ __global__ void moe_combine_kernel(float* residual, const float* y, const float*
 
 }  // namespace
 
-// form: bit 0 softmax scores instead of sigmoid ones, bit 1 weights not divided by their sum.
+// form: bit 0 softmax scores instead of sigmoid ones, bit 1 weights not divided by their sum, bit 2 a group counts by its
+// largest score instead of the sum of its two largest.  correction may be null.
 // split > 1 (steps of up to ROUTE_SPLIT_TOKENS tokens): the router's rows are cut over that many blocks per token;
 // split_sums: float32 [n_tokens, experts + 1] scratch, split_count: int32 [n_tokens], zero before the call and after it.
 RI_API int ri_moe_route(const void* x, int dtype, const float* router, const float* correction, const float* gate_w,

@@ -5,6 +5,10 @@
 //     state space    S <- a S + k (s v)^T                      o = S^T q + skip * v
 //     delta rule     S <- a S;  u = s (v - S^T k);  S <- S + k u^T      o = S^T q
 //
+// The delta rule also comes with a decay per key channel, S <- diag(a) S with a in [0, 1]^dim, which a low-rank map of the
+// layer's input gives; the state space's form also with a decay per head that never changes and s = 1 (linear attention
+// with a fixed decay).
+//
 // (state space: k = B, q = C, v = x, s = dt, a = exp(-exp(A_log) dt);  delta rule: s = beta, a = exp(-exp(A_log)
 // softplus(.)); the read-out sees the token's own write.)  Heads share keys and queries in groups.  The state lives in
 // a per-slot area of the cache, starts at zero when a slot is handed out and is carried from step to step; so do the
@@ -14,11 +18,13 @@
 // Four kernels, all reading the step's arrays on the device (graph-safe), everything float32:
 //   prepare     per token: the short convolution (+ bias) and silu over a range of the projection's columns; unit
 //               vectors x / sqrt(sum x^2 + 1e-6) for the first heads of that range (the first of them times a factor);
-//               the decay and the step of every head
+//               the decay and the step of every head; decays per key channel from their low-rank input (steps of few
+//               tokens, which also get a low-rank gate here) or from products formed before.  In a step of one token
+//               per sequence it moves the carried inputs on as well
 //   conv_state  per (sequence, channel): the convolution's carried inputs move on by the step's tokens
 //   scan        per (sequence, head, tile of value columns): the recurrence over the sequence's new tokens in
 //               order; the state is read first and written last
-//   finish      per (token, group of channels): RMS norm over the group and a silu gate, before or after the norm
+//   finish      per (token, group of channels): RMS norm over the group and a silu or sigmoid gate, before or after the norm
 //
 // What an earlier kernel of the step wrote is read after `wait_for_previous_kernels()` through plain pointers.
 #include "common.cuh"
@@ -56,7 +62,43 @@ struct Prepare {
     const int* token_seq;
     const int* seq_slot;
     int tile_ch;               // convolved channels per block: a multiple of unit_dim where there are unit vectors
+    int conv_tiles;            // tiles of convolved channels (blockIdx.y); further tiles hold CHANNEL_TILE low-rank channels each
+    int single;                // 1: every sequence brings one token, and the carried inputs move on here
+    // decays per key channel, exp(-exp(a_log[head]) softplus(raw + dt_bias[channel])): channels 0: one decay per head
+    int channels, head_dim;
+    const float* raw;          // [tokens, channels] the low-rank map's result (may be `decay`), or null: formed here
+    float* decay;              // [tokens, channels]
+    const void* w2;            // [channels, rank], in the run dtype
+    int rank, low_col;         // the low-rank input's columns of z
+    // the low-rank gate, formed here as well (gate_channels 0: not): gate_out = gate_w2 . z[gate_low_col ..]
+    int gate_channels, gate_rank, gate_low_col;
+    const void* gate_w2;
+    float* gate_out;           // [tokens, gate_channels]
+    int w2_bf16;
 };
+
+constexpr int CHANNEL_TILE = 256;
+
+// A row of a low-rank map (rank values in the run dtype) times the input in shared memory.
+template <typename T>
+__device__ __forceinline__ float low_rank_dot(const T* __restrict__ w, const float* a, int rank) {
+    float acc0 = 0.f, acc1 = 0.f;
+    constexpr int V = 16 / sizeof(T);
+    if (rank % V == 0) {
+        for (int r = 0; r < rank; r += V) {
+            const uint4 pk = *reinterpret_cast<const uint4*>(w + r);
+            const T* e = reinterpret_cast<const T*>(&pk);
+#pragma unroll
+            for (int k = 0; k < V; k += 2) {
+                acc0 = fmaf(to_f32<T>(e[k]), a[r + k], acc0);
+                acc1 = fmaf(to_f32<T>(e[k + 1]), a[r + k + 1], acc1);
+            }
+        }
+    } else {
+        for (int r = 0; r < rank; ++r) acc0 = fmaf(to_f32<T>(w[r]), a[r], acc0);
+    }
+    return acc0 + acc1;
+}
 
 // A block per (token, tile of p.tile_ch convolved channels); tiles hold whole heads of the unit vectors.  The first
 // tile's block also writes the heads' decays and steps.
@@ -66,12 +108,38 @@ __global__ void __launch_bounds__(256) scan_prepare_kernel(Prepare p) {
     const int c0 = blockIdx.y * p.tile_ch, c1 = min(p.conv_ch, c0 + p.tile_ch);
     let_next_kernel_start();
     wait_for_previous_kernels();
+    if ((int)blockIdx.y >= p.conv_tiles) {
+        // low-rank channels: the decays', then the gate's; a tile holds channels of one of the two
+        const int tiles = (p.channels + CHANNEL_TILE - 1) / CHANNEL_TILE;
+        const int tile = (int)blockIdx.y - p.conv_tiles;
+        const bool gate = tile >= tiles;
+        const int c = (gate ? tile - tiles : tile) * CHANNEL_TILE + (int)threadIdx.x;
+        const bool formed = gate || p.raw == nullptr;
+        const int rank = gate ? p.gate_rank : p.rank;
+        if (formed) {
+            const float* low = p.z + (size_t)t * p.ld + (gate ? p.gate_low_col : p.low_col);
+            for (int r = threadIdx.x; r < rank; r += blockDim.x) ch[r] = low[r];
+            __syncthreads();
+        }
+        if (c >= (gate ? p.gate_channels : p.channels)) return;
+        float v;
+        if (formed) {
+            const void* w = gate ? p.gate_w2 : p.w2;
+            v = p.w2_bf16 ? low_rank_dot(reinterpret_cast<const __nv_bfloat16*>(w) + (size_t)c * rank, ch, rank)
+                          : low_rank_dot(reinterpret_cast<const float*>(w) + (size_t)c * rank, ch, rank);
+        } else {
+            v = p.raw[(size_t)t * p.channels + c];
+        }
+        if (gate) p.gate_out[(size_t)t * p.gate_channels + c] = v;
+        else p.decay[(size_t)t * p.channels + c] = expf(-expf(p.a_log[c / p.head_dim]) * softplus_f32(v + p.dt_bias[c]));
+        return;
+    }
     const int b = p.token_seq[t];
     const int i = t - p.cu_seqlens[b];            // place among the sequence's new tokens
     int slot = p.seq_slot[b];
     if (!RI_BLOCK_IN_LIMIT(slot, RI_LIMIT_SLOTS, RI_CHECK_SLOT)) slot = 0;
     const int K = p.k_taps;
-    const float* carried = p.conv_state + (size_t)slot * (K - 1) * p.conv_ch;
+    float* carried = p.conv_state + (size_t)slot * (K - 1) * p.conv_ch;
     for (int c = c0 + threadIdx.x; c < c1; c += blockDim.x) {
         float acc = p.conv_bias != nullptr ? p.conv_bias[c] : 0.f;
         for (int k = 0; k < K; ++k) {             // the input k tokens back
@@ -81,6 +149,10 @@ __global__ void __launch_bounds__(256) scan_prepare_kernel(Prepare p) {
             acc = fmaf(p.taps[(size_t)c * K + (K - 1 - k)], x, acc);
         }
         ch[c - c0] = silu_f32(acc);
+        if (p.single && K > 1) {                  // the channel's inputs move on by this one token; only this thread has read them
+            for (int s = 0; s < K - 2; ++s) carried[(size_t)s * p.conv_ch + c] = carried[(size_t)(s + 1) * p.conv_ch + c];
+            carried[(size_t)(K - 2) * p.conv_ch + c] = p.z[(size_t)t * p.ld + p.conv_col + c];
+        }
     }
     __syncthreads();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
@@ -100,8 +172,11 @@ __global__ void __launch_bounds__(256) scan_prepare_kernel(Prepare p) {
     for (int c = c0 + threadIdx.x; c < c1; c += blockDim.x) out[c] = ch[c - c0];
     if (blockIdx.y == 0)
         for (int h = threadIdx.x; h < p.heads; h += blockDim.x) {
-            const float dt = softplus_f32(p.z[(size_t)t * p.ld + p.decay_col + h] + p.dt_bias[h]);
-            out[p.conv_ch + h] = expf(-expf(p.a_log[h]) * dt);
+            float dt = 0.f;
+            if (p.channels == 0) {
+                dt = softplus_f32(p.z[(size_t)t * p.ld + p.decay_col + h] + p.dt_bias[h]);
+                out[p.conv_ch + h] = expf(-expf(p.a_log[h]) * dt);
+            }
             out[p.conv_ch + p.heads + h] = p.step_col >= 0 ? sigmoid_f32(p.z[(size_t)t * p.ld + p.step_col + h]) : dt;
         }
 }
@@ -149,6 +224,7 @@ struct Scan {
     const float* u;            // [tokens, ld]: the prepared rows
     int ld;
     int q_col, k_col, v_col, decay_col, step_col;
+    const float* decay;        // CHANNELS: [tokens, heads * dim], a decay per key channel; FIXED: [heads], decays that never change
     const float* skip;         // [heads] or null: o += skip * v
     float* state;              // [slots, heads, dim, vdim]
     float* o;                  // [tokens, heads * vdim]
@@ -169,10 +245,15 @@ struct Scan {
 // slot; FINAL scans every piece again from its start state and writes the read-outs.
 enum { WHOLE = 0, LOCAL = 1, FINAL = 2 };
 
-template <int ROWS, bool DELTA, int MODE>
+// Where the decays come from: PER_TOKEN a column per head beside the steps; CHANNELS (the delta rule) a row per token and
+// head with a value per key channel; FIXED (not the delta rule) one number per head for all tokens, with step 1.
+enum { PER_TOKEN = 0, CHANNELS = 1, FIXED = 2 };
+
+template <int ROWS, bool DELTA, int MODE, int DECAY>
 __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(Scan p) {
     constexpr int SLICE = ROWS + 4;
-    constexpr int TOKEN = 2 * R * SLICE + COLS + 4;       // k, q, the block's values, decay and step
+    constexpr int V_AT = (DECAY == CHANNELS ? 3 : 2) * R * SLICE;     // k, q (, decays), then the block's values, decay and step
+    constexpr int TOKEN = V_AT + COLS + 4;
     extern __shared__ __align__(16) float tile[];          // two tiles of tile_t tokens
     const int b = MODE == WHOLE ? blockIdx.x : blockIdx.x / p.max_pieces, h = blockIdx.y, j0 = blockIdx.z * COLS;
     const int pc = MODE == WHOLE ? 0 : blockIdx.x % p.max_pieces;
@@ -193,6 +274,7 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(Scan p) {
 #pragma unroll
     for (int k = 0; k < ROWS; ++k) s[k] = (MODE != LOCAL && live && i0 + k < p.dim) ? S[(size_t)(i0 + k) * p.vdim + j] : 0.f;
     float decays = 1.f;
+    const float fixed = DECAY == FIXED ? p.decay[h] : 1.f;
     const int g = h / (p.heads / p.groups);
     const int q_off = p.q_col + g * p.dim, k_off = p.k_col + g * p.dim, v_off = p.v_col + h * p.vdim + j0;
     const int cols = min(COLS, p.vdim - j0);
@@ -202,33 +284,39 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(Scan p) {
     // the copies of the tokens tb .. tb + n_tok - 1 into one of the two tiles; every thread commits one group
     auto fetch = [&](float* dst, int tb, int n_tok) {
         if (p.vec) {
-            const int dq = p.dim >> 2, cq = cols >> 2, per = 2 * dq + cq;
+            const int dq = p.dim >> 2, cq = cols >> 2, parts = DECAY == CHANNELS ? 3 : 2, per = parts * dq + cq;
             for (int tok = 0; tok < n_tok; ++tok) {
                 const float* row = p.u + (size_t)(tb + tok) * p.ld;
                 float* base = dst + tok * TOKEN;
                 for (int it = threadIdx.x; it < per; it += SCAN_THREADS) {
                     if (it < dq) copy_async16(base + (4 * it / ROWS) * SLICE + 4 * it % ROWS, row + k_off + 4 * it);
                     else if (it < 2 * dq) copy_async16(base + R * SLICE + (4 * (it - dq) / ROWS) * SLICE + 4 * (it - dq) % ROWS, row + q_off + 4 * (it - dq));
-                    else copy_async16(base + 2 * R * SLICE + 4 * (it - 2 * dq), row + v_off + 4 * (it - 2 * dq));
+                    else if (DECAY == CHANNELS && it < 3 * dq) copy_async16(base + 2 * R * SLICE + (4 * (it - 2 * dq) / ROWS) * SLICE + 4 * (it - 2 * dq) % ROWS, p.decay + ((size_t)(tb + tok) * p.heads + h) * p.dim + 4 * (it - 2 * dq));
+                    else copy_async16(base + V_AT + 4 * (it - parts * dq), row + v_off + 4 * (it - parts * dq));
                 }
             }
         } else {
-            const int per = 2 * p.dim + cols;
+            const int parts = DECAY == CHANNELS ? 3 : 2, per = parts * p.dim + cols;
             for (int tok = 0; tok < n_tok; ++tok) {
                 const float* row = p.u + (size_t)(tb + tok) * p.ld;
                 float* base = dst + tok * TOKEN;
                 for (int it = threadIdx.x; it < per; it += SCAN_THREADS) {
                     if (it < p.dim) copy_async4(base + (it / ROWS) * SLICE + it % ROWS, row + k_off + it);
                     else if (it < 2 * p.dim) copy_async4(base + R * SLICE + ((it - p.dim) / ROWS) * SLICE + (it - p.dim) % ROWS, row + q_off + it - p.dim);
-                    else copy_async4(base + 2 * R * SLICE + it - 2 * p.dim, row + v_off + it - 2 * p.dim);
+                    else if (DECAY == CHANNELS && it < 3 * p.dim) copy_async4(base + 2 * R * SLICE + ((it - 2 * p.dim) / ROWS) * SLICE + (it - 2 * p.dim) % ROWS, p.decay + ((size_t)(tb + tok) * p.heads + h) * p.dim + it - 2 * p.dim);
+                    else copy_async4(base + V_AT + it - parts * p.dim, row + v_off + it - parts * p.dim);
                 }
             }
         }
-        for (int tok = threadIdx.x; tok < 2 * n_tok; tok += SCAN_THREADS) {      // decay and step of every token
-            const int tk = tok >> 1, which = tok & 1;
-            copy_async4(dst + tk * TOKEN + 2 * R * SLICE + COLS + which,
-                        p.u + (size_t)(tb + tk) * p.ld + (which ? p.step_col : p.decay_col) + h);
-        }
+        if (DECAY == PER_TOKEN)
+            for (int tok = threadIdx.x; tok < 2 * n_tok; tok += SCAN_THREADS) {      // decay and step of every token
+                const int tk = tok >> 1, which = tok & 1;
+                copy_async4(dst + tk * TOKEN + V_AT + COLS + which,
+                            p.u + (size_t)(tb + tk) * p.ld + (which ? p.step_col : p.decay_col) + h);
+            }
+        if (DECAY == CHANNELS)
+            for (int tk = threadIdx.x; tk < n_tok; tk += SCAN_THREADS)
+                copy_async4(dst + tk * TOKEN + V_AT + COLS + 1, p.u + (size_t)(tb + tk) * p.ld + p.step_col + h);
         copy_async_commit();
     };
 
@@ -253,8 +341,9 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(Scan p) {
             const float* base = cur + tok * TOKEN;
             const float4* k4 = reinterpret_cast<const float4*>(base + r * SLICE);
             const float4* q4 = reinterpret_cast<const float4*>(base + R * SLICE + r * SLICE);
-            const float v = base[2 * R * SLICE + jj];
-            const float a = base[2 * R * SLICE + COLS], step = base[2 * R * SLICE + COLS + 1];
+            const float v = base[V_AT + jj];
+            const float a = DECAY == FIXED ? fixed : DECAY == CHANNELS ? 1.f : base[V_AT + COLS];
+            const float step = DECAY == FIXED ? 1.f : base[V_AT + COLS + 1];
             float kk[ROWS], qq[ROWS];
 #pragma unroll
             for (int k = 0; k < ROWS / 4; ++k) {
@@ -266,10 +355,20 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(Scan p) {
             if (MODE == LOCAL) decays *= a;
             if (DELTA) {
                 float d0 = 0.f, d1 = 0.f;
+                if (DECAY == CHANNELS) {
+                    const float4* a4 = reinterpret_cast<const float4*>(base + 2 * R * SLICE + r * SLICE);
+#pragma unroll
+                    for (int k = 0; k < ROWS / 4; ++k) {
+                        const float4 av = a4[k];
+                        s[4 * k] *= av.x; s[4 * k + 1] *= av.y; s[4 * k + 2] *= av.z; s[4 * k + 3] *= av.w;
+                    }
+                }
 #pragma unroll
                 for (int k = 0; k < ROWS; k += 2) {
-                    s[k] *= a;
-                    s[k + 1] *= a;
+                    if (DECAY != CHANNELS) {
+                        s[k] *= a;
+                        s[k + 1] *= a;
+                    }
                     d0 = fmaf(s[k], kk[k], d0);
                     d1 = fmaf(s[k + 1], kk[k + 1], d1);
                 }
@@ -324,12 +423,14 @@ __global__ void __launch_bounds__(256) scan_carry_kernel(float* state, float* pi
     *dst = s;
 }
 
+__device__ __forceinline__ float gate_f32(float x, int sigmoid) { return sigmoid ? sigmoid_f32(x) : silu_f32(x); }
+
 // One warp per (token, group of `gs` channels): with gate_first the channels are multiplied by silu(gate) and then
-// normalised, otherwise normalised and then multiplied; the weight of channel c of a token's row is w[c % w_len].
+// normalised, otherwise normalised and then multiplied (sigmoid != 0: by sigmoid(gate)); the weight of channel c of a token's row is w[c % w_len].
 template <typename T>
 __global__ void gated_group_norm_kernel(const float* x, int x_ld, const float* gate, int gate_ld, int gate_col,
                                         const float* __restrict__ w, int w_len, T* __restrict__ out, int n_tokens, int groups,
-                                        int gs, int gate_first, float eps, float out_scale) {
+                                        int gs, int gate_first, int sigmoid, float eps, float out_scale) {
     let_next_kernel_start();
     wait_for_previous_kernels();
     const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
@@ -339,14 +440,14 @@ __global__ void gated_group_norm_kernel(const float* x, int x_ld, const float* g
     const float* gt = gate + (size_t)t * gate_ld + gate_col + g * gs;
     float ss = 0.f;
     for (int d = lane; d < gs; d += 32) {
-        const float v = gate_first ? src[d] * silu_f32(gt[d]) : src[d];
+        const float v = gate_first ? src[d] * gate_f32(gt[d], sigmoid) : src[d];
         ss = fmaf(v, v, ss);
     }
     ss = warp_sum(ss);
     const float inv = out_scale / sqrtf(ss / (float)gs + eps);
     T* dst = out + ((size_t)t * groups + g) * gs;
     for (int d = lane; d < gs; d += 32) {
-        const float sg = silu_f32(gt[d]);
+        const float sg = gate_f32(gt[d], sigmoid);
         const float v = gate_first ? src[d] * sg : src[d];
         const float y = v * inv * w[(g * gs + d) % w_len];
         dst[d] = from_f32<T>(gate_first ? y : y * sg);
@@ -357,7 +458,7 @@ __global__ void gated_group_norm_kernel(const float* x, int x_ld, const float* g
 template <typename T>
 __global__ void __launch_bounds__(256) gated_group_norm_block_kernel(const float* x, int x_ld, const float* gate, int gate_ld, int gate_col,
                                         const float* __restrict__ w, int w_len, T* __restrict__ out, int groups,
-                                        int gs, int gate_first, float eps, float out_scale) {
+                                        int gs, int gate_first, int sigmoid, float eps, float out_scale) {
     __shared__ float scratch[33];
     let_next_kernel_start();
     wait_for_previous_kernels();
@@ -366,14 +467,14 @@ __global__ void __launch_bounds__(256) gated_group_norm_block_kernel(const float
     const float* gt = gate + (size_t)t * gate_ld + gate_col + g * gs;
     float ss = 0.f;
     for (int d = threadIdx.x; d < gs; d += blockDim.x) {
-        const float v = gate_first ? src[d] * silu_f32(gt[d]) : src[d];
+        const float v = gate_first ? src[d] * gate_f32(gt[d], sigmoid) : src[d];
         ss = fmaf(v, v, ss);
     }
     ss = block_sum(ss, scratch);
     const float inv = out_scale / sqrtf(ss / (float)gs + eps);
     T* dst = out + ((size_t)t * groups + g) * gs;
     for (int d = threadIdx.x; d < gs; d += blockDim.x) {
-        const float sg = silu_f32(gt[d]);
+        const float sg = gate_f32(gt[d], sigmoid);
         const float v = gate_first ? src[d] * sg : src[d];
         const float y = v * inv * w[(g * gs + d) % w_len];
         dst[d] = from_f32<T>(gate_first ? y : y * sg);
@@ -382,9 +483,9 @@ __global__ void __launch_bounds__(256) gated_group_norm_block_kernel(const float
 
 constexpr int SCAN_SMEM_LIMIT = 44 * 1024;
 
-template <int ROWS>
-int launch_scan(bool delta, dim3 grid, cudaStream_t stream, Scan p, int longest, int n_seqs) {
-    const int token_bytes = (2 * R * (ROWS + 4) + COLS + 4) * (int)sizeof(float);
+template <int ROWS, bool DELTA, int DECAY>
+int launch_scan(dim3 grid, cudaStream_t stream, Scan p, int longest, int n_seqs) {
+    const int token_bytes = ((DECAY == CHANNELS ? 3 : 2) * R * (ROWS + 4) + COLS + 4) * (int)sizeof(float);
     int tile_t = SCAN_SMEM_LIMIT / (2 * token_bytes);     // two tiles
     if (tile_t > 16) tile_t = 16;
     if (longest > 0 && tile_t > longest) tile_t = longest;
@@ -392,33 +493,53 @@ int launch_scan(bool delta, dim3 grid, cudaStream_t stream, Scan p, int longest,
     p.tile_t = tile_t;
     const size_t smem = (size_t)2 * tile_t * token_bytes;
     cudaError_t e;
-    if (delta) {
-        e = launch_dependent(state_scan_kernel<ROWS, true, WHOLE>, grid, SCAN_THREADS, smem, stream, p);
-    } else if (p.piece <= 0) {
-        e = launch_dependent(state_scan_kernel<ROWS, false, WHOLE>, grid, SCAN_THREADS, smem, stream, p);
-    } else {
-        const dim3 pieces(grid.x * p.max_pieces, grid.y, grid.z);
-        e = launch_dependent(state_scan_kernel<ROWS, false, LOCAL>, pieces, SCAN_THREADS, smem, stream, p);
-        if (check_launch(e, "state_scan (pieces from zero)")) return 1;
-        const int per_head = p.dim * p.vdim;
-        e = launch_dependent(scan_carry_kernel, dim3((per_head + 255) / 256, p.heads, n_seqs), 256, 0, stream, p.state, p.piece_state,
-                             (const float*)p.piece_decay, p.cu_seqlens, p.seq_slot, p.heads, per_head, p.piece, p.max_pieces);
-        if (check_launch(e, "state_scan (carry)")) return 1;
-        e = launch_dependent(state_scan_kernel<ROWS, false, FINAL>, pieces, SCAN_THREADS, smem, stream, p);
+    if constexpr (!DELTA) {
+        if (p.piece > 0) {
+            const dim3 pieces(grid.x * p.max_pieces, grid.y, grid.z);
+            e = launch_dependent(state_scan_kernel<ROWS, false, LOCAL, DECAY>, pieces, SCAN_THREADS, smem, stream, p);
+            if (check_launch(e, "state_scan (pieces from zero)")) return 1;
+            const int per_head = p.dim * p.vdim;
+            e = launch_dependent(scan_carry_kernel, dim3((per_head + 255) / 256, p.heads, n_seqs), 256, 0, stream, p.state, p.piece_state,
+                                 (const float*)p.piece_decay, p.cu_seqlens, p.seq_slot, p.heads, per_head, p.piece, p.max_pieces);
+            if (check_launch(e, "state_scan (carry)")) return 1;
+            e = launch_dependent(state_scan_kernel<ROWS, false, FINAL, DECAY>, pieces, SCAN_THREADS, smem, stream, p);
+            return check_launch(e, "state_scan");
+        }
     }
+    e = launch_dependent(state_scan_kernel<ROWS, DELTA, WHOLE, DECAY>, grid, SCAN_THREADS, smem, stream, p);
     return check_launch(e, "state_scan");
+}
+
+template <int ROWS>
+int pick_scan(bool delta, int decay, dim3 grid, cudaStream_t stream, Scan p, int longest, int n_seqs) {
+    if (delta) return decay == CHANNELS ? launch_scan<ROWS, true, CHANNELS>(grid, stream, p, longest, n_seqs)
+                                        : launch_scan<ROWS, true, PER_TOKEN>(grid, stream, p, longest, n_seqs);
+    return decay == FIXED ? launch_scan<ROWS, false, FIXED>(grid, stream, p, longest, n_seqs)
+                          : launch_scan<ROWS, false, PER_TOKEN>(grid, stream, p, longest, n_seqs);
 }
 
 }  // namespace
 
-RI_API int ri_scan_prepare(const float* z, int ld, int conv_col, int conv_ch, const float* taps, const float* conv_bias,
-                           int k_taps, float* conv_state, int unit_heads, int unit_dim, int scaled_heads, float unit_scale,
-                           int heads, int decay_col, int step_col, const float* a_log, const float* dt_bias, float* out,
-                           int out_ld, const int* cu_seqlens, const int* token_seq, const int* seq_slot, int n_tokens,
-                           int n_seqs, cudaStream_t stream) {
+// A step's decays per key channel and its low-rank gate: see `Prepare`.  channels 0: none of it.
+struct LowRank {
+    int channels, head_dim;
+    const float* raw;
+    float* decay;
+    const void* w2;
+    int rank, low_col, gate_channels, gate_rank, gate_low_col;
+    const void* gate_w2;
+    float* gate_out;
+    int w2_bf16;
+};
+
+static int scan_prepare(const float* z, int ld, int conv_col, int conv_ch, const float* taps, const float* conv_bias, int k_taps,
+                        float* conv_state, int unit_heads, int unit_dim, int scaled_heads, float unit_scale, int heads,
+                        int decay_col, int step_col, const float* a_log, const float* dt_bias, float* out, int out_ld,
+                        const int* cu_seqlens, const int* token_seq, const int* seq_slot, int n_tokens, int n_seqs,
+                        int longest_run, const LowRank& low, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (k_taps < 1 || conv_ch < 1) return fail("scan_prepare: a convolution of %d taps over %d channels", k_taps, conv_ch);
-    if (conv_col < 0 || conv_col + conv_ch > ld || decay_col + heads > ld || step_col + heads > ld)
+    if (conv_col < 0 || conv_col + conv_ch > ld || decay_col + (low.channels ? 0 : heads) > ld || step_col + heads > ld)
         return fail("scan_prepare: columns beyond the projection's %d", ld);
     if (unit_heads * unit_dim > conv_ch || scaled_heads > unit_heads) return fail("scan_prepare: unit vectors beyond the convolved channels");
     if (out_ld < conv_ch + 2 * heads) return fail("scan_prepare: output rows of %d values are too short", out_ld);
@@ -427,18 +548,26 @@ RI_API int ri_scan_prepare(const float* z, int ld, int conv_col, int conv_ch, co
     int tile_ch = 512;
     if (unit_heads > 0 && unit_dim > 0) tile_ch = unit_dim * ((512 + unit_dim - 1) / unit_dim);
     if (tile_ch > conv_ch) tile_ch = conv_ch;
-    const size_t smem = (size_t)tile_ch * sizeof(float);
+    int shared_floats = tile_ch;
+    const bool formed = low.channels > 0 && low.raw == nullptr;
+    if (formed && low.rank > shared_floats) shared_floats = low.rank;
+    if (low.gate_channels > 0 && low.gate_rank > shared_floats) shared_floats = low.gate_rank;
+    const size_t smem = (size_t)shared_floats * sizeof(float);
     if (smem > 200 * 1024) return fail("scan_prepare: heads of %d channels do not fit shared memory", unit_dim);
     static PerDeviceOnce once;
     if (smem > 48 * 1024)
         if (int rc = raise_dynamic_smem(scan_prepare_kernel, 200 * 1024, once, "scan_prepare")) return rc;
-    const int tiles = (conv_ch + tile_ch - 1) / tile_ch;
+    const int conv_tiles = (conv_ch + tile_ch - 1) / tile_ch;
+    const int tiles = conv_tiles + (low.channels + CHANNEL_TILE - 1) / CHANNEL_TILE + (low.gate_channels + CHANNEL_TILE - 1) / CHANNEL_TILE;
     if (tiles > 65535) return fail("scan_prepare: %d tiles of channels exceed the grid limit", tiles);
+    const int single = longest_run == 1 ? 1 : 0;
     Prepare p{z, ld, conv_col, conv_ch, taps, conv_bias, k_taps, conv_state, unit_heads, unit_dim, scaled_heads, unit_scale,
-              heads, decay_col, step_col, a_log, dt_bias, out, out_ld, cu_seqlens, token_seq, seq_slot, tile_ch};
+              heads, decay_col, step_col, a_log, dt_bias, out, out_ld, cu_seqlens, token_seq, seq_slot, tile_ch, conv_tiles, single,
+              low.channels, low.head_dim, low.raw, low.decay, low.w2, low.rank, low.low_col, low.gate_channels, low.gate_rank,
+              low.gate_low_col, low.gate_w2, low.gate_out, low.w2_bf16};
     cudaError_t e = launch_dependent(scan_prepare_kernel, dim3(n_tokens, tiles), 256, smem, stream, p);
     if (check_launch(e, "scan_prepare")) return 1;
-    if (k_taps > 1) {
+    if (k_taps > 1 && !single) {
         dim3 grid((conv_ch + 127) / 128, n_seqs);
         e = launch_dependent(conv_state_kernel, grid, 128, 0, stream, z, ld, conv_col, conv_ch, k_taps, conv_state, cu_seqlens, seq_slot);
         if (check_launch(e, "scan_prepare (carried inputs)")) return 1;
@@ -446,41 +575,122 @@ RI_API int ri_scan_prepare(const float* z, int ld, int conv_col, int conv_ch, co
     return 0;
 }
 
+// longest_run: the most new tokens any sequence brings (0: unknown); in a step of one token per sequence the carried inputs
+// move on in the same kernel.
+RI_API int ri_scan_prepare(const float* z, int ld, int conv_col, int conv_ch, const float* taps, const float* conv_bias,
+                           int k_taps, float* conv_state, int unit_heads, int unit_dim, int scaled_heads, float unit_scale,
+                           int heads, int decay_col, int step_col, const float* a_log, const float* dt_bias, float* out,
+                           int out_ld, const int* cu_seqlens, const int* token_seq, const int* seq_slot, int n_tokens,
+                           int n_seqs, int longest_run, cudaStream_t stream) {
+    return scan_prepare(z, ld, conv_col, conv_ch, taps, conv_bias, k_taps, conv_state, unit_heads, unit_dim, scaled_heads, unit_scale,
+                        heads, decay_col, step_col, a_log, dt_bias, out, out_ld, cu_seqlens, token_seq, seq_slot, n_tokens, n_seqs,
+                        longest_run, LowRank{}, stream);
+}
+
+// The same with a decay per key channel, decay[t, c] = exp(-exp(a_log[c / head_dim]) softplus(x[t, c] + dt_bias[c])) for
+// heads * head_dim channels.  x: `raw` (float32 [n_tokens, channels], may be `decay`), or with raw null w2 . z[t, low_col ..]
+// formed here (w2 [channels, rank] in `w2_dtype`, rows on 16-byte boundaries where rank allows).  gate_channels > 0:
+// gate_out[t, c] = gate_w2 . z[t, gate_low_col ..] as well.
+RI_API int ri_scan_prepare_channels(const float* z, int ld, int conv_col, int conv_ch, const float* taps, const float* conv_bias,
+                                    int k_taps, float* conv_state, int unit_heads, int unit_dim, int scaled_heads,
+                                    float unit_scale, int heads, int step_col, const float* a_log, const float* dt_bias,
+                                    float* out, int out_ld, const int* cu_seqlens, const int* token_seq, const int* seq_slot,
+                                    int n_tokens, int n_seqs, int longest_run, int head_dim, const float* raw, float* decay,
+                                    const void* w2, int rank, int low_col, int gate_channels, int gate_rank, int gate_low_col,
+                                    const void* gate_w2, float* gate_out, int w2_dtype, cudaStream_t stream) {
+    if (heads < 1 || head_dim < 1 || decay == nullptr) return fail("scan_prepare: decays of %d heads of %d channels", heads, head_dim);
+    if (raw == nullptr && (w2 == nullptr || rank < 1 || low_col < 0 || low_col + rank > ld || (uintptr_t)w2 % 16))
+        return fail("scan_prepare: a low-rank map of rank %d at column %d of %d", rank, low_col, ld);
+    if (gate_channels > 0 && (gate_w2 == nullptr || gate_out == nullptr || gate_rank < 1 || gate_low_col < 0 ||
+                              gate_low_col + gate_rank > ld || (uintptr_t)gate_w2 % 16))
+        return fail("scan_prepare: a low-rank gate of rank %d at column %d of %d", gate_rank, gate_low_col, ld);
+    if (w2_dtype != RI_F32 && w2_dtype != RI_BF16) return fail("scan_prepare: unknown dtype %d", w2_dtype);
+    const LowRank low{heads * head_dim, head_dim, raw, decay, w2, rank, low_col, gate_channels, gate_rank, gate_low_col, gate_w2,
+                      gate_out, w2_dtype == RI_BF16 ? 1 : 0};
+    return scan_prepare(z, ld, conv_col, conv_ch, taps, conv_bias, k_taps, conv_state, unit_heads, unit_dim, scaled_heads, unit_scale,
+                        heads, 0, step_col, a_log, dt_bias, out, out_ld, cu_seqlens, token_seq, seq_slot, n_tokens, n_seqs,
+                        longest_run, low, stream);
+}
+
+// `rank` columns of z at low_col as a matrix of their own for a product with the low-rank map.  bfloat16: out [n_tokens, 2 *
+// padded]: the value rounded and, in the second half, the rounding of the remainder (the map's matrix stands there twice
+// side by side, so the product keeps 16 significant bits of the input); float32: out [n_tokens, padded].  Columns from rank
+// to padded are zero.
+namespace {
+template <typename T>
+__global__ void low_rank_rows_kernel(const float* z, int ld, int low_col, int rank, int padded, T* __restrict__ out, int n_tokens) {
+    let_next_kernel_start();
+    wait_for_previous_kernels();
+    const int total = n_tokens * padded;
+    for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < total; i += gridDim.x * blockDim.x) {
+        const int t = i / padded, r = i % padded;
+        const float v = r < rank ? z[(size_t)t * ld + low_col + r] : 0.f;
+        if constexpr (sizeof(T) == 4) {
+            out[i] = v;
+        } else {
+            const T hi = from_f32<T>(v);
+            out[(size_t)t * 2 * padded + r] = hi;
+            out[(size_t)t * 2 * padded + padded + r] = from_f32<T>(v - to_f32<T>(hi));
+        }
+    }
+}
+}  // namespace
+
+RI_API int ri_low_rank_rows(const float* z, int ld, int low_col, int rank, int padded, void* out, int dtype, int n_tokens,
+                            cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    if (rank < 1 || padded < rank || low_col < 0 || low_col + rank > ld || (long long)n_tokens * padded > 0x7fffffffLL)
+        return fail("low_rank_rows: %d (%d) columns at %d of %d", rank, padded, low_col, ld);
+    const int blocks = (int)(((long long)n_tokens * padded + 255) / 256 < 1184 ? ((long long)n_tokens * padded + 255) / 256 : 1184);
+    cudaError_t e;
+    if (dtype == RI_F32)
+        e = launch_dependent(low_rank_rows_kernel<float>, blocks, 256, 0, stream, z, ld, low_col, rank, padded, (float*)out, n_tokens);
+    else if (dtype == RI_BF16)
+        e = launch_dependent(low_rank_rows_kernel<__nv_bfloat16>, blocks, 256, 0, stream, z, ld, low_col, rank, padded, (__nv_bfloat16*)out, n_tokens);
+    else
+        return fail("low_rank_rows: unknown dtype %d", dtype);
+    return check_launch(e, "low_rank_rows");
+}
+
 // u: float32 [n_tokens, ld] with the columns of queries and keys ([groups, dim] each), values ([heads, vdim]), decays and
 // steps ([heads] each).  state: float32 [slots, heads, dim, vdim].  o: float32 [n_tokens, heads * vdim].
 // delta != 0: the gated delta rule; else the state space (with skip [heads] or null).  longest_run: the most new tokens
 // any sequence brings (0: unknown), which sizes the scan's shared memory.  piece > 0 (state space only): the three passes
 // over pieces of that many tokens, with scratch piece_state [n_seqs, max_pieces, heads, dim, vdim] and piece_decay
-// [n_seqs, max_pieces, heads]; max_pieces * piece covers the longest run.
-RI_API int ri_state_scan(const float* u, int ld, int q_col, int k_col, int v_col, int decay_col, int step_col, const float* skip,
-                         float* state, float* o, const int* cu_seqlens, const int* seq_slot, int n_seqs, int heads, int groups,
-                         int dim, int vdim, int delta, int longest_run, int piece, int max_pieces, float* piece_state,
-                         float* piece_decay, cudaStream_t stream) {
+// [n_seqs, max_pieces, heads]; max_pieces * piece covers the longest run.  `decay` null: decays at decay_col; else, for the
+// delta rule, a decay per key channel (float32 [n_tokens, heads * dim]; decay_col is not read), for the state space a decay
+// per head that never changes (float32 [heads]; the step is 1, and neither decay_col nor step_col is read).
+RI_API int ri_state_scan(const float* u, int ld, int q_col, int k_col, int v_col, int decay_col, int step_col, const float* decay,
+                         const float* skip, float* state, float* o, const int* cu_seqlens, const int* seq_slot, int n_seqs,
+                         int heads, int groups, int dim, int vdim, int delta, int longest_run, int piece, int max_pieces,
+                         float* piece_state, float* piece_decay, cudaStream_t stream) {
     if (n_seqs <= 0) return 0;
     if (groups <= 0 || heads % groups) return fail("state_scan: %d heads are not a multiple of %d groups", heads, groups);
     if (heads > 65535) return fail("state_scan: %d heads exceed the grid limit", heads);
     if (dim > 32 * R) return fail("state_scan: a state of %d rows exceeds %d", dim, 32 * R);
     int rows = (dim + R - 1) / R;
     rows = rows <= 4 ? 4 : rows <= 8 ? 8 : rows <= 16 ? 16 : 32;
-    const int vec = ((ld | q_col | k_col | v_col | dim | vdim) % 4 == 0 && (reinterpret_cast<uintptr_t>(u) & 15) == 0) ? 1 : 0;
+    const int source = decay == nullptr ? PER_TOKEN : (delta ? CHANNELS : FIXED);
+    const int vec = ((ld | q_col | k_col | v_col | dim | vdim) % 4 == 0 && (reinterpret_cast<uintptr_t>(u) & 15) == 0 &&
+                     (source != CHANNELS || (reinterpret_cast<uintptr_t>(decay) & 15) == 0)) ? 1 : 0;
     if (piece > 0) {
         if (delta) return fail("state_scan: the delta rule's update is not a scalar times the state: no pieces");
         if (max_pieces < 1 || piece_state == nullptr || piece_decay == nullptr) return fail("state_scan: pieces need their scratch");
         if ((long long)n_seqs * max_pieces > 0x7fffffffLL || n_seqs > 65535) return fail("state_scan: %d sequences of %d pieces exceed the grid limit", n_seqs, max_pieces);
         if (longest_run <= 0 || longest_run > piece) longest_run = piece;
     }
-    Scan p{u, ld, q_col, k_col, v_col, decay_col, step_col, skip, state, o, cu_seqlens, seq_slot, heads, groups, dim, vdim, 1, vec,
+    Scan p{u, ld, q_col, k_col, v_col, decay_col, step_col, decay, skip, state, o, cu_seqlens, seq_slot, heads, groups, dim, vdim, 1, vec,
            piece > 0 ? piece : 0, piece > 0 ? max_pieces : 1, piece_state, piece_decay};
     dim3 grid(n_seqs, heads, (vdim + COLS - 1) / COLS);
-    if (rows == 4) return launch_scan<4>(delta != 0, grid, stream, p, longest_run, n_seqs);
-    if (rows == 8) return launch_scan<8>(delta != 0, grid, stream, p, longest_run, n_seqs);
-    if (rows == 16) return launch_scan<16>(delta != 0, grid, stream, p, longest_run, n_seqs);
-    return launch_scan<32>(delta != 0, grid, stream, p, longest_run, n_seqs);
+    if (rows == 4) return pick_scan<4>(delta != 0, source, grid, stream, p, longest_run, n_seqs);
+    if (rows == 8) return pick_scan<8>(delta != 0, source, grid, stream, p, longest_run, n_seqs);
+    if (rows == 16) return pick_scan<16>(delta != 0, source, grid, stream, p, longest_run, n_seqs);
+    return pick_scan<32>(delta != 0, source, grid, stream, p, longest_run, n_seqs);
 }
 
 RI_API int ri_gated_group_norm(const float* x, int x_ld, const float* gate, int gate_ld, int gate_col, const float* w, int w_len,
-                               void* out, int dtype, int n_tokens, int groups, int gs, int gate_first, float eps, float out_scale,
-                               cudaStream_t stream) {
+                               void* out, int dtype, int n_tokens, int groups, int gs, int gate_first, int sigmoid, float eps,
+                               float out_scale, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (groups <= 0 || gs <= 0 || w_len <= 0) return fail("gated_group_norm: %d groups of %d channels, %d weights", groups, gs, w_len);
     const long long warps = (long long)n_tokens * groups;
@@ -489,14 +699,14 @@ RI_API int ri_gated_group_norm(const float* x, int x_ld, const float* gate, int 
     cudaError_t e;
     if (dtype == RI_F32)
         e = wide ? launch_dependent(gated_group_norm_block_kernel<float>, (int)warps, 256, 0, stream, x, x_ld, gate, gate_ld, gate_col,
-                                    w, w_len, (float*)out, groups, gs, gate_first, eps, out_scale)
+                                    w, w_len, (float*)out, groups, gs, gate_first, sigmoid, eps, out_scale)
                  : launch_dependent(gated_group_norm_kernel<float>, blocks, 256, 0, stream, x, x_ld, gate, gate_ld, gate_col, w, w_len,
-                                    (float*)out, n_tokens, groups, gs, gate_first, eps, out_scale);
+                                    (float*)out, n_tokens, groups, gs, gate_first, sigmoid, eps, out_scale);
     else if (dtype == RI_BF16)
         e = wide ? launch_dependent(gated_group_norm_block_kernel<__nv_bfloat16>, (int)warps, 256, 0, stream, x, x_ld, gate, gate_ld,
-                                    gate_col, w, w_len, (__nv_bfloat16*)out, groups, gs, gate_first, eps, out_scale)
+                                    gate_col, w, w_len, (__nv_bfloat16*)out, groups, gs, gate_first, sigmoid, eps, out_scale)
                  : launch_dependent(gated_group_norm_kernel<__nv_bfloat16>, blocks, 256, 0, stream, x, x_ld, gate, gate_ld, gate_col, w,
-                                    w_len, (__nv_bfloat16*)out, n_tokens, groups, gs, gate_first, eps, out_scale);
+                                    w_len, (__nv_bfloat16*)out, n_tokens, groups, gs, gate_first, sigmoid, eps, out_scale);
     else
         return fail("gated_group_norm: unknown dtype %d", dtype);
     return check_launch(e, "gated_group_norm");

@@ -41,7 +41,7 @@ class _Layer:
         self.block = arrangement(**self.parts)
 
     def cache_request(self):
-        return self.cache_owner.cache_request() if self.cache_owner is not None else None
+        return self.block.cache_request(self.cache_owner.cache_request() if self.cache_owner is not None else None)
 
     def named_parts(self):
         for role, part in self.parts.items():

@@ -37,6 +37,7 @@ MODULES = {
     "latent_attention_mma": "latent_attention_mma.cu",
     "stream": "stream.cu",
     "state_scan": "state_scan.cu",
+    "short_conv": "short_conv.cu",
     "wait_probe": "wait_probe.cu",
     "host_runtime": "host_runtime.cpp",
 }

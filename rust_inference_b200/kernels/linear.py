@@ -39,8 +39,13 @@ def project(x, w: Weight, out, ctx, bias=None):
     return ops.gemm_simt(x, w.t, out, ops.EPI_STORE, bias=bias)
 
 
-def logits(x, w: Weight, out, ctx):
-    """out<float32> = x W^T."""
+def logits(x, w: Weight, out, ctx, silu_cols=None):
+    """out<float32> = x W^T; with silu_cols (float32 [1] on the device) the first so many columns through silu."""
+    if silu_cols is not None:
+        if _use_tensor_cores(x, w):
+            from . import tcgen05
+            return tcgen05.gemm(x, w, out, ops.EPI_SILU_F32, ctx, silu_cols=silu_cols)
+        return ops.gemm_simt(x, w.t, out, ops.EPI_SILU_F32, silu_cols=silu_cols)
     if _use_tensor_cores(x, w):
         from . import tcgen05
         return tcgen05.gemm(x, w, out, ops.EPI_STORE_F32, ctx)
@@ -66,8 +71,8 @@ def gated(x, w_gate: Weight, w_up: Weight, out, ctx, form=None):
 
 
 def activated(x, w: Weight, out, ctx, form):
-    """out<run dtype> = act(x W^T), the learned activation of `ops.xielu` with its two constants `form` (float32 [2] on
-    the device), applied to the float32 accumulators in the product's epilogue."""
+    """out<run dtype> = act(x W^T), an activation with its four constants `form` (float32 on the device: `ops.xielu`'s
+    two learned numbers through `ops.whole_act_form`, or `ops.RELU_SQUARED_FORM`), applied to the float32 accumulators in the product's epilogue."""
     if _use_tensor_cores(x, w):
         from . import tcgen05
         return tcgen05.gemm(x, w, out, ops.EPI_ACT, ctx, act_form=form)

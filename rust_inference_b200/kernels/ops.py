@@ -323,7 +323,7 @@ def silu_mul(gate_up: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
 
 
 # epilogues of the contractions
-EPI_STORE, EPI_STORE_F32, EPI_RESIDUAL, EPI_SILU_MUL, EPI_ACT = 0, 1, 2, 3, 4
+EPI_STORE, EPI_STORE_F32, EPI_RESIDUAL, EPI_SILU_MUL, EPI_ACT, EPI_SILU_F32 = 0, 1, 2, 3, 4, 5
 
 
 GELU_TANH_ALPHA = 2.0 * math.sqrt(2.0 / math.pi)      # 0.5 z (1 + tanh(y)) = z sigmoid(2 y)
@@ -345,19 +345,31 @@ def whole_gate_form(form: torch.Tensor) -> torch.Tensor:
     return form
 
 
+RELU_SQUARED_FORM = (1.0, 0.0, 0.0, 1.0)          # the activation epilogue's constants for max(z, 0)^2
+
+
+def whole_act_form(form: torch.Tensor) -> torch.Tensor:
+    """An activation given as its two learned numbers (`xielu`) gets the slope 1/2 and the mark of a learned form."""
+    if form.numel() == 2:
+        return torch.cat([form.reshape(-1), form.new_tensor([0.5, 0.0])])
+    return form
+
+
 def gemm_simt(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, mode: int, *,
               bias: torch.Tensor | None = None, w2: torch.Tensor | None = None,
-              gate_form: torch.Tensor | None = None, act_form: torch.Tensor | None = None) -> torch.Tensor:
+              gate_form: torch.Tensor | None = None, act_form: torch.Tensor | None = None,
+              silu_cols: torch.Tensor | None = None) -> torch.Tensor:
     """out = x @ w.T with the chosen epilogue, on the FFMA pipe (float32 accumulate).  gate_form (gated
     epilogue only): float32 [5] on the device (`gate_form`; the first three alone are accepted), {alpha, limit, shift, cubic, mult} of mult g' sigmoid(alpha g' (1 + cubic g'^2)) (u' + shift) with
-    g' = min(g, limit), u' = clamp(u, -limit, limit); None: SiLU(g) * u.  act_form (EPI_ACT only): float32 [2] on the
-    device, the two constants of the learned activation (`xielu`)."""
+    g' = min(g, limit), u' = clamp(u, -limit, limit); None: SiLU(g) * u.  act_form (EPI_ACT only): float32 [4] on the
+    device, the activation's constants (`RELU_SQUARED_FORM`; two learned ones alone are accepted, `whole_act_form`).
+    silu_cols (EPI_SILU_F32 only): float32 [1] on the device, how many of the first columns become silu of themselves."""
     _need_cuda(x, w, out, bias, w2)
     m, k = x.shape
     n = w.shape[0]
     _need(w.shape[1] == k and x.dtype == w.dtype and x.is_contiguous() and w.is_contiguous()
           and out.is_contiguous() and out.shape == (m, n), "gemm: bad shapes")
-    want_out = torch.float32 if mode in (EPI_STORE_F32, EPI_RESIDUAL) else x.dtype
+    want_out = torch.float32 if mode in (EPI_STORE_F32, EPI_RESIDUAL, EPI_SILU_F32) else x.dtype
     _need(out.dtype == want_out, f"gemm: epilogue {mode} writes {want_out}, out is {out.dtype}")
     if bias is not None:
         _need(bias.dtype == torch.float32 and bias.numel() == n, "gemm: bias must be float32 [N]")
@@ -370,9 +382,15 @@ def gemm_simt(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, mode: int, *,
         bias = gate_form                      # the gated epilogue takes no bias: its constants travel in that argument
     _need((mode == EPI_ACT) == (act_form is not None), "gemm: the activation epilogue and its constants go together")
     if act_form is not None:
-        _need(bias is None and act_form.is_cuda and act_form.dtype == torch.float32 and act_form.numel() == 2,
-              "gemm: an activation's form is two float32 constants, and its epilogue takes no bias")
+        act_form = whole_act_form(act_form)
+        _need(bias is None and act_form.is_cuda and act_form.dtype == torch.float32 and act_form.numel() == 4,
+              "gemm: an activation's form is four float32 constants, and its epilogue takes no bias")
         bias = act_form
+    _need((mode == EPI_SILU_F32) == (silu_cols is not None), "gemm: the partly activated epilogue and its number of columns go together")
+    if silu_cols is not None:
+        _need(bias is None and silu_cols.is_cuda and silu_cols.dtype == torch.float32 and silu_cols.numel() == 1,
+              "gemm: the number of activated columns is one float32 on the device, and its epilogue takes no bias")
+        bias = silu_cols
     _call("gemm_simt", "ri_gemm_simt", _p(x), _p(w), _p(w2), _p(bias), _p(out), c_int(dtype_code(x.dtype)),
           c_int(mode), c_int(m), c_int(n), c_int(k), _stream())
     return out
@@ -762,13 +780,14 @@ def gated_linear_attention(z: torch.Tensor, *, q_col: int, k_col: int, v_col: in
 # ----------------------------------------------------------------------------
 # Routed experts (csrc/moe.cu)
 # ----------------------------------------------------------------------------
-def moe_route(x: torch.Tensor, router: torch.Tensor, correction: torch.Tensor, ids: torch.Tensor,
+def moe_route(x: torch.Tensor, router: torch.Tensor, correction: torch.Tensor | None, ids: torch.Tensor,
               weights: torch.Tensor, *, top: int, groups: int = 1, keep: int = 1,
               gate_weight: torch.Tensor | None = None, gate_out: torch.Tensor | None = None,
               softmax: bool = False, normalise: bool = True, split: int = 1, split_sums: torch.Tensor | None = None,
-              split_count: torch.Tensor | None = None) -> None:
+              split_count: torch.Tensor | None = None, group_max: bool = False) -> None:
     """Per token the `top` experts with the largest sigmoid(router x) + correction among the `keep` best of
-    `groups` groups (a group's score: the sum of its two largest), ids int32 [T, top], and their weights
+    `groups` groups (a group's score: the sum of its two largest, or with group_max its largest alone; correction None:
+    zero), ids int32 [T, top], and their weights
     float32 [T, top] (the plain sigmoid scores, normalised).  gate_weight float32 [width]: gate_out[t] =
     sigmoid(gate_weight . x_t) as well.  softmax: the scores are softmax(router x) over all experts instead of
     sigmoids; normalise False: the weights are the chosen scores as they are.  split > 1 (steps of fewer than 296
@@ -778,7 +797,7 @@ def moe_route(x: torch.Tensor, router: torch.Tensor, correction: torch.Tensor, i
     n, width = x.shape
     experts = router.shape[0]
     _need(x.is_contiguous() and router.dtype == torch.float32 and router.is_contiguous() and router.shape[1] == width
-          and correction.dtype == torch.float32 and correction.numel() == experts, "moe_route: router and correction")
+          and (correction is None or (correction.dtype == torch.float32 and correction.numel() == experts)), "moe_route: router and correction")
     _need(ids.dtype == torch.int32 and ids.is_contiguous() and ids.numel() >= n * top and weights.dtype == torch.float32
           and weights.is_contiguous() and weights.numel() >= n * top, "moe_route: ids int32 and weights float32 [T, top]")
     _need((gate_weight is None) == (gate_out is None), "moe_route: gate weight and output go together")
@@ -792,7 +811,7 @@ def moe_route(x: torch.Tensor, router: torch.Tensor, correction: torch.Tensor, i
               and split_count.numel() >= n, "moe_route: rows cut over blocks need few tokens, float32 sums and int32 counters")
     _call("moe", "ri_moe_route", _p(x), c_int(dtype_code(x.dtype)), _p(router), _p(correction), _p(gate_weight), _p(ids),
           _p(weights), _p(gate_out), c_int(n), c_int(width), c_int(experts), c_int(top), c_int(groups), c_int(keep),
-          c_int((1 if softmax else 0) | (0 if normalise else 2)), c_int(max(1, split)), _p(split_sums if split > 1 else None),
+          c_int((1 if softmax else 0) | (0 if normalise else 2) | (4 if group_max else 0)), c_int(max(1, split)), _p(split_sums if split > 1 else None),
           _p(split_count if split > 1 else None), _stream())
 
 
@@ -1064,6 +1083,7 @@ def xielu(x: torch.Tensor, out: torch.Tensor, pq: torch.Tensor) -> torch.Tensor:
     _need_cuda(x, out, pq)
     _need(x.dtype == out.dtype and x.is_contiguous() and out.is_contiguous() and x.numel() == out.numel(), "xielu: shapes")
     _f32_vec(pq, 2, "xielu: parameters")
+    pq = whole_act_form(pq)
     _call("stream", "ri_xielu", _p(x), _p(out), c_int(dtype_code(x.dtype)), _p(pq), c_longlong(x.numel()), _stream())
     return out
 
@@ -1083,13 +1103,14 @@ def add_row_bias(x: torch.Tensor, bias: torch.Tensor) -> torch.Tensor:
 def scan_prepare(z: torch.Tensor, *, conv_col: int, conv_ch: int, taps: torch.Tensor, conv_bias, conv_state: torch.Tensor,
                  unit_heads: int, unit_dim: int, scaled_heads: int, unit_scale: float, heads: int, decay_col: int,
                  step_col: int, a_log: torch.Tensor, dt_bias: torch.Tensor, out: torch.Tensor, cu_seqlens, token_seq,
-                 seq_slot, n_seqs: int) -> torch.Tensor:
+                 seq_slot, n_seqs: int, longest_run: int = 0) -> torch.Tensor:
     """Per token of z (float32 [T, ld]): the short causal convolution (taps float32 [conv_ch, K], last column the
     current token's; bias or None) and silu of the columns conv_col .. conv_col + conv_ch, reading the inputs before
     the step from conv_state (float32 [slots, K - 1, conv_ch]) and moving those on; the first unit_heads heads of
     unit_dim channels made unit vectors (the first scaled_heads of them times unit_scale); per head the decay
     exp(-exp(a_log) * softplus(z[decay_col + h] + dt_bias)) and the step (sigmoid(z[step_col + h]), or with
-    step_col < 0 the softplus itself).  out: float32 [T, >= conv_ch + 2 heads] = [channels | decays | steps]."""
+    step_col < 0 the softplus itself).  out: float32 [T, >= conv_ch + 2 heads] = [channels | decays | steps].
+    longest_run: the most new tokens any sequence brings (0: unknown)."""
     _need_cuda(z, taps, conv_bias, conv_state, a_log, dt_bias, out, cu_seqlens, token_seq, seq_slot)
     t = z.shape[0]
     k = taps.shape[1]
@@ -1103,21 +1124,76 @@ def scan_prepare(z: torch.Tensor, *, conv_col: int, conv_ch: int, taps: torch.Te
     _call("state_scan", "ri_scan_prepare", _p(z), c_int(z.shape[1]), c_int(conv_col), c_int(conv_ch), _p(taps), _p(conv_bias),
           c_int(k), _p(conv_state), c_int(unit_heads), c_int(unit_dim), c_int(scaled_heads), c_float(unit_scale), c_int(heads),
           c_int(decay_col), c_int(step_col), _p(a_log), _p(dt_bias), _p(out), c_int(out.shape[1]), _p(cu_seqlens),
-          _p(token_seq), _p(seq_slot), c_int(t), c_int(n_seqs), _stream())
+          _p(token_seq), _p(seq_slot), c_int(t), c_int(n_seqs), c_int(longest_run), _stream())
+    return out
+
+
+LOW_RANK_FORMED_TOKENS = 16        # steps of up to so many tokens: `scan_prepare_channels` forms the low-rank maps itself
+
+
+def scan_prepare_channels(z: torch.Tensor, *, conv_col: int, conv_ch: int, taps: torch.Tensor, conv_state: torch.Tensor,
+                          unit_heads: int, unit_dim: int, scaled_heads: int, unit_scale: float, heads: int, head_dim: int,
+                          step_col: int, a_log: torch.Tensor, dt_bias: torch.Tensor, out: torch.Tensor, decay: torch.Tensor,
+                          cu_seqlens, token_seq, seq_slot, n_seqs: int, longest_run: int = 0, raw: torch.Tensor | None = None,
+                          w2: torch.Tensor | None = None, low_col: int = 0, gate_w2: torch.Tensor | None = None,
+                          gate_low_col: int = 0, gate_out: torch.Tensor | None = None) -> torch.Tensor:
+    """`scan_prepare` with a decay per head and key channel: decay (float32 [T, heads * head_dim]) receives
+    exp(-exp(a_log[head]) * softplus(x + dt_bias[channel])), x = raw (the same shape; may be `decay` itself) or, with raw
+    None, x = w2 (z[:, low_col : low_col + rank]) formed here (w2 [heads * head_dim, rank], float32 or bfloat16).  gate_w2 (its
+    dtype, [channels, rank']): gate_out (float32 [T, channels]) = gate_w2 (z[:, gate_low_col ..]) as well."""
+    _need_cuda(z, taps, conv_state, a_log, dt_bias, out, decay, raw, w2, gate_w2, gate_out, cu_seqlens, token_seq, seq_slot)
+    t, k, n = z.shape[0], taps.shape[1], heads * head_dim
+    _need(z.dtype == torch.float32 and z.is_contiguous() and out.dtype == torch.float32 and out.is_contiguous()
+          and out.shape[0] == t, "scan_prepare: z and out must be float32 [T, .]")
+    _need(taps.dtype == torch.float32 and taps.is_contiguous() and taps.shape[0] == conv_ch, "scan_prepare: taps")
+    _need(conv_state.dtype == torch.float32 and conv_state.is_contiguous()
+          and tuple(conv_state.shape[1:]) == (max(k - 1, 0), conv_ch), "scan_prepare: carried inputs must be [slots, K - 1, channels]")
+    _f32_vec(a_log, heads, "scan_prepare: A_log"); _f32_vec(dt_bias, n, "scan_prepare: dt_bias")
+    for m in (decay, raw):
+        _need(m is None or (m.dtype == torch.float32 and m.is_contiguous() and tuple(m.shape) == (t, n)), "scan_prepare: decays must be float32 [T, heads * head_dim]")
+    _need((raw is None) == (w2 is not None), "scan_prepare: decays come from `raw` or from `w2`")
+    _need(w2 is None or (w2.is_contiguous() and w2.shape[0] == n and w2.dtype in _DTYPE_CODE), "scan_prepare: w2 must be [heads * head_dim, rank]")
+    _need((gate_w2 is None) == (gate_out is None), "scan_prepare: a low-rank gate and its result go together")
+    if gate_w2 is not None:
+        _need(gate_w2.is_contiguous() and gate_out.dtype == torch.float32 and gate_out.is_contiguous()
+              and tuple(gate_out.shape) == (t, gate_w2.shape[0]) and (w2 is None or gate_w2.dtype == w2.dtype), "scan_prepare: the low-rank gate")
+    some = w2 if w2 is not None else gate_w2
+    _call("state_scan", "ri_scan_prepare_channels", _p(z), c_int(z.shape[1]), c_int(conv_col), c_int(conv_ch), _p(taps), _p(None),
+          c_int(k), _p(conv_state), c_int(unit_heads), c_int(unit_dim), c_int(scaled_heads), c_float(unit_scale), c_int(heads),
+          c_int(step_col), _p(a_log), _p(dt_bias), _p(out), c_int(out.shape[1]), _p(cu_seqlens), _p(token_seq), _p(seq_slot), c_int(t),
+          c_int(n_seqs), c_int(longest_run), c_int(head_dim), _p(raw), _p(decay), _p(w2), c_int(w2.shape[1] if w2 is not None else 0),
+          c_int(low_col), c_int(gate_w2.shape[0] if gate_w2 is not None else 0), c_int(gate_w2.shape[1] if gate_w2 is not None else 0),
+          c_int(gate_low_col), _p(gate_w2), _p(gate_out), c_int(dtype_code(some.dtype) if some is not None else RI_F32), _stream())
+    return out
+
+
+def low_rank_rows(z: torch.Tensor, low_col: int, rank: int, padded: int, out: torch.Tensor) -> torch.Tensor:
+    """The columns low_col .. low_col + rank of z (float32 [T, .]) as rows of their own: float32 out [T, padded], or bfloat16
+    out [T, 2 * padded] with the rounded values and then the rounded remainders; columns beyond rank are zero."""
+    _need_cuda(z, out)
+    halves = 2 if out.dtype == torch.bfloat16 else 1
+    _need(z.dtype == torch.float32 and z.is_contiguous() and out.is_contiguous() and tuple(out.shape) == (z.shape[0], halves * padded),
+          "low_rank_rows: shapes")
+    _call("state_scan", "ri_low_rank_rows", _p(z), c_int(z.shape[1]), c_int(low_col), c_int(rank), c_int(padded), _p(out),
+          c_int(dtype_code(out.dtype)), c_int(z.shape[0]), _stream())
     return out
 
 
 def state_scan(u: torch.Tensor, state: torch.Tensor, o: torch.Tensor, cu_seqlens, seq_slot, *, n_seqs: int, heads: int,
                groups: int, dim: int, vdim: int, q_col: int, k_col: int, v_col: int, decay_col: int, step_col: int,
                delta: bool, skip=None, longest_run: int = 0, piece: int = 0, max_pieces: int = 1, piece_state=None,
-               piece_decay=None) -> torch.Tensor:
+               piece_decay=None, decay: torch.Tensor | None = None) -> torch.Tensor:
     """The recurrence over every sequence's new tokens from its slot's state (float32 [slots, heads, dim, vdim]), which
     moves on.  u: float32 [T, ld] with the columns of queries and keys ([groups, dim] each), values ([heads, vdim]),
     decays and steps ([heads] each); o: float32 [T, heads * vdim].  delta: the gated delta rule
     (S <- a S; S += k (step (v - S^T k))^T); else S <- a S + k (step v)^T and o += skip * v.  piece > 0 (not the delta
     rule): long runs are scanned in pieces of that many tokens side by side, from zero, then again from start states that
     a carry over the pieces gives; float32 scratch piece_state [n_seqs, max_pieces, heads, dim, vdim] and piece_decay
-    [n_seqs, max_pieces, heads], max_pieces * piece at least the longest run."""
+    [n_seqs, max_pieces, heads], max_pieces * piece at least the longest run.  decay: with delta a decay per key channel
+    (float32 [T, heads * dim]) in place of the column; without, one that never changes per head (float32 [heads]), with step 1."""
+    if decay is not None:
+        _need_cuda(decay)
+        _f32_vec(decay, u.shape[0] * heads * dim if delta else heads, "state_scan: decay")
     _need_cuda(u, state, o, cu_seqlens, seq_slot, skip, piece_state, piece_decay)
     if piece > 0:
         _need(not delta and piece_state is not None and piece_decay is not None and piece_state.dtype == torch.float32
@@ -1131,7 +1207,7 @@ def state_scan(u: torch.Tensor, state: torch.Tensor, o: torch.Tensor, cu_seqlens
     if skip is not None:
         _f32_vec(skip, heads, "state_scan: skip")
     _call("state_scan", "ri_state_scan", _p(u), c_int(u.shape[1]), c_int(q_col), c_int(k_col), c_int(v_col), c_int(decay_col),
-          c_int(step_col), _p(skip), _p(state), _p(o), _p(cu_seqlens), _p(seq_slot), c_int(n_seqs), c_int(heads), c_int(groups),
+          c_int(step_col), _p(decay), _p(skip), _p(state), _p(o), _p(cu_seqlens), _p(seq_slot), c_int(n_seqs), c_int(heads), c_int(groups),
           c_int(dim), c_int(vdim), c_int(1 if delta else 0), c_int(longest_run), c_int(piece), c_int(max_pieces),
           _p(piece_state), _p(piece_decay), _stream())
     return o
@@ -1151,18 +1227,74 @@ def scan_pieces(max_new: int, blocks: int) -> tuple:
 
 
 def gated_group_norm(x: torch.Tensor, gate: torch.Tensor, gate_col: int, weight: torch.Tensor, out: torch.Tensor, *,
-                     groups: int, group_size: int, gate_first: bool, eps: float, out_scale: float = 1.0) -> torch.Tensor:
+                     groups: int, group_size: int, gate_first: bool, eps: float, out_scale: float = 1.0,
+                     gate_act: str = "silu") -> torch.Tensor:
     """Per token and group of group_size channels of x (float32 [T, groups * group_size]): RMS norm over the group times
-    weight[channel % len(weight)], and a gate silu(gate[t, gate_col + channel]) applied before the norm (gate_first) or
-    after it; the result times out_scale into out (float32 or bfloat16)."""
+    weight[channel % len(weight)], and a gate silu(gate[t, gate_col + channel]) (gate_act "sigmoid": the sigmoid instead)
+    applied before the norm (gate_first) or after it; the result times out_scale into out (float32 or bfloat16)."""
     _need_cuda(x, gate, weight, out)
     t = x.shape[0]
     _need(x.dtype == torch.float32 and x.is_contiguous() and x.shape[1] == groups * group_size, "gated_group_norm: x")
     _need(gate.dtype == torch.float32 and gate.is_contiguous() and gate.shape[0] == t
           and gate.shape[1] >= gate_col + groups * group_size, "gated_group_norm: gate")
     _need(weight.dtype == torch.float32 and weight.is_contiguous(), "gated_group_norm: weight")
+    _need(gate_act in ("silu", "sigmoid"), "gated_group_norm: gate_act is silu or sigmoid")
     _need(out.is_contiguous() and tuple(out.shape) == (t, groups * group_size), "gated_group_norm: out")
     _call("state_scan", "ri_gated_group_norm", _p(x), c_int(x.shape[1]), _p(gate), c_int(gate.shape[1]), c_int(gate_col), _p(weight),
           c_int(weight.numel()), _p(out), c_int(dtype_code(out.dtype)), c_int(t), c_int(groups), c_int(group_size),
-          c_int(1 if gate_first else 0), c_float(eps), c_float(out_scale), _stream())
+          c_int(1 if gate_first else 0), c_int(1 if gate_act == "sigmoid" else 0), c_float(eps), c_float(out_scale), _stream())
     return out
+
+
+# ----------------------------------------------------------------------------
+# Short causal convolutions on a layer's input and on an attention's projections (csrc/short_conv.cu)
+# ----------------------------------------------------------------------------
+def input_conv(x: torch.Tensor, weight, eps: float, taps_a: torch.Tensor, taps_b, carried: torch.Tensor, out_a: torch.Tensor,
+               out_b, cu_seqlens, token_seq, seq_slot, *, n_seqs: int, longest_run: int) -> None:
+    """h = x / sqrt(mean(x^2) + eps) * weight (weight None: h = x) of the float32 rows x [T, n]; out_a = h + conv_a(h), and
+    with taps_b out_b = h + conv_b(h): causal convolutions per channel, taps float32 [K, n] (the last row the current
+    token's), the inputs before the step from carried (float32 [slots, K - 1, n]), which moves on.  longest_run: the most
+    new tokens any sequence brings."""
+    _need_cuda(x, weight, taps_a, taps_b, carried, out_a, out_b, cu_seqlens, token_seq, seq_slot)
+    t, n = x.shape
+    k = taps_a.shape[0]
+    _need(x.dtype == torch.float32 and x.is_contiguous(), "input_conv: x must be float32 [T, n]")
+    _need((taps_b is None) == (out_b is None), "input_conv: a second filter and its output go together")
+    for w in (taps_a, taps_b):
+        _need(w is None or (w.dtype == torch.float32 and w.is_contiguous() and tuple(w.shape) == (k, n)), "input_conv: taps must be float32 [K, n]")
+    if weight is not None:
+        _f32_vec(weight, n, "input_conv: weight")
+    _need(carried.dtype == torch.float32 and carried.is_contiguous() and tuple(carried.shape[1:]) == (k - 1, n),
+          "input_conv: carried inputs must be float32 [slots, K - 1, n]")
+    for o in (out_a, out_b):
+        _need(o is None or (o.is_contiguous() and tuple(o.shape) == (t, n) and o.dtype == out_a.dtype), "input_conv: outputs")
+    _call("short_conv", "ri_input_conv", _p(x), _p(weight), c_float(eps), _p(taps_a), _p(taps_b), c_int(k), _p(carried), _p(out_a),
+          _p(out_b), c_int(dtype_code(out_a.dtype)), _p(cu_seqlens), _p(token_seq), _p(seq_slot), c_int(t), c_int(n_seqs), c_int(n),
+          c_int(longest_run), _stream())
+
+
+def conv_store(z: torch.Tensor, bias, taps: torch.Tensor, carried: torch.Tensor, q_out: torch.Tensor, kcache, vcache, cu_seqlens,
+               token_pos, token_seq, seq_slot, page_table, *, n_seqs: int, n_kv_heads: int, head_dim: int, v_head_dim: int,
+               page_size: int, longest_run: int) -> torch.Tensor:
+    """From the projection z (float32 [T, >= channels]: queries, keys, values) plus bias: a short causal convolution per channel
+    (taps float32 [K, channels], the last row the current token's; inputs before the step, biases included, from carried,
+    float32 [slots, K - 1, channels], which moves on), then the queries into q_out [T, q channels] and keys and values into
+    the tokens' places of the paged cache."""
+    _need_cuda(z, bias, taps, carried, q_out, kcache, vcache, cu_seqlens, token_pos, token_seq, seq_slot, page_table)
+    t, q_dim = q_out.shape
+    k, channels = taps.shape
+    _need(z.dtype == torch.float32 and z.is_contiguous() and z.shape[0] == t and z.shape[1] >= channels
+          and channels == q_dim + n_kv_heads * (head_dim + v_head_dim), "conv_store: z must be float32 [T, channels]")
+    _need(taps.dtype == torch.float32 and taps.is_contiguous(), "conv_store: taps must be float32 [K, channels]")
+    if bias is not None:
+        _f32_vec(bias, channels, "conv_store: bias")
+    _need(carried.dtype == torch.float32 and carried.is_contiguous() and tuple(carried.shape[1:]) == (k - 1, channels),
+          "conv_store: carried inputs must be float32 [slots, K - 1, channels]")
+    _need(q_out.is_contiguous() and kcache.dtype == q_out.dtype and vcache.dtype == q_out.dtype and kcache.is_contiguous()
+          and vcache.is_contiguous() and tuple(kcache.shape[1:]) == (n_kv_heads, page_size, head_dim)
+          and tuple(vcache.shape[1:]) == (n_kv_heads, page_size, v_head_dim), "conv_store: queries and cache")
+    _call("short_conv", "ri_conv_store", _p(z), c_int(z.shape[1]), _p(bias), _p(taps), c_int(k), _p(carried), _p(q_out), _p(kcache),
+          _p(vcache), c_int(dtype_code(q_out.dtype)), _p(cu_seqlens), _p(token_pos), _p(token_seq), _p(seq_slot), _p(page_table),
+          c_int(page_table.shape[1]), c_int(t), c_int(n_seqs), c_int(q_dim), c_int(n_kv_heads), c_int(head_dim), c_int(v_head_dim),
+          c_int(page_size), c_int(longest_run), _stream())
+    return q_out

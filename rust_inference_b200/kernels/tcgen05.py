@@ -117,13 +117,13 @@ def _x_map(x: torch.Tensor, tn: int) -> torch.Tensor:
 
 
 def gemm(x: torch.Tensor, w, out: torch.Tensor, mode: int, ctx=None, bias=None, w2=None, split_k: int | None = None,
-         gate_form=None, act_form=None):
+         gate_form=None, act_form=None, silu_cols=None):
     _need_cuda(x, w.t, out, bias)
     m, k = x.shape
     n = w.n
     _need(w.k == k and x.dtype == torch.bfloat16 and w.t.dtype == torch.bfloat16 and x.is_contiguous()
           and out.is_contiguous() and out.shape == (m, n), "gemm_tcgen05: bad shapes or dtypes")
-    want_out = torch.float32 if mode in (ops.EPI_STORE_F32, ops.EPI_RESIDUAL) else torch.bfloat16
+    want_out = torch.float32 if mode in (ops.EPI_STORE_F32, ops.EPI_RESIDUAL, ops.EPI_SILU_F32) else torch.bfloat16
     _need(out.dtype == want_out, f"gemm_tcgen05: epilogue {mode} writes {want_out}, out is {out.dtype}")
     if bias is not None:
         _need(bias.dtype == torch.float32 and bias.numel() == n, "gemm_tcgen05: bias must be float32 [N]")
@@ -139,9 +139,15 @@ def gemm(x: torch.Tensor, w, out: torch.Tensor, mode: int, ctx=None, bias=None, 
         bias = gate_form
     _need((mode == ops.EPI_ACT) == (act_form is not None), "gemm_tcgen05: the activation epilogue and its constants go together")
     if act_form is not None:
-        _need(bias is None and act_form.is_cuda and act_form.dtype == torch.float32 and act_form.numel() == 2,
-              "gemm_tcgen05: an activation's form is two float32 constants, and its epilogue takes no bias")
+        act_form = ops.whole_act_form(act_form)
+        _need(bias is None and act_form.is_cuda and act_form.dtype == torch.float32 and act_form.numel() == 4,
+              "gemm_tcgen05: an activation's form is four float32 constants, and its epilogue takes no bias")
         bias = act_form
+    _need((mode == ops.EPI_SILU_F32) == (silu_cols is not None), "gemm_tcgen05: the partly activated epilogue and its number of columns go together")
+    if silu_cols is not None:
+        _need(bias is None and silu_cols.is_cuda and silu_cols.dtype == torch.float32 and silu_cols.numel() == 1,
+              "gemm_tcgen05: the number of activated columns is one float32 on the device, and its epilogue takes no bias")
+        bias = silu_cols
     if m == 0:
         return out
     tile, planned = plan(m, n, k, mode)

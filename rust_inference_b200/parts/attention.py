@@ -5,8 +5,8 @@ import math
 
 import torch
 
-from ..cache.sequence_cache import KVRequest
-from ..kernels import linear, attention as attn_kernels
+from ..cache.sequence_cache import KVRequest, StateRequest
+from ..kernels import linear, ops, attention as attn_kernels
 from .base import Mixer
 from .registry import register, lookup
 from .spec import TensorSpec, PartSpec
@@ -37,11 +37,16 @@ class GQAttention(Mixer):
     # projection, `names`: o_bias); `own_kv` False: the layer has no key and value projections and attends over the
     # cache of the layer the schedule gives it, with its own queries.  `out_gate`: the concatenated heads' result is
     # multiplied element by element with sigmoid(W_g x) before the output projection (one more row per value channel of
-    # every head in the projection, `names`: out_gate).
+    # every head in the projection, `names`: out_gate).  `conv`: queries, keys and values each pass a short causal convolution
+    # per channel right after the projection and its bias (so many taps, no activation; `names`: q_conv, k_conv, v_conv,
+    # [channels, taps], the last column the current token's); the projection's last conv - 1 rows, biases included, are a
+    # state of the sequence beside its keys and values.  `fixed_sink`: a sink that is the same number for every head and
+    # no tensor.
     _NAMES = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o": "o_proj.weight",
               "q_bias": "q_proj.bias", "k_bias": "k_proj.bias", "v_bias": "v_proj.bias",
               "q_norm": "q_norm.weight", "k_norm": "k_norm.weight", "o_bias": "o_proj.bias", "sink": "sinks",
-              "gate": "gate_proj.weight", "r1": "distance_r1", "r2": "distance_r2", "out_gate": "out_gate_proj.weight"}
+              "gate": "gate_proj.weight", "r1": "distance_r1", "r2": "distance_r2", "out_gate": "out_gate_proj.weight",
+              "q_conv": "q_conv1d.weight", "k_conv": "k_conv1d.weight", "v_conv": "v_conv1d.weight"}
 
     def __init__(self, *, n_heads: int, n_kv_heads: int, head_dim: int, qkv_bias: bool,
                  position: PartSpec, window: int | None = None, v_head_dim: int | None = None,
@@ -49,6 +54,7 @@ class GQAttention(Mixer):
                  names: dict | None = None, qk_norm_eps: float | None = None, values_from_keys: bool = False,
                  softcap: float = 0.0, distance_bias: bool = False, keep_first: int = 0, sink: bool = False,
                  head_gate: bool = False, o_bias: bool = False, own_kv: bool = True, out_gate: bool = False,
+                 conv: int | None = None, fixed_sink: float | None = None,
                  hidden_size: int, dtype, device):
         super().__init__(hidden_size=hidden_size, dtype=dtype, device=device)
         if n_heads % n_kv_heads:
@@ -83,7 +89,21 @@ class GQAttention(Mixer):
         # what only the general path (one projection, then the position encoding, then attention with these forms) does
         self.extended = bool(self.softcap or self.distance_bias or self.keep_first or self.sink or self.head_gate
                              or self.out_gate or not self.own_kv)
+        self.conv = None if conv is None else int(conv)
+        if self.conv is not None:
+            if self.conv < 1:
+                raise ValueError(f"a convolution has at least one tap, found {conv}")
+            if (self.values_from_keys or self.qk_norm_eps is not None or self.head_gate or self.out_gate or not self.own_kv
+                    or position.kind != "unrotated"):
+                raise ValueError("convolved projections go without rotation, head norms, gates, values taken from keys and another layer's keys")
+        if fixed_sink is not None and self.sink:
+            raise ValueError("a learned sink and a fixed one are not combined")
+        self.fixed_sink = None if fixed_sink is None else float(fixed_sink)
+        self.extended = self.extended or self.fixed_sink is not None or self.conv is not None
         self.sinks = self.dist = self.b_o = None
+        self.w_conv = None                      # [taps, channels]
+        # a caller that adds the output projection's bias itself (with what it does next to the result) sets this
+        self.hands_over_bias = False
         self.window = window
         self.chunk = chunk
         self.out_scale = float(out_scale)
@@ -116,6 +136,9 @@ class GQAttention(Mixer):
             specs[nm["r2"]] = TensorSpec((self.n_heads,), role="vector", init="ones")
         if self.o_bias:
             specs[nm["o_bias"]] = TensorSpec((h,), role="vector")
+        if self.conv is not None:
+            for name, rows in (("q_conv", self.q_dim), ("k_conv", self.kv_dim), ("v_conv", self.v_dim)):
+                specs[nm[name]] = TensorSpec((rows, self.conv), role="vector")
         if self.qk_norm_eps is not None:
             specs[nm["q_norm"]] = TensorSpec((self.head_dim,), role="vector", init="ones")
             specs[nm["k_norm"]] = TensorSpec((self.head_dim,), role="vector", init="ones")
@@ -141,6 +164,10 @@ class GQAttention(Mixer):
         self.w_qkv = linear.Weight(torch.cat(mats, dim=0))
         if self.sink:
             self.sinks = tensors[nm["sink"]].contiguous()
+        if self.fixed_sink is not None:
+            self.sinks = torch.full((self.n_heads,), self.fixed_sink, dtype=torch.float32, device=self.device)
+        if self.conv is not None:
+            self.w_conv = torch.cat([tensors[nm[n]] for n in ("q_conv", "k_conv", "v_conv")], dim=0).t().contiguous()
         if self.distance_bias:
             self.dist = torch.stack([tensors[nm["r1"]], tensors[nm["r2"]]], dim=0).contiguous()
         if self.o_bias:
@@ -178,6 +205,9 @@ class GQAttention(Mixer):
             out[nm["o_bias"]] = self.b_o
         if self.qk_norm_eps is not None:
             out[nm["q_norm"]], out[nm["k_norm"]] = self.q_norm, self.k_norm
+        if self.conv is not None:
+            taps = self.w_conv.t()
+            out[nm["q_conv"]], out[nm["k_conv"]], out[nm["v_conv"]] = taps[:q], taps[q:q + kv], taps[q + kv:]
         if self.qkv_bias:
             b = self.b_qkv
             out[nm["q_bias"]] = b[:q]
@@ -189,8 +219,25 @@ class GQAttention(Mixer):
         self.position.prepare(max_positions)
 
     def cache_request(self):
-        return KVRequest(self.n_kv_heads, self.head_dim, self.window,
+        keys = KVRequest(self.n_kv_heads, self.head_dim, self.window,
                          None if self.v_head_dim == self.head_dim else self.v_head_dim)
+        if self.conv is None:
+            return keys
+        return keys, StateRequest((self.conv - 1, self.q_dim + self.kv_dim + self.v_dim), torch.float32)
+
+    def _convolved(self, x, ctx, cache_layer, writes_cache):
+        """The queries [T, heads * head_dim] behind projection and convolution; keys and values go into the cache."""
+        if not writes_cache:
+            raise ValueError("a convolution's carried inputs have one writer: a layer cannot read another layer's")
+        keys, carried = cache_layer.parts
+        n = x.shape[0]
+        z = ctx.buffer("conv_z", (n, self.w_qkv.n), torch.float32)
+        linear.logits(x, self.w_qkv, z, ctx)                       # float32 results in both precisions
+        q = ctx.buffer("q_conv", (n, self.q_dim), self.dtype)
+        ops.conv_store(z, self.b_qkv, self.w_conv, carried.state, q, keys.k, keys.v, ctx.cu_seqlens, ctx.token_pos, ctx.token_seq,
+                       ctx.seq_slot, ctx.page_table, n_seqs=ctx.n_seqs, n_kv_heads=self.n_kv_heads, head_dim=self.head_dim,
+                       v_head_dim=self.v_head_dim, page_size=ctx.page_size, longest_run=ctx.max_new)
+        return q, keys
 
     def forward(self, x, residual, ctx, cache_layer, writes_cache):
         n = x.shape[0]
@@ -202,7 +249,9 @@ class GQAttention(Mixer):
         usual = (self.v_head_dim == self.head_dim and not getattr(self.position, "partial", False) and not special
                  and not self.extended)
         from_acc = getattr(self.position, "apply_and_store_from_accumulators", None) if usual else None
-        if from_acc is not None and linear.wants_split(x, self.w_qkv):
+        if self.conv is not None:
+            qkv, cache_layer = self._convolved(x, ctx, cache_layer, writes_cache)
+        elif from_acc is not None and linear.wants_split(x, self.w_qkv):
             # a small step: the projection is split over K into float32 accumulators, and the
             # position encoding adds the bias, rotates and stores from there
             acc = ctx.zeroed_buffer("qkv_acc", (n, width), torch.float32)
@@ -232,10 +281,9 @@ class GQAttention(Mixer):
                                out_scale=1.0 if self.out_gate else self.out_scale, softcap=self.softcap,
                                keep_first=self.keep_first, sink=self.sinks, dist=self.dist,
                                gate=qkv[:, gate_col:gate_col + self.n_heads] if self.head_gate else None)
-        from ..kernels import ops
         if self.out_gate:
             # the gates of the projection's last columns, the mixer's factor with them (float32, one rounding)
             ops.sigmoid_gate_(mixed, qkv, gate_col, self.out_scale)
         linear.into_residual(mixed, self.w_o, residual, ctx)
-        if self.o_bias:
+        if self.o_bias and not self.hands_over_bias:
             ops.add_row_bias(residual, self.b_o_scaled)

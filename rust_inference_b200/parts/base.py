@@ -148,7 +148,8 @@ class Arrangement:
 
     ROLES maps each role the arrangement has to the category its part is looked up in; a layer spec
     must give exactly these roles (those in OPTIONAL may be left out and are then None).  At most
-    one role may be of category "mixer": its part owns the layer's cache."""
+    one role may be of category "mixer": its part owns the layer's cache.  An arrangement that keeps something per sequence
+    itself says so in `cache_request` and takes its share out of the cache layer it is handed."""
 
     ROLES = {"mixer": "mixer", "feed_forward": "feed_forward", "mixer_norm": "norm", "feed_forward_norm": "norm"}
     OPTIONAL: tuple = ()
@@ -156,6 +157,10 @@ class Arrangement:
     def __init__(self, **parts):
         for role in self.ROLES:
             setattr(self, role, parts.get(role))
+
+    def cache_request(self, mixer_request):
+        """What the layer needs of the cache, given what its mixer asks for (None: it has none or asks for nothing)."""
+        return mixer_request
 
     def forward(self, residual: torch.Tensor, ctx, cache_layer, writes_cache: bool) -> None:
         raise NotImplementedError

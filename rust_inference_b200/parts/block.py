@@ -3,6 +3,7 @@ from __future__ import annotations
 
 import torch
 
+from ..cache.sequence_cache import StateRequest
 from ..kernels import ops
 from .base import Arrangement
 from .registry import register
@@ -77,6 +78,40 @@ class ParallelSharedNorm(Arrangement):
         self.mixer.forward(normed, residual, ctx, cache_layer, writes_cache)
         if self.feed_forward is not None:
             self.feed_forward.forward(normed, residual, ctx)
+
+
+@register("arrangement", "parallel_shared_norm_conv")
+class ParallelSharedNormConv(Arrangement):
+    """x <- x + (mixer(h + conv_a(h)) + ff(h + conv_b(h))) with h = norm(x): one norm, and each branch reads its output
+    behind a short causal convolution of its own.  Norm and both convolutions are one kernel; the last inputs h of a
+    sequence, which the two convolutions share, are a state of the layer beside the mixer's (they are carried in float32
+    from step to step).  A layer may have no feed-forward (and then no convolution for it)."""
+
+    ROLES = {"mixer": "mixer", "feed_forward": "feed_forward", "norm": "norm", "mixer_conv": "input_conv",
+             "feed_forward_conv": "input_conv"}
+    OPTIONAL = ("feed_forward", "feed_forward_conv")
+
+    def __init__(self, **parts):
+        super().__init__(**parts)
+        if (self.feed_forward is None) != (self.feed_forward_conv is None):
+            raise ValueError("parallel_shared_norm_conv: a feed-forward comes with its convolution, and the convolution with it")
+        if self.feed_forward_conv is not None and self.feed_forward_conv.taps != self.mixer_conv.taps:
+            raise ValueError("parallel_shared_norm_conv: the two convolutions share their carried inputs and have equally many taps")
+
+    def cache_request(self, mixer_request):
+        return mixer_request, StateRequest((self.mixer_conv.taps - 1, self.mixer_conv.hidden_size), torch.float32)
+
+    def forward(self, residual, ctx, cache_layer, writes_cache):
+        if not writes_cache:
+            raise ValueError("a convolution's carried inputs have one writer: a layer cannot read another layer's")
+        mixer_cache, carried = cache_layer.parts
+        shape = (residual.shape[0], residual.shape[1])
+        mixer_in = ctx.buffer("normed", shape, ctx.dtype)
+        ff_in = ctx.buffer("normed_ff", shape, ctx.dtype) if self.feed_forward is not None else None
+        self.mixer_conv.run(residual, self.norm, self.mixer_conv, self.feed_forward_conv, carried.state, mixer_in, ff_in, ctx)
+        self.mixer.forward(mixer_in, residual, ctx, mixer_cache, writes_cache)
+        if self.feed_forward is not None:
+            self.feed_forward.forward(ff_in, residual, ctx)
 
 
 @register("arrangement", "pre_post_norm")

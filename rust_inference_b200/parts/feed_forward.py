@@ -1,7 +1,7 @@
 """Feed-forwards without biases: SwiGLU (mlp.rs:31-46), down( silu(gate x) * (up x) ), the same with another gate
 activation and a factor on the result (`gated_dense`), the bounded gated
 form down( g sigmoid(alpha g) (u + shift) ) with g = min(gate x, limit), u = clamp(up x, -limit, limit), and the
-ungated form down( act(up x) ) with a learned activation."""
+ungated form down( act(up x) ) with a learned activation or the square of relu."""
 from __future__ import annotations
 
 import torch
@@ -129,10 +129,11 @@ class GatedDense(FeedForward):
 class DenseActivation(FeedForward):
     """out = W_down act(W_up x), no gate.  `activation` "xielu": with the two learned numbers p, q of the tensor `act`,
     act(z) = softplus(p) z^2 + z / 2 for z > 0 and (1/2 + softplus(q)) (e^z - 1 - z) + z / 2 otherwise, applied to
-    the up projection's float32 accumulators in that product's epilogue; p and q are read on the device.  `names`: up, down, act below the prefix."""
+    the up projection's float32 accumulators in that product's epilogue; p and q are read on the device.  "relu_squared":
+    act(z) = max(z, 0)^2 in the same epilogue, without a tensor of its own.  `names`: up, down, act below the prefix."""
 
     _NAMES = {"up": "up_proj.weight", "down": "down_proj.weight", "act": "act"}
-    ACTIVATIONS = ("xielu",)
+    ACTIVATIONS = ("xielu", "relu_squared")
 
     def __init__(self, *, intermediate_size: int, activation: str = "xielu", names: dict | None = None,
                  hidden_size: int, dtype, device):
@@ -141,20 +142,29 @@ class DenseActivation(FeedForward):
             raise ValueError(f"dense_act: unknown activation {activation!r}; known: {', '.join(self.ACTIVATIONS)}")
         self.intermediate_size, self.activation = int(intermediate_size), activation
         self.names = dict(self._NAMES, **(names or {}))
-        self.w_up = self.w_down = self.act = None
+        self.w_up = self.w_down = self.act = None          # act: the epilogue's four constants
 
     def tensor_specs(self):
         i, h, nm = self.intermediate_size, self.hidden_size, self.names
-        return {nm["up"]: TensorSpec((i, h)), nm["down"]: TensorSpec((h, i)), nm["act"]: TensorSpec((2,), role="vector")}
+        specs = {nm["up"]: TensorSpec((i, h)), nm["down"]: TensorSpec((h, i))}
+        if self.activation == "xielu":
+            specs[nm["act"]] = TensorSpec((2,), role="vector")
+        return specs
 
     def set_tensors(self, tensors):
         nm = self.names
         self.w_up, self.w_down = linear.Weight(tensors[nm["up"]]), linear.Weight(tensors[nm["down"]])
-        self.act = tensors[nm["act"]].contiguous()
+        if self.activation == "xielu":
+            self.act = ops.whole_act_form(tensors[nm["act"]]).contiguous()
+        else:
+            self.act = torch.tensor(ops.RELU_SQUARED_FORM, dtype=torch.float32, device=self.device)
 
     def get_tensors(self):
         nm = self.names
-        return {nm["up"]: self.w_up.t, nm["down"]: self.w_down.t, nm["act"]: self.act}
+        out = {nm["up"]: self.w_up.t, nm["down"]: self.w_down.t}
+        if self.activation == "xielu":
+            out[nm["act"]] = self.act[:2]
+        return out
 
     def forward(self, x, residual, ctx):
         act = ctx.buffer("ffn_act", (x.shape[0], self.intermediate_size), self.dtype)

@@ -1,11 +1,12 @@
 """The output head: final norm, then logits = W h in float32, on the wanted rows only
 (transformer.rs:89, :97).  The matrix is the embedding's when the model ties them: the same
-storage, where the reference clones it (model.rs:221-226).  `softcap` > 0: logits <- softcap * tanh(logits / softcap)."""
+storage, where the reference clones it (model.rs:221-226).  `scale`: logits = scale * W h (with the final norm where that can
+take the factor, otherwise on the logits).  `softcap` > 0: logits <- softcap * tanh(logits / softcap)."""
 from __future__ import annotations
 
 import torch
 
-from ..kernels import linear
+from ..kernels import linear, ops
 from .base import Head
 from .registry import lookup, register
 from .spec import PartSpec, TensorSpec
@@ -14,11 +15,12 @@ from .spec import PartSpec, TensorSpec
 @register("head", "linear_head")
 class LinearHead(Head):
     def __init__(self, *, vocab_size: int, norm: PartSpec, tied: bool, weight_prefix: str | None = "lm_head.",
-                 weight_name: str = "weight", softcap: float = 0.0, hidden_size: int, dtype, device):
+                 weight_name: str = "weight", softcap: float = 0.0, scale: float = 1.0, hidden_size: int, dtype, device):
         super().__init__(hidden_size=hidden_size, dtype=dtype, device=device)
         self.vocab_size = vocab_size
         self.wants_tie = bool(tied)
         self.softcap = float(softcap or 0.0)
+        self.scale = float(scale)
         if self.softcap < 0:
             raise ValueError(f"a cap on the logits is not negative, found {softcap}")
         self.weight_prefix = weight_prefix
@@ -62,11 +64,16 @@ class LinearHead(Head):
 
     def forward(self, residual, ctx, logits_out=None):
         normed = ctx.buffer("head_in", (ctx.n_logit_rows, self.hidden_size), self.dtype)
-        self.norm.forward(residual, normed, rows=ctx.logit_rows)
+        with_norm = self.scale != 1.0 and hasattr(self.norm, "forward_times")
+        if with_norm:
+            self.norm.forward_times(self.scale, residual, normed, rows=ctx.logit_rows)
+        else:
+            self.norm.forward(residual, normed, rows=ctx.logit_rows)
         if logits_out is None:
             logits_out = torch.empty((ctx.n_logit_rows, self.vocab_size), dtype=torch.float32, device=residual.device)
         linear.logits(normed, self.weight, logits_out, ctx)
+        if self.scale != 1.0 and not with_norm:
+            ops.scale_(logits_out, self.scale)
         if self.softcap:
-            from ..kernels import ops
             ops.softcap_(logits_out, self.softcap)
         return logits_out

@@ -23,7 +23,7 @@ class RMSNorm(Norm):
         self.eps = float(eps)
         self.unit_offset = bool(unit_offset)
         self.weight_name = weight_name
-        self.weight = self.factor = None
+        self.weight = self.factor = self._times = None
 
     def tensor_specs(self):
         return {self.weight_name: TensorSpec((self.hidden_size,), role="vector",
@@ -32,12 +32,19 @@ class RMSNorm(Norm):
     def set_tensors(self, tensors):
         self.weight = tensors[self.weight_name]
         self.factor = self.weight + 1.0 if self.unit_offset else self.weight
+        self._times = None
 
     def get_tensors(self):
         return {self.weight_name: self.weight}
 
     def forward(self, x, out, rows=None):
         return ops.rmsnorm(x, self.factor, self.eps, out, rows)
+
+    def forward_times(self, factor: float, x, out, rows=None):
+        """`forward` with the result times a number: it multiplies the weight in float32, once."""
+        if self._times is None or self._times[0] != factor:
+            self._times = (factor, self.factor * factor)
+        return ops.rmsnorm(x, self._times[1], self.eps, out, rows)
 
     # up to so many rows two norms of the same stream run as one kernel (a launch costs more than the rows)
     PAIR_MAX_ROWS = 128

@@ -20,7 +20,7 @@ class ParallelMixers(Mixer):
     `member_norm` = {"eps": e, "weight_name": name}: every member's result is RMS-normed over the model width with a
     plain weight of its own (the tensor `name` below the member's prefix) before it is scaled and added:
     residual += sum_m scale_m * rmsnorm(mixer_m(x)) * w_m.  A member then writes into a zeroed float32 buffer of its
-    own, and one kernel norms and adds all of them."""
+    own, and one kernel norms and adds all of them (with the output bias of a member that can hand it over)."""
 
     def __init__(self, *, members, member_norm: dict | None = None, hidden_size: int, dtype, device):
         super().__init__(hidden_size=hidden_size, dtype=dtype, device=device)
@@ -35,6 +35,8 @@ class ParallelMixers(Mixer):
             inner_scale = 1.0 if self.member_norm is not None else float(scale)     # a norm would undo a factor before it
             part = lookup("mixer", spec.kind)(hidden_size=hidden_size, dtype=dtype, device=device,
                                               **dict(spec.params, out_scale=inner_scale))
+            if self.member_norm is not None and getattr(part, "o_bias", False):
+                part.hands_over_bias = True
             self.members.append((spec.prefix, part))
             self.scales.append(float(scale))
         if not self.members:
@@ -84,5 +86,5 @@ class ParallelMixers(Mixer):
         for m, ((_, part), sub) in enumerate(zip(self.members, cache_layer.parts)):
             own = ctx.zeroed_buffer(f"member_result_{m}", tuple(residual.shape), torch.float32)
             part.forward(x, own, ctx, sub, writes_cache)
-            joined.append((own, None, self.norm_weights[m], self.scales[m]))
+            joined.append((own, part.b_o if getattr(part, "hands_over_bias", False) else None, self.norm_weights[m], self.scales[m]))
         ops.normed_sum(joined, residual, self.member_norm["eps"], accumulate=True)

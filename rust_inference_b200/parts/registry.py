@@ -13,13 +13,14 @@ Interfaces (see `parts.base`):
   embedding         Embedding (token ids -> hidden stream)
   head              Head (hidden stream -> logits)
   depth             DepthMix (what a layer hands on, as a function of the results of all layers so far)
+  input_conv        a short convolution in front of a sublayer (wired and run by an arrangement)
   stream            StreamStep (something that happens to the whole stream between layer runs the schedule names)
 """
 from __future__ import annotations
 
 _REGISTRIES: dict[str, dict] = {
     "norm": {}, "position": {}, "mixer": {}, "feed_forward": {}, "arrangement": {}, "embedding": {}, "head": {},
-    "depth": {}, "stream": {},
+    "depth": {}, "stream": {}, "input_conv": {},
 }
 
 
@@ -59,3 +60,4 @@ def _ensure_builtin() -> None:
     from . import recurrence, parallel_mixer, routed_experts, latent_attention  # noqa: F401
     from . import depth, state_space, delta_rule  # noqa: F401
     from . import linear_attention, loop  # noqa: F401
+    from . import input_conv, fixed_decay_attention  # noqa: F401

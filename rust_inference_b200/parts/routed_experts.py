@@ -25,7 +25,8 @@ class RoutedExperts(FeedForward):
     weight); `expert_form` / `shared_form` (a dict with limit and optionally alpha, shift: the bounded gate
     g' sigmoid(alpha g') (u' + shift) of `bounded_glu` instead of SiLU); `shared_gate` False (the shared expert has no
     learned gate and is added as it is); `out_scale` (a factor on the part's whole result, applied in float32 as it
-    joins the stream).
+    joins the stream); `correction` False (no such tensor: the scores rank the experts by themselves); `group_score` "max" (a
+    group is ranked by its largest c alone instead of the sum of its two largest).
 
     Everything from the router to the sum runs on the device (`csrc/moe.cu`), so decode steps stay
     inside captured graphs.  Experts are kept stacked: gate, up [experts, ff, hidden], down [experts,
@@ -37,15 +38,19 @@ class RoutedExperts(FeedForward):
               "shared_down": "shared.down_proj.weight", "shared_mix": "shared.mix.weight"}
 
     ROUTERS = ("sigmoid", "softmax")
+    GROUP_SCORES = ("top2_sum", "max")
 
     def __init__(self, *, n_experts: int, top: int, expert_size: int, n_groups: int = 1, group_keep: int = 1,
                  shared_size: int | None = None, names: dict | None = None, router_kind: str = "sigmoid",
                  normalise: bool = True, identity: int = 0, expert_form: dict | None = None,
                  shared_form: dict | None = None, shared_gate: bool = True, out_scale: float = 1.0,
-                 hidden_size: int, dtype, device):
+                 correction: bool = True, group_score: str = "top2_sum", hidden_size: int, dtype, device):
         super().__init__(hidden_size=hidden_size, dtype=dtype, device=device)
         if router_kind not in self.ROUTERS:
             raise ValueError(f"routed_experts: unknown router {router_kind!r}; known: {', '.join(self.ROUTERS)}")
+        if group_score not in self.GROUP_SCORES:
+            raise ValueError(f"routed_experts: unknown group score {group_score!r}; known: {', '.join(self.GROUP_SCORES)}")
+        self.has_correction, self.group_max = bool(correction), group_score == "max"
         if identity < 0 or (identity and n_groups != 1):
             raise ValueError(f"{identity} experts without tensors (not negative; not combined with groups)")
         if not 0 < top <= n_experts + identity:
@@ -79,8 +84,9 @@ class RoutedExperts(FeedForward):
     def tensor_specs(self):
         h, f, nm = self.hidden_size, self.expert_size, self.names
         outputs = self.n_experts + self.identity
-        specs = {nm["router"]: TensorSpec((outputs, h), role="vector"),
-                 nm["correction"]: TensorSpec((outputs,), role="vector", init="zeros")}
+        specs = {nm["router"]: TensorSpec((outputs, h), role="vector")}
+        if self.has_correction:
+            specs[nm["correction"]] = TensorSpec((outputs,), role="vector", init="zeros")
         for e in range(self.n_experts):
             specs[nm["gate"].format(e=e)] = TensorSpec((f, h))
             specs[nm["up"].format(e=e)] = TensorSpec((f, h))
@@ -97,7 +103,7 @@ class RoutedExperts(FeedForward):
     def set_tensors(self, tensors):
         nm, n = self.names, self.n_experts
         self.router = tensors[nm["router"]].contiguous()
-        self.correction = tensors[nm["correction"]].contiguous()
+        self.correction = tensors[nm["correction"]].contiguous() if self.has_correction else None
         self.w_gate = torch.stack([tensors[nm["gate"].format(e=e)] for e in range(n)]).contiguous()
         self.w_up = torch.stack([tensors[nm["up"].format(e=e)] for e in range(n)]).contiguous()
         self.w_down = torch.stack([tensors[nm["down"].format(e=e)] for e in range(n)]).contiguous()
@@ -108,7 +114,9 @@ class RoutedExperts(FeedForward):
 
     def get_tensors(self):
         nm = self.names
-        out = {nm["router"]: self.router, nm["correction"]: self.correction}
+        out = {nm["router"]: self.router}
+        if self.has_correction:
+            out[nm["correction"]] = self.correction
         for e in range(self.n_experts):
             out[nm["gate"].format(e=e)] = self.w_gate[e]
             out[nm["up"].format(e=e)] = self.w_up[e]
@@ -155,7 +163,7 @@ class RoutedExperts(FeedForward):
         cut = self.route_cut(n, ctx)
         ops.moe_route(x, self.router, self.correction, ids, weights, top=top, groups=self.n_groups,
                       keep=self.group_keep, gate_weight=self.shared_mix, gate_out=gate,
-                      softmax=self.router_kind == "softmax", normalise=self.normalise, **cut)
+                      softmax=self.router_kind == "softmax", normalise=self.normalise, group_max=self.group_max, **cut)
         fast = self._on_tensor_cores(x)
         if fast:
             from ..kernels import tcgen05

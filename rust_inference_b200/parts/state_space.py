@@ -94,7 +94,8 @@ class SelectiveStateSpace(Mixer):
         ops.scan_prepare(z, conv_col=self.inner, conv_ch=self.conv_ch, taps=self.w_conv, conv_bias=self.b_conv,
                          conv_state=carried.state, unit_heads=0, unit_dim=0, scaled_heads=0, unit_scale=1.0, heads=H,
                          decay_col=2 * self.inner + 2 * gn, step_col=-1, a_log=self.a_log, dt_bias=self.dt_bias, out=u,
-                         cu_seqlens=ctx.cu_seqlens, token_seq=ctx.token_seq, seq_slot=ctx.seq_slot, n_seqs=ctx.n_seqs)
+                         cu_seqlens=ctx.cu_seqlens, token_seq=ctx.token_seq, seq_slot=ctx.seq_slot, n_seqs=ctx.n_seqs,
+                         longest_run=ctx.max_new)
         y = ctx.buffer("scan_o", (n, self.inner), torch.float32)
         piece, max_pieces = ops.scan_pieces(ctx.max_new, ctx.n_seqs * H * -(-self.v_head_dim // 16))
         pieces = {}
