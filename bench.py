@@ -6,6 +6,7 @@
     python bench.py --arch vadodra [--arch-sizes 1k|2k|4k]     (likewise)
     python bench.py --arch redodra [--arch-sizes 1k|2k|4k]     (likewise, beside a Lulisun-style model too)
     python bench.py --arch belizen [--arch-sizes 1k|2k|4k]     (likewise)
+    python bench.py --arch gatarax [--arch-sizes 1k|2k|4k]     (likewise)
 
 Default run: a Qwen2.5-7B-sized dense decoder (28 layers, hidden 3584, 28 heads, 4 kv
 heads, head_dim 128, intermediate 18944, vocabulary 152064, q/k/v biases, untied head)
@@ -201,10 +202,10 @@ def main() -> int:
     ap.add_argument("--tokens", type=int, default=8, help="with --kernel: tokens in the step")
     ap.add_argument("--context", type=int, default=1024, help="with --kernel: cached positions per sequence")
     ap.add_argument("--once", action="store_true", help="with --kernel: launch the workload once, untimed (for ncu)")
-    ap.add_argument("--arch", default="dense", choices=["dense", "lulisun", "vadodra", "redodra", "belizen"],
-                    help="lulisun / vadodra / redodra: prefill and decode throughput of a model of that design beside a dense decoder of "
+    ap.add_argument("--arch", default="dense", choices=["dense", "lulisun", "vadodra", "redodra", "belizen", "gatarax"],
+                    help="lulisun / vadodra / redodra / belizen / gatarax: prefill and decode throughput of a model of that design beside a dense decoder of "
                          "equal size, kernel by kernel against the rooflines, instead of the default workload")
-    ap.add_argument("--arch-sizes", default="2k", choices=["1k", "2k", "4k"], help="with --arch lulisun / vadodra / redodra / belizen: the layer sizes")
+    ap.add_argument("--arch-sizes", default="2k", choices=["1k", "2k", "4k"], help="with --arch lulisun / vadodra / redodra / belizen / gatarax: the layer sizes")
     args = ap.parse_args()
 
     if args.impl == "reference":
@@ -241,6 +242,12 @@ def main() -> int:
         from rust_inference_b200.kernels import belizen_bench
         peaks, peak_source = load_peaks()
         return belizen_bench.main(args.arch_sizes, peaks, peak_source, prefill_tokens=max(1, args.prefill_tokens),
+                                  batch=args.batch, context=args.context if args.context != 1024 else None,
+                                  steps=max(1, min(args.steps, 64)))
+    if args.arch == "gatarax":
+        from rust_inference_b200.kernels import gatarax_bench
+        peaks, peak_source = load_peaks()
+        return gatarax_bench.main(args.arch_sizes, peaks, peak_source, prefill_tokens=max(1, args.prefill_tokens),
                                   batch=args.batch, context=args.context if args.context != 1024 else None,
                                   steps=max(1, min(args.steps, 64)))
     warmup = max(3, args.warmup)

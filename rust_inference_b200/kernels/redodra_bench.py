@@ -118,7 +118,7 @@ def time_parts(engine, s: dict, lens_before: list, new_tokens: int, peaks: dict,
         u = torch.empty(n, part.conv_ch + 2 * H, dtype=f32, device=dev)
         ms = timer(lambda: ops.scan_prepare(z, conv_ch=part.conv_ch, taps=part.w_conv, conv_state=carried.state, heads=H, a_log=part.a_log,
                                             dt_bias=part.dt_bias, out=u, cu_seqlens=ctx.cu_seqlens, token_seq=ctx.token_seq,
-                                            seq_slot=ctx.seq_slot, n_seqs=ctx.n_seqs, **prepare_kw))
+                                            seq_slot=ctx.seq_slot, n_seqs=ctx.n_seqs, longest_run=ctx.max_new, **prepare_kw))
         row(tag + "_prepare", ms, 0.0, n * (part.conv_ch * 8 + 4 * H * 4) + 2 * B * carried.state[0].numel() * 4)
         o = torch.empty(n, H * vdim, dtype=f32, device=dev)
         piece, max_pieces = (0, 1) if delta else ops.scan_pieces(ctx.max_new, ctx.n_seqs * H * -(-vdim // 16))     # as the part calls it

@@ -67,10 +67,19 @@ class FixedDecayLinearAttention(Mixer):
     def forward(self, x, residual, ctx, cache_layer, writes_cache):
         if not writes_cache:
             raise ValueError("a recurrent state has one writer: a layer cannot read another layer's state")
-        n, H = x.shape[0], self.n_heads
+        n = x.shape[0]
         z = ctx.buffer("scan_z", (n, self.width), torch.float32)
         linear.logits(x, self.w_in, z, ctx, silu_cols=self.activated)
         o = ctx.buffer("scan_o", (n, self.v_dim), torch.float32)
+        self.scan(z, cache_layer, o, ctx)
+        normed = ctx.buffer("scan_normed", (n, self.v_dim), self.dtype)
+        ops.gated_group_norm(o, z, self.gate_col, self.norm, normed, groups=1, group_size=self.v_dim, gate_first=False,
+                             gate_act="sigmoid", eps=self.eps, out_scale=self.out_scale)
+        linear.into_residual(normed, self.w_o, residual, ctx)
+
+    def scan(self, z, cache_layer, o, ctx):
+        """The recurrence over the step's tokens: o (float32 [T, heads * v_head_dim]) from the activated projection z."""
+        H = self.n_heads
         piece, max_pieces = ops.scan_pieces(ctx.max_new, ctx.n_seqs * H * -(-self.v_head_dim // 16))
         pieces = {}
         if piece:                      # a long run of new tokens: its pieces side by side, from zero and again from their start states
@@ -80,7 +89,3 @@ class FixedDecayLinearAttention(Mixer):
         ops.state_scan(z, cache_layer.state, o, ctx.cu_seqlens, ctx.seq_slot, n_seqs=ctx.n_seqs, heads=H, groups=H,
                        dim=self.head_dim, vdim=self.v_head_dim, q_col=0, k_col=self.qk_dim, v_col=2 * self.qk_dim, decay_col=0,
                        step_col=0, delta=False, decay=self.decays, longest_run=ctx.max_new, **pieces)
-        normed = ctx.buffer("scan_normed", (n, self.v_dim), self.dtype)
-        ops.gated_group_norm(o, z, self.gate_col, self.norm, normed, groups=1, group_size=self.v_dim, gate_first=False,
-                             gate_act="sigmoid", eps=self.eps, out_scale=self.out_scale)
-        linear.into_residual(normed, self.w_o, residual, ctx)
