@@ -346,6 +346,7 @@ cudaError_t launch_input(const InputConv& p, cudaStream_t stream) {
 template <typename T>
 cudaError_t dispatch_input(const InputConv& p, bool vec, cudaStream_t stream) {
     if (p.n_tokens < 512) return vec ? launch_input<T, 4, 1>(p, stream) : launch_input<T, 1, 1>(p, stream);
+    if (p.n_tokens < 4096) return vec ? launch_input<T, 4, 4>(p, stream) : launch_input<T, 1, 4>(p, stream);
     return vec ? launch_input<T, 4, MAX_TOKENS>(p, stream) : launch_input<T, 1, MAX_TOKENS>(p, stream);
 }
 
@@ -383,7 +384,7 @@ RI_API int ri_input_conv(const float* x, const float* w, float eps, const float*
     return 0;
 }
 
-// z: float32 [n_tokens, ld] with q_dim query channels, then n_kv_heads * hd key and n_kv_heads * v_hd value channels.  bias
+// z: float32 rows, ld apart, with q_dim query channels, then n_kv_heads * hd key and n_kv_heads * v_hd value channels.  bias
 // (float32, all channels, or null) is added before the convolution and is part of the carried inputs.  q_out [n_tokens,
 // q_dim] and the caches ([pages, n_kv_heads, page_size, hd] / [.., v_hd]) in `dtype`.
 RI_API int ri_conv_store(const float* z, int ld, const float* bias, const float* taps, int k_taps, float* carried, void* q_out,

@@ -40,6 +40,19 @@ __device__ __forceinline__ float sigmoid_f32(float x) {
     return e / (1.f + e);
 }
 
+// V consecutive floats as one access (V = 4: 16 bytes; the address must allow it).
+template <int V> struct Floats { float v[V]; };
+template <int V> __device__ __forceinline__ Floats<V> load_floats(const float* p) {
+    Floats<V> r;
+    if constexpr (V == 4) {
+        const float4 t = *reinterpret_cast<const float4*>(p);
+        r.v[0] = t.x; r.v[1] = t.y; r.v[2] = t.z; r.v[3] = t.w;
+    } else {
+        r.v[0] = *p;
+    }
+    return r;
+}
+
 struct Prepare {
     const float* z;            // [tokens, ld] the projection's results
     int ld;
@@ -75,6 +88,7 @@ struct Prepare {
     const void* gate_w2;
     float* gate_out;           // [tokens, gate_channels]
     int w2_bf16;
+    int n_tokens;
 };
 
 constexpr int CHANNEL_TILE = 256;
@@ -181,6 +195,89 @@ __global__ void __launch_bounds__(256) scan_prepare_kernel(Prepare p) {
         }
 }
 
+// The same for steps of many tokens: a block takes PREP_TOKENS consecutive tokens and p.tile_ch convolved channels.  A thread
+// owns V neighbouring channels, keeps their filters in registers and walks down the tokens (a row it looks back at is one
+// it has just read); channels that are made unit vectors go through shared memory, the rest straight out.  Further tiles
+// turn the low-rank products in `raw` into decays.
+constexpr int PREP_TOKENS = 8;
+template <int V, int KT>
+__global__ void __launch_bounds__(256) scan_prepare_rows_kernel(Prepare p) {
+    extern __shared__ float ch[];                 // [PREP_TOKENS][tile_ch]
+    const int t0 = blockIdx.x * PREP_TOKENS, t1 = min(p.n_tokens, t0 + PREP_TOKENS);
+    let_next_kernel_start();
+    if ((int)blockIdx.y >= p.conv_tiles) {
+        const int c = ((int)blockIdx.y - p.conv_tiles) * CHANNEL_TILE + (int)threadIdx.x;
+        const bool mine = c < p.channels;
+        const float rate = mine ? -expf(p.a_log[c / p.head_dim]) : 0.f, bias = mine ? p.dt_bias[c] : 0.f;
+        wait_for_previous_kernels();
+        if (!mine) return;
+        for (int t = t0; t < t1; ++t) p.decay[(size_t)t * p.channels + c] = expf(rate * softplus_f32(p.raw[(size_t)t * p.channels + c] + bias));
+        return;
+    }
+    const int c0 = blockIdx.y * p.tile_ch, c1 = min(p.conv_ch, c0 + p.tile_ch);
+    const int K = KT > 0 ? KT : p.k_taps, unit_end = p.unit_heads * p.unit_dim;
+    wait_for_previous_kernels();
+    for (int c = c0 + (int)threadIdx.x * V; c < c1; c += blockDim.x * V) {
+        float f[KT > 0 ? KT * V : 1];
+        if constexpr (KT > 0) {
+#pragma unroll
+            for (int i = 0; i < KT * V; ++i) f[i] = p.taps[(size_t)c * KT + i];
+        }
+        float bias[V];
+#pragma unroll
+        for (int k = 0; k < V; ++k) bias[k] = p.conv_bias != nullptr ? p.conv_bias[c + k] : 0.f;
+        for (int t = t0; t < t1; ++t) {
+            const int b = p.token_seq[t];
+            const int i = t - p.cu_seqlens[b];
+            int slot = p.seq_slot[b];
+            if (!RI_IN_LIMIT(slot, RI_LIMIT_SLOTS, RI_CHECK_SLOT)) slot = 0;
+            const float* carried = p.conv_state + (size_t)slot * (K - 1) * p.conv_ch + c;
+            float acc[V];
+#pragma unroll
+            for (int k = 0; k < V; ++k) acc[k] = bias[k];
+#pragma unroll
+            for (int j = 0; j < K; ++j) {         // the input j tokens back
+                const float* src = i >= j ? p.z + (size_t)(t - j) * p.ld + p.conv_col + c : carried + (size_t)(K - 1 + i - j) * p.conv_ch;
+                const Floats<V> x = load_floats<V>(src);
+#pragma unroll
+                for (int k = 0; k < V; ++k)
+                    acc[k] = fmaf(KT > 0 ? f[KT > 0 ? k * KT + (KT - 1 - j) : 0] : p.taps[(size_t)(c + k) * K + (K - 1 - j)], x.v[k], acc[k]);
+            }
+            float* dst = c < unit_end ? ch + (t - t0) * p.tile_ch + (c - c0) : p.out + (size_t)t * p.out_ld + c;
+#pragma unroll
+            for (int k = 0; k < V; ++k) acc[k] = silu_f32(acc[k]);
+            if constexpr (V == 4) *reinterpret_cast<float4*>(dst) = make_float4(acc[0], acc[1], acc[2], acc[3]);
+            else *dst = acc[0];
+        }
+    }
+    if (c0 < unit_end) {
+        __syncthreads();
+        const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+        const int h0 = c0 / p.unit_dim, heads = min(p.unit_heads, c1 / p.unit_dim) - h0;         // tiles are multiples of unit_dim there
+        for (int it = warp; it < heads * (t1 - t0); it += warps) {
+            const int tk = it / heads, h = h0 + it % heads;
+            const float* v = ch + tk * p.tile_ch + (h - h0) * p.unit_dim;
+            float ss = 0.f;
+            for (int d = lane; d < p.unit_dim; d += 32) ss = fmaf(v[d], v[d], ss);
+            ss = warp_sum(ss);
+            const float f = (h < p.scaled_heads ? p.unit_scale : 1.f) / sqrtf(ss + 1e-6f);
+            float* dst = p.out + (size_t)(t0 + tk) * p.out_ld + h * p.unit_dim;
+            for (int d = lane; d < p.unit_dim; d += 32) dst[d] = v[d] * f;
+        }
+    }
+    if (blockIdx.y == 0)
+        for (int it = threadIdx.x; it < (t1 - t0) * p.heads; it += blockDim.x) {
+            const int t = t0 + it / p.heads, h = it % p.heads;
+            float* out = p.out + (size_t)t * p.out_ld + p.conv_ch;
+            float dt = 0.f;
+            if (p.channels == 0) {
+                dt = softplus_f32(p.z[(size_t)t * p.ld + p.decay_col + h] + p.dt_bias[h]);
+                out[h] = expf(-expf(p.a_log[h]) * dt);
+            }
+            out[p.heads + h] = p.step_col >= 0 ? sigmoid_f32(p.z[(size_t)t * p.ld + p.step_col + h]) : dt;
+        }
+}
+
 __global__ void conv_state_kernel(const float* z, int ld, int conv_col, int conv_ch, int k_taps, float* conv_state,
                                   const int* cu_seqlens, const int* seq_slot) {
     let_next_kernel_start();
@@ -273,7 +370,9 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(Scan p) {
     float s[ROWS];
 #pragma unroll
     for (int k = 0; k < ROWS; ++k) s[k] = (MODE != LOCAL && live && i0 + k < p.dim) ? S[(size_t)(i0 + k) * p.vdim + j] : 0.f;
-    float decays = 1.f;
+    float decays = 1.f, v_before = 0.f, q_before[ROWS];
+#pragma unroll
+    for (int k = 0; k < ROWS; ++k) q_before[k] = 0.f;
     const float fixed = DECAY == FIXED ? p.decay[h] : 1.f;
     const int g = h / (p.heads / p.groups);
     const int q_off = p.q_col + g * p.dim, k_off = p.k_col + g * p.dim, v_off = p.v_col + h * p.vdim + j0;
@@ -334,63 +433,76 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(Scan p) {
         }
         __syncthreads();
         const float* cur = tile + buf * tile_floats;
-        // unrolled: only the state's update chains the tokens, so the loads and the read-out's sums of one token overlap
-        // the next token's update
+        // Only the state chains the tokens.  What a token reads of the state before its own update (the delta rule's
+        // S^T k) and the read-out of the token before (which wants the state after that one's update) are sums over the same
+        // values, so they are formed together and their shuffles overlap; S^T k of the decayed state is taken as S^T (a k).
+        // Unrolled, a token's loads overlap the token before.
 #pragma unroll(DELTA ? 2 : 4)
         for (int tok = 0; tok < n_tok; ++tok) {
             const float* base = cur + tok * TOKEN;
             const float4* k4 = reinterpret_cast<const float4*>(base + r * SLICE);
             const float4* q4 = reinterpret_cast<const float4*>(base + R * SLICE + r * SLICE);
+            const float4* a4 = reinterpret_cast<const float4*>(base + 2 * R * SLICE + r * SLICE);      // CHANNELS only
             const float v = base[V_AT + jj];
             const float a = DECAY == FIXED ? fixed : DECAY == CHANNELS ? 1.f : base[V_AT + COLS];
             const float step = DECAY == FIXED ? 1.f : base[V_AT + COLS + 1];
-            float kk[ROWS], qq[ROWS];
+            float kk[ROWS], qq[ROWS], aa[ROWS];
 #pragma unroll
             for (int k = 0; k < ROWS / 4; ++k) {
-                const float4 kv = k4[k], qv = q4[k];
+                const float4 kv = k4[k];
                 kk[4 * k] = kv.x; kk[4 * k + 1] = kv.y; kk[4 * k + 2] = kv.z; kk[4 * k + 3] = kv.w;
-                qq[4 * k] = qv.x; qq[4 * k + 1] = qv.y; qq[4 * k + 2] = qv.z; qq[4 * k + 3] = qv.w;
-            }
-            float write = step * v;
-            if (MODE == LOCAL) decays *= a;
-            if (DELTA) {
-                float d0 = 0.f, d1 = 0.f;
+                if (MODE != LOCAL) {
+                    const float4 qv = q4[k];
+                    qq[4 * k] = qv.x; qq[4 * k + 1] = qv.y; qq[4 * k + 2] = qv.z; qq[4 * k + 3] = qv.w;
+                }
                 if (DECAY == CHANNELS) {
-                    const float4* a4 = reinterpret_cast<const float4*>(base + 2 * R * SLICE + r * SLICE);
-#pragma unroll
-                    for (int k = 0; k < ROWS / 4; ++k) {
-                        const float4 av = a4[k];
-                        s[4 * k] *= av.x; s[4 * k + 1] *= av.y; s[4 * k + 2] *= av.z; s[4 * k + 3] *= av.w;
-                    }
+                    const float4 av = a4[k];
+                    aa[4 * k] = av.x; aa[4 * k + 1] = av.y; aa[4 * k + 2] = av.z; aa[4 * k + 3] = av.w;
                 }
-#pragma unroll
-                for (int k = 0; k < ROWS; k += 2) {
-                    if (DECAY != CHANNELS) {
-                        s[k] *= a;
-                        s[k + 1] *= a;
-                    }
-                    d0 = fmaf(s[k], kk[k], d0);
-                    d1 = fmaf(s[k + 1], kk[k + 1], d1);
-                }
-                float dot = d0 + d1;
-#pragma unroll
-                for (int o = R / 2; o > 0; o >>= 1) dot += __shfl_xor_sync(0xffffffffu, dot, o);
-                write = step * (v - dot);
             }
-            float a0 = 0.f, a1 = 0.f;
+            if (MODE == LOCAL) decays *= a;
+            float d0 = 0.f, d1 = 0.f, e0 = 0.f, e1 = 0.f;
 #pragma unroll
             for (int k = 0; k < ROWS; k += 2) {
-                s[k] = DELTA ? fmaf(kk[k], write, s[k]) : fmaf(a, s[k], kk[k] * write);
-                s[k + 1] = DELTA ? fmaf(kk[k + 1], write, s[k + 1]) : fmaf(a, s[k + 1], kk[k + 1] * write);
-                a0 = fmaf(s[k], qq[k], a0);
-                a1 = fmaf(s[k + 1], qq[k + 1], a1);
+                if (DELTA) {
+                    d0 = fmaf(s[k], DECAY == CHANNELS ? aa[k] * kk[k] : kk[k], d0);
+                    d1 = fmaf(s[k + 1], DECAY == CHANNELS ? aa[k + 1] * kk[k + 1] : kk[k + 1], d1);
+                }
+                if (MODE != LOCAL) {
+                    e0 = fmaf(s[k], q_before[k], e0);
+                    e1 = fmaf(s[k + 1], q_before[k + 1], e1);
+                }
             }
-            float acc = a0 + a1;
+            float dot = d0 + d1, acc = e0 + e1;
 #pragma unroll
-            for (int o = R / 2; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
-            if (MODE != LOCAL && live && r == 0) p.o[(size_t)(tb + tok) * o_ld + h * p.vdim + j] = fmaf(skip, v, acc);
+            for (int o = R / 2; o > 0; o >>= 1) {
+                if (DELTA) dot += __shfl_xor_sync(0xffffffffu, dot, o);
+                if (MODE != LOCAL) acc += __shfl_xor_sync(0xffffffffu, acc, o);
+            }
+            if (MODE != LOCAL) {
+                if (live && r == 0 && tb + tok > t0) p.o[(size_t)(tb + tok - 1) * o_ld + h * p.vdim + j] = fmaf(skip, v_before, acc);
+                v_before = v;
+            }
+            const float write = DELTA ? step * (v - (DECAY == CHANNELS ? dot : a * dot)) : step * v;
+#pragma unroll
+            for (int k = 0; k < ROWS; ++k) {
+                s[k] = fmaf(DECAY == CHANNELS ? aa[k] : a, s[k], kk[k] * write);
+                if (MODE != LOCAL) q_before[k] = qq[k];
+            }
         }
         __syncthreads();                                  // this tile may be overwritten by the fetch after next
+    }
+    if (MODE != LOCAL) {                                  // the last token's read-out
+        float e0 = 0.f, e1 = 0.f;
+#pragma unroll
+        for (int k = 0; k < ROWS; k += 2) {
+            e0 = fmaf(s[k], q_before[k], e0);
+            e1 = fmaf(s[k + 1], q_before[k + 1], e1);
+        }
+        float acc = e0 + e1;
+#pragma unroll
+        for (int o = R / 2; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
+        if (live && r == 0) p.o[(size_t)(t1 - 1) * o_ld + h * p.vdim + j] = fmaf(skip, v_before, acc);
     }
     if (MODE == FINAL) return;                            // the carry kernel left the final state in the slot
 #pragma unroll
@@ -454,9 +566,10 @@ __global__ void gated_group_norm_kernel(const float* x, int x_ld, const float* g
     }
 }
 
-// The same with a block per (token, group), for groups of many channels.
-template <typename T>
-__global__ void __launch_bounds__(256) gated_group_norm_block_kernel(const float* x, int x_ld, const float* gate, int gate_ld, int gate_col,
+// The same with a block per (token, group), for groups of many channels; V = 4: 16 bytes at a time, where rows, columns
+// and the weight's length allow.
+template <typename T, int V>
+__global__ void __launch_bounds__(1024) gated_group_norm_block_kernel(const float* x, int x_ld, const float* gate, int gate_ld, int gate_col,
                                         const float* __restrict__ w, int w_len, T* __restrict__ out, int groups,
                                         int gs, int gate_first, int sigmoid, float eps, float out_scale) {
     __shared__ float scratch[33];
@@ -465,19 +578,45 @@ __global__ void __launch_bounds__(256) gated_group_norm_block_kernel(const float
     const int t = blockIdx.x / groups, g = blockIdx.x % groups;
     const float* src = x + (size_t)t * x_ld + g * gs;
     const float* gt = gate + (size_t)t * gate_ld + gate_col + g * gs;
+    // the thread's first run of channels stays in registers; wider groups read the rest again
+    Floats<V> x0, g0;
     float ss = 0.f;
-    for (int d = threadIdx.x; d < gs; d += blockDim.x) {
-        const float v = gate_first ? src[d] * gate_f32(gt[d], sigmoid) : src[d];
-        ss = fmaf(v, v, ss);
+    for (int d = threadIdx.x * V; d < gs; d += blockDim.x * V) {
+        Floats<V> xv = load_floats<V>(src + d), gv = load_floats<V>(gt + d);
+#pragma unroll
+        for (int k = 0; k < V; ++k) {
+            gv.v[k] = gate_f32(gv.v[k], sigmoid);
+            const float v = gate_first ? xv.v[k] * gv.v[k] : xv.v[k];
+            ss = fmaf(v, v, ss);
+        }
+        if (d == (int)threadIdx.x * V) { x0 = xv; g0 = gv; }
     }
     ss = block_sum(ss, scratch);
     const float inv = out_scale / sqrtf(ss / (float)gs + eps);
     T* dst = out + ((size_t)t * groups + g) * gs;
-    for (int d = threadIdx.x; d < gs; d += blockDim.x) {
-        const float sg = gate_f32(gt[d], sigmoid);
-        const float v = gate_first ? src[d] * sg : src[d];
-        const float y = v * inv * w[(g * gs + d) % w_len];
-        dst[d] = from_f32<T>(gate_first ? y : y * sg);
+    for (int d = threadIdx.x * V; d < gs; d += blockDim.x * V) {
+        Floats<V> xv = x0, gv = g0;
+        if (d != (int)threadIdx.x * V) {
+            xv = load_floats<V>(src + d);
+            gv = load_floats<V>(gt + d);
+#pragma unroll
+            for (int k = 0; k < V; ++k) gv.v[k] = gate_f32(gv.v[k], sigmoid);
+        }
+        const Floats<V> wv = load_floats<V>(w + (g * gs + d) % w_len);
+        float y[V];
+#pragma unroll
+        for (int k = 0; k < V; ++k) y[k] = xv.v[k] * gv.v[k] * inv * wv.v[k];
+        if constexpr (V == 4 && sizeof(T) == 2) {
+            const __nv_bfloat162 lo = __floats2bfloat162_rn(y[0], y[1]), hi = __floats2bfloat162_rn(y[2], y[3]);
+            uint2 pk;
+            pk.x = *reinterpret_cast<const uint32_t*>(&lo);
+            pk.y = *reinterpret_cast<const uint32_t*>(&hi);
+            *reinterpret_cast<uint2*>(dst + d) = pk;
+        } else if constexpr (V == 4) {
+            *reinterpret_cast<float4*>(dst + d) = make_float4(y[0], y[1], y[2], y[3]);
+        } else {
+            dst[d] = from_f32<T>(y[0]);
+        }
     }
 }
 
@@ -564,8 +703,27 @@ static int scan_prepare(const float* z, int ld, int conv_col, int conv_ch, const
     Prepare p{z, ld, conv_col, conv_ch, taps, conv_bias, k_taps, conv_state, unit_heads, unit_dim, scaled_heads, unit_scale,
               heads, decay_col, step_col, a_log, dt_bias, out, out_ld, cu_seqlens, token_seq, seq_slot, tile_ch, conv_tiles, single,
               low.channels, low.head_dim, low.raw, low.decay, low.w2, low.rank, low.low_col, low.gate_channels, low.gate_rank,
-              low.gate_low_col, low.gate_w2, low.gate_out, low.w2_bf16};
-    cudaError_t e = launch_dependent(scan_prepare_kernel, dim3(n_tokens, tiles), 256, smem, stream, p);
+              low.gate_low_col, low.gate_w2, low.gate_out, low.w2_bf16, n_tokens};
+    cudaError_t e;
+    // many tokens, the low-rank maps (if any) as products: several tokens per block
+    int rows_ch = unit_heads > 0 && unit_dim > 0 ? unit_dim * ((1024 + unit_dim - 1) / unit_dim) : 1024;
+    if (rows_ch > conv_ch) rows_ch = (conv_ch + 3) / 4 * 4;
+    const size_t rows_smem = unit_heads > 0 ? (size_t)PREP_TOKENS * rows_ch * sizeof(float) : 0;
+    if (n_tokens >= 64 * PREP_TOKENS && !formed && low.gate_channels == 0 && rows_smem <= 48 * 1024) {
+        p.tile_ch = rows_ch;
+        p.conv_tiles = (conv_ch + rows_ch - 1) / rows_ch;
+        const dim3 grid((n_tokens + PREP_TOKENS - 1) / PREP_TOKENS, p.conv_tiles + (low.channels + CHANNEL_TILE - 1) / CHANNEL_TILE);
+        const bool vec = (ld | conv_col | conv_ch | out_ld | rows_ch | (unit_heads * unit_dim)) % 4 == 0 &&
+                         ((reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(conv_state)) & 15) == 0;
+#define RI_PREP(V) (k_taps == 2 ? launch_dependent(scan_prepare_rows_kernel<V, 2>, grid, 256, rows_smem, stream, p)   \
+                    : k_taps == 3 ? launch_dependent(scan_prepare_rows_kernel<V, 3>, grid, 256, rows_smem, stream, p) \
+                    : k_taps == 4 ? launch_dependent(scan_prepare_rows_kernel<V, 4>, grid, 256, rows_smem, stream, p) \
+                                  : launch_dependent(scan_prepare_rows_kernel<V, 0>, grid, 256, rows_smem, stream, p))
+        e = vec ? RI_PREP(4) : RI_PREP(1);
+#undef RI_PREP
+    } else {
+        e = launch_dependent(scan_prepare_kernel, dim3(n_tokens, tiles), 256, smem, stream, p);
+    }
     if (check_launch(e, "scan_prepare")) return 1;
     if (k_taps > 1 && !single) {
         dim3 grid((conv_ch + 127) / 128, n_seqs);
@@ -696,19 +854,23 @@ RI_API int ri_gated_group_norm(const float* x, int x_ld, const float* gate, int 
     const long long warps = (long long)n_tokens * groups;
     const int blocks = (int)((warps * 32 + 255) / 256);
     const bool wide = gs >= 512 && warps <= 0x7fffffffLL;          // a block per group instead of a warp
+    const bool vec = (gs | x_ld | gate_ld | gate_col | w_len) % 4 == 0 &&
+                     ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(w) |
+                       reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+    const int per = vec ? 4 : 1;
+    int threads = ((gs + per - 1) / per + 31) / 32 * 32;
+    threads = threads > 1024 ? 1024 : threads;
     cudaError_t e;
-    if (dtype == RI_F32)
-        e = wide ? launch_dependent(gated_group_norm_block_kernel<float>, (int)warps, 256, 0, stream, x, x_ld, gate, gate_ld, gate_col,
-                                    w, w_len, (float*)out, groups, gs, gate_first, sigmoid, eps, out_scale)
-                 : launch_dependent(gated_group_norm_kernel<float>, blocks, 256, 0, stream, x, x_ld, gate, gate_ld, gate_col, w, w_len,
-                                    (float*)out, n_tokens, groups, gs, gate_first, sigmoid, eps, out_scale);
-    else if (dtype == RI_BF16)
-        e = wide ? launch_dependent(gated_group_norm_block_kernel<__nv_bfloat16>, (int)warps, 256, 0, stream, x, x_ld, gate, gate_ld,
-                                    gate_col, w, w_len, (__nv_bfloat16*)out, groups, gs, gate_first, sigmoid, eps, out_scale)
-                 : launch_dependent(gated_group_norm_kernel<__nv_bfloat16>, blocks, 256, 0, stream, x, x_ld, gate, gate_ld, gate_col, w,
-                                    w_len, (__nv_bfloat16*)out, n_tokens, groups, gs, gate_first, sigmoid, eps, out_scale);
-    else
-        return fail("gated_group_norm: unknown dtype %d", dtype);
+#define RI_NORM_WIDE(T, V) launch_dependent(gated_group_norm_block_kernel<T, V>, (int)warps, threads, 0, stream, x, x_ld, gate, gate_ld, \
+                                            gate_col, w, w_len, (T*)out, groups, gs, gate_first, sigmoid, eps, out_scale)
+#define RI_NORM(T) (!wide ? launch_dependent(gated_group_norm_kernel<T>, blocks, 256, 0, stream, x, x_ld, gate, gate_ld, gate_col, w,   \
+                                             w_len, (T*)out, n_tokens, groups, gs, gate_first, sigmoid, eps, out_scale)                  \
+                    : vec ? RI_NORM_WIDE(T, 4) : RI_NORM_WIDE(T, 1))
+    if (dtype == RI_F32) e = RI_NORM(float);
+    else if (dtype == RI_BF16) e = RI_NORM(__nv_bfloat16);
+    else return fail("gated_group_norm: unknown dtype %d", dtype);
+#undef RI_NORM
+#undef RI_NORM_WIDE
     return check_launch(e, "gated_group_norm");
 }
 

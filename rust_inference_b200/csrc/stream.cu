@@ -10,7 +10,8 @@
 //                   every stage optional; the branch buffer is left zeroed for its next user
 //   normed_sum      out (+)= sum_m scale_m * rmsnorm(x_m + bias_m) * w_m over up to four branch buffers (the members of a
 //                   mixer made of several mixers, each normalised over the model width before they are added);
-//                   the buffers are left zeroed
+//                   the buffers are left zeroed; so is one more matrix of as many rows, if given (an accumulator that the
+//                   members have read)
 //   xielu           act(z) = a_p z^2 + z/2 for z > 0, a_n (e^z - 1 - z) + z/2 otherwise, a_p = softplus(p),
 //                   a_n = 1/2 + softplus(q), p and q read from device memory
 //   add_row_bias    x[t, :] += bias
@@ -161,6 +162,8 @@ struct NormedSum {
     const float* w[MAX_MEMBERS];
     float scale[MAX_MEMBERS];
     int members;
+    float* clear;              // [rows, clear_n] zeroed as well, or null
+    int clear_n;
 };
 
 // A block per row; the row of every member is read twice (sum of squares, then the weighted values): it stays in L1.
@@ -197,6 +200,10 @@ __global__ void __launch_bounds__(256) normed_sum_kernel(NormedSum p, float* out
             for (int k = 0; k < V; ++k) acc.v[k] = fmaf((x.v[k] + bv.v[k]) * inv[m], wv.v[k], acc.v[k]);
         }
         store_pack<V>(out + row + c, acc);
+    }
+    if (p.clear != nullptr) {
+        float* row0 = p.clear + (size_t)blockIdx.x * p.clear_n;
+        for (int c = threadIdx.x; c < p.clear_n; c += blockDim.x) row0[c] = 0.f;
     }
 }
 
@@ -281,11 +288,13 @@ RI_API int ri_stream_update(float* stream_x, float* branch, const float* branch_
 }
 
 RI_API int ri_normed_sum(float* const* xs, const float* const* biases, const float* const* ws, const float* scales, int members,
-                         float* out, int n_tokens, int n, float eps, int accumulate, cudaStream_t stream) {
+                         float* out, int n_tokens, int n, float eps, int accumulate, float* clear, int clear_n, cudaStream_t stream) {
     if (n_tokens <= 0 || n <= 0) return 0;
     if (members < 1 || members > MAX_MEMBERS) return fail("normed_sum: %d members, at most %d", members, MAX_MEMBERS);
     NormedSum p{};
     p.members = members;
+    p.clear = clear;
+    p.clear_n = clear_n;
     for (int m = 0; m < members; ++m) {
         p.x[m] = xs[m];
         p.bias[m] = biases[m];

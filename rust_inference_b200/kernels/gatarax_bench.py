@@ -82,9 +82,11 @@ def time_parts(engine, s: dict, lens_before: list, new_tokens: int, peaks: dict,
         vis += sum(min(window, p + 1) for p in range(before, before + new_tokens))
         kv_bytes += (before + new_tokens - max(0, before - window + 1)) * kv * 2 * hd * 2
     keys, proj = left_cache.parts
+    both = torch.zeros(n, par.w_in.n, device=dev)
+    project = linear.accumulate_split if linear.wants_split(x, par.w_in) else linear.logits           # as the part calls it
+    row("members_projection", timer(lambda: project(x, par.w_in, both, ctx)), 2.0 * n * par.w_in.n * width,
+        par.w_in.n * width * 2 + n * (width * 2 + par.w_in.n * 4))
     z = torch.randn(n, left.w_qkv.n, device=dev) * 0.5
-    row("left_projection", timer(lambda: linear.logits(x, left.w_qkv, z, ctx)), 2.0 * n * left.w_qkv.n * width,
-        left.w_qkv.n * width * 2 + n * (width * 2 + left.w_qkv.n * 4))
     q = torch.empty(n, left.q_dim, dtype=bf, device=dev)
     ms = timer(lambda: ops.conv_store(z, left.b_qkv, left.w_conv, proj.state, q, keys.k, keys.v, ctx.cu_seqlens, ctx.token_pos,
                                       ctx.token_seq, ctx.seq_slot, ctx.page_table, n_seqs=ctx.n_seqs, n_kv_heads=kv, head_dim=hd,
@@ -95,14 +97,12 @@ def time_parts(engine, s: dict, lens_before: list, new_tokens: int, peaks: dict,
                                               window=window, sink=left.sinks))
     row("window_attention", ms, 4.0 * hd * vis * heads, kv_bytes + n * heads * hd * 2 * 2)
     joined = [(torch.randn(n, width, device=dev), bias, w, 0.5) for w, bias in zip(par.norm_weights, (left.b_o, None))]
-    row("normed_sum", timer(lambda: ops.normed_sum(joined, residual, 1e-5, accumulate=True)), 0.0, n * width * (2 * 8 + 8))
+    row("normed_sum", timer(lambda: ops.normed_sum(joined, residual, 1e-5, accumulate=True, clear=both if project is linear.accumulate_split else None)), 0.0, n * width * (2 * 8 + 8))
 
     # ---- the delta rule with decays per key channel (right member) ----------------------------------------------------
     matrix, conv = right_cache.parts
     H, G, dim, vdim = right.n_heads, right.n_kv_heads, right.head_dim, right.v_head_dim
     z = torch.randn(n, right.width, device=dev) * 0.5
-    row("right_projection", timer(lambda: linear.logits(x, right.w_in, z, ctx)), 2.0 * n * right.width * width,
-        right.width * width * 2 + n * (width * 2 + right.width * 4))
     u = torch.empty(n, -(-(right.conv_ch + 2 * H) // 4) * 4, dtype=f32, device=dev)
     decay = torch.empty(n, H * dim, dtype=f32, device=dev)
     gate = torch.empty(n, right.v_dim, dtype=f32, device=dev)
@@ -112,7 +112,7 @@ def time_parts(engine, s: dict, lens_before: list, new_tokens: int, peaks: dict,
                   longest_run=ctx.max_new)
     # convolved channels read and written, the low-rank inputs read, decays and gates written, the maps read once
     maps = s["rank"] * (H * dim + right.v_dim)
-    row("delta_prepare", timer(lambda: right._prepare_channels(z, decay, gate, n, ctx, common)), 2.0 * n * maps,
+    row("delta_prepare", timer(lambda: right._prepare_channels(z, 0, decay, gate, n, ctx, common)), 2.0 * n * maps,
         n * (right.conv_ch * 8 + (H * dim + right.v_dim) * 4 + 2 * s["rank"] * 4 + H * 8) + maps * 2 + 2 * B * conv.state[0].numel() * 4)
     o = torch.empty(n, right.v_dim, dtype=f32, device=dev)
     ms = timer(lambda: ops.state_scan(u, matrix.state, o, ctx.cu_seqlens, ctx.seq_slot, n_seqs=ctx.n_seqs, heads=H, groups=G, dim=dim,
@@ -185,7 +185,7 @@ def time_parts(engine, s: dict, lens_before: list, new_tokens: int, peaks: dict,
 
 # how far each kernel of the design is from its roofline, over the like kernel of the closest model
 LIKE = {"norm_and_input_convolutions": ("dense", "rms_norm"), "window_attention": ("lulisun", "attention"),
-        "convolve_store": ("dense", "rotate_store"), "left_projection": ("dense", "down"), "right_projection": ("dense", "down"),
+        "convolve_store": ("dense", "rotate_store"), "members_projection": ("dense", "down"),
         "lightning_projection": ("dense", "down"), "normed_sum": ("redodra", "normed_sum"), "delta_prepare": ("redodra", "delta_rule_prepare"),
         "delta_scan": ("redodra", "delta_rule_scan"), "delta_gated_norm": ("redodra", "delta_rule_gated_norm"),
         "lightning_scan": ("redodra", "state_space_scan"), "lightning_gated_norm": ("redodra", "state_space_gated_norm"),

@@ -1058,10 +1058,13 @@ def stream_update(stream_x: torch.Tensor, *, branch=None, branch_bias=None, post
           _p(next_out if next_norm is not None else None), c_int(next_dtype), c_int(t), c_int(n), _stream())
 
 
-def normed_sum(members: list, out: torch.Tensor, eps: float, accumulate: bool = False) -> torch.Tensor:
+def normed_sum(members: list, out: torch.Tensor, eps: float, accumulate: bool = False, clear: torch.Tensor | None = None) -> torch.Tensor:
     """out (+)= sum over members (x, bias or None, weight, scale) of scale * rmsnorm(x + bias) * weight, row by row; every x
-    (float32 [T, n]) is left zeroed."""
+    (float32 [T, n]) is left zeroed, and so is `clear` (float32 [T, .], None: nothing more)."""
     t, n = out.shape
+    if clear is not None:
+        _need_cuda(clear)
+        _need(clear.dtype == torch.float32 and clear.is_contiguous() and clear.shape[0] == t, "normed_sum: clear must be float32 [T, .]")
     _need(1 <= len(members) <= 4, "normed_sum: one to four members")
     _need(out.dtype == torch.float32 and out.is_contiguous(), "normed_sum: out must be float32")
     xs, bs, ws, sc = (c_void_p * 4)(), (c_void_p * 4)(), (c_void_p * 4)(), (c_float * 4)()
@@ -1073,7 +1076,7 @@ def normed_sum(members: list, out: torch.Tensor, eps: float, accumulate: bool = 
             _f32_vec(bias, n, "normed_sum: bias")
         xs[m], bs[m], ws[m], sc[m] = x.data_ptr(), (bias.data_ptr() if bias is not None else None), w.data_ptr(), float(scale)
     _call("stream", "ri_normed_sum", xs, bs, ws, sc, c_int(len(members)), _p(out), c_int(t), c_int(n), c_float(eps),
-          c_int(1 if accumulate else 0), _stream())
+          c_int(1 if accumulate else 0), _p(clear), c_int(clear.shape[1] if clear is not None else 0), _stream())
     return out
 
 
@@ -1275,15 +1278,15 @@ def input_conv(x: torch.Tensor, weight, eps: float, taps_a: torch.Tensor, taps_b
 
 def conv_store(z: torch.Tensor, bias, taps: torch.Tensor, carried: torch.Tensor, q_out: torch.Tensor, kcache, vcache, cu_seqlens,
                token_pos, token_seq, seq_slot, page_table, *, n_seqs: int, n_kv_heads: int, head_dim: int, v_head_dim: int,
-               page_size: int, longest_run: int) -> torch.Tensor:
-    """From the projection z (float32 [T, >= channels]: queries, keys, values) plus bias: a short causal convolution per channel
+               page_size: int, longest_run: int, z_col: int = 0) -> torch.Tensor:
+    """From the projection z (float32 [T, .], queries, keys, values from column z_col on) plus bias: a short causal convolution per channel
     (taps float32 [K, channels], the last row the current token's; inputs before the step, biases included, from carried,
     float32 [slots, K - 1, channels], which moves on), then the queries into q_out [T, q channels] and keys and values into
     the tokens' places of the paged cache."""
     _need_cuda(z, bias, taps, carried, q_out, kcache, vcache, cu_seqlens, token_pos, token_seq, seq_slot, page_table)
     t, q_dim = q_out.shape
     k, channels = taps.shape
-    _need(z.dtype == torch.float32 and z.is_contiguous() and z.shape[0] == t and z.shape[1] >= channels
+    _need(z.dtype == torch.float32 and z.is_contiguous() and z.shape[0] == t and z_col >= 0 and z.shape[1] >= z_col + channels
           and channels == q_dim + n_kv_heads * (head_dim + v_head_dim), "conv_store: z must be float32 [T, channels]")
     _need(taps.dtype == torch.float32 and taps.is_contiguous(), "conv_store: taps must be float32 [K, channels]")
     if bias is not None:
@@ -1293,7 +1296,7 @@ def conv_store(z: torch.Tensor, bias, taps: torch.Tensor, carried: torch.Tensor,
     _need(q_out.is_contiguous() and kcache.dtype == q_out.dtype and vcache.dtype == q_out.dtype and kcache.is_contiguous()
           and vcache.is_contiguous() and tuple(kcache.shape[1:]) == (n_kv_heads, page_size, head_dim)
           and tuple(vcache.shape[1:]) == (n_kv_heads, page_size, v_head_dim), "conv_store: queries and cache")
-    _call("short_conv", "ri_conv_store", _p(z), c_int(z.shape[1]), _p(bias), _p(taps), c_int(k), _p(carried), _p(q_out), _p(kcache),
+    _call("short_conv", "ri_conv_store", c_void_p(z.data_ptr() + 4 * z_col), c_int(z.shape[1]), _p(bias), _p(taps), c_int(k), _p(carried), _p(q_out), _p(kcache),
           _p(vcache), c_int(dtype_code(q_out.dtype)), _p(cu_seqlens), _p(token_pos), _p(token_seq), _p(seq_slot), _p(page_table),
           c_int(page_table.shape[1]), c_int(t), c_int(n_seqs), c_int(q_dim), c_int(n_kv_heads), c_int(head_dim), c_int(v_head_dim),
           c_int(page_size), c_int(longest_run), _stream())

@@ -225,22 +225,41 @@ class GQAttention(Mixer):
             return keys
         return keys, StateRequest((self.conv - 1, self.q_dim + self.kv_dim + self.v_dim), torch.float32)
 
-    def _convolved(self, x, ctx, cache_layer, writes_cache):
-        """The queries [T, heads * head_dim] behind projection and convolution; keys and values go into the cache."""
+    @property
+    def float32_projection(self) -> bool:
+        """True: the part reads its projection in float32 and can be handed it inside a wider matrix (`forward_projected`)."""
+        return self.conv is not None
+
+    def projection(self):
+        return self.w_qkv
+
+    def set_projection(self, w) -> None:
+        self.w_qkv = w
+
+    def _convolved(self, z, col, ctx, cache_layer, writes_cache):
+        """The queries [T, heads * head_dim] behind the convolution of the projection (the columns of z from `col` on); keys
+        and values go into the cache."""
         if not writes_cache:
             raise ValueError("a convolution's carried inputs have one writer: a layer cannot read another layer's")
         keys, carried = cache_layer.parts
-        n = x.shape[0]
-        z = ctx.buffer("conv_z", (n, self.w_qkv.n), torch.float32)
-        linear.logits(x, self.w_qkv, z, ctx)                       # float32 results in both precisions
-        q = ctx.buffer("q_conv", (n, self.q_dim), self.dtype)
+        q = ctx.buffer("q_conv", (z.shape[0], self.q_dim), self.dtype)
         ops.conv_store(z, self.b_qkv, self.w_conv, carried.state, q, keys.k, keys.v, ctx.cu_seqlens, ctx.token_pos, ctx.token_seq,
                        ctx.seq_slot, ctx.page_table, n_seqs=ctx.n_seqs, n_kv_heads=self.n_kv_heads, head_dim=self.head_dim,
-                       v_head_dim=self.v_head_dim, page_size=ctx.page_size, longest_run=ctx.max_new)
+                       v_head_dim=self.v_head_dim, page_size=ctx.page_size, longest_run=ctx.max_new, z_col=col)
         return q, keys
+
+    def forward_projected(self, z, col, residual, ctx, cache_layer, writes_cache):
+        """`forward` from the projection: float32 [T, .], this part's columns from `col` on."""
+        q, keys = self._convolved(z, col, ctx, cache_layer, writes_cache)
+        self._attend(q, 0, residual, ctx, keys)
 
     def forward(self, x, residual, ctx, cache_layer, writes_cache):
         n = x.shape[0]
+        if self.conv is not None:
+            z = ctx.buffer("conv_z", (n, self.w_qkv.n), torch.float32)
+            linear.logits(x, self.w_qkv, z, ctx)                       # float32 results in both precisions
+            self.forward_projected(z, 0, residual, ctx, cache_layer, writes_cache)
+            return
         # a layer that has key and value projections but is scheduled to read another layer's cache leaves its own unused
         kv_width = (self.kv_dim + (0 if self.values_from_keys else self.v_dim)) if self.own_kv else 0
         gate_col = self.q_dim + kv_width
@@ -249,9 +268,7 @@ class GQAttention(Mixer):
         usual = (self.v_head_dim == self.head_dim and not getattr(self.position, "partial", False) and not special
                  and not self.extended)
         from_acc = getattr(self.position, "apply_and_store_from_accumulators", None) if usual else None
-        if self.conv is not None:
-            qkv, cache_layer = self._convolved(x, ctx, cache_layer, writes_cache)
-        elif from_acc is not None and linear.wants_split(x, self.w_qkv):
+        if from_acc is not None and linear.wants_split(x, self.w_qkv):
             # a small step: the projection is split over K into float32 accumulators, and the
             # position encoding adds the bias, rotates and stores from there
             acc = ctx.zeroed_buffer("qkv_acc", (n, width), torch.float32)
@@ -274,7 +291,11 @@ class GQAttention(Mixer):
                 self.position.apply_and_store(qkv, ctx, cache_layer, n_heads=self.n_heads,
                                               n_kv_heads=self.n_kv_heads, head_dim=self.head_dim,
                                               write_kv=writes_cache and self.own_kv, **extra)
-        mixed = ctx.buffer("attn_out", (n, self.o_dim), self.dtype)
+        self._attend(qkv, gate_col, residual, ctx, cache_layer)
+
+    def _attend(self, qkv, gate_col, residual, ctx, cache_layer):
+        """Attention over the cache, gates and the output projection; the queries are qkv's first columns."""
+        mixed = ctx.buffer("attn_out", (qkv.shape[0], self.o_dim), self.dtype)
         attn_kernels.attention(qkv, cache_layer, mixed, ctx, n_heads=self.n_heads,
                                n_kv_heads=self.n_kv_heads, head_dim=self.head_dim, scale=self.scale,
                                window=self.window or 0, chunk=self.chunk or 0, v_head_dim=self.v_head_dim,

@@ -140,26 +140,38 @@ class GatedDeltaRule(Mixer):
         return (StateRequest((self.n_heads, self.head_dim, self.v_head_dim), torch.float32),
                 StateRequest((self.taps - 1, self.conv_ch), torch.float32))
 
+    float32_projection = True       # the projection may come inside a wider matrix (`forward_projected`)
+
+    def projection(self):
+        return self.w_in
+
+    def set_projection(self, w) -> None:
+        self.w_in = w
+
     def forward(self, x, residual, ctx, cache_layer, writes_cache):
+        z = ctx.buffer("scan_z", (x.shape[0], self.width), torch.float32)
+        linear.logits(x, self.w_in, z, ctx)                            # float32 results in both precisions
+        self.forward_projected(z, 0, residual, ctx, cache_layer, writes_cache)
+
+    def forward_projected(self, z, col, residual, ctx, cache_layer, writes_cache):
+        """`forward` from the projection: float32 [T, .], this part's columns from `col` on."""
         if not writes_cache:
             raise ValueError("a recurrent state has one writer: a layer cannot read another layer's state")
         matrix, carried = cache_layer.parts
-        n, H, G = x.shape[0], self.n_heads, self.n_kv_heads
-        z = ctx.buffer("scan_z", (n, self.width), torch.float32)
-        linear.logits(x, self.w_in, z, ctx)                            # float32 results in both precisions
+        n, H, G = z.shape[0], self.n_heads, self.n_kv_heads
         u = ctx.buffer("scan_u", (n, -(-(self.conv_ch + 2 * H) // 4) * 4), torch.float32)
-        common = dict(conv_col=0, conv_ch=self.conv_ch, taps=self.w_conv, conv_state=carried.state, unit_heads=2 * G,
-                      unit_dim=self.head_dim, scaled_heads=G, unit_scale=self.head_dim ** -0.5, heads=H, step_col=self.beta_col,
+        common = dict(conv_col=col, conv_ch=self.conv_ch, taps=self.w_conv, conv_state=carried.state, unit_heads=2 * G,
+                      unit_dim=self.head_dim, scaled_heads=G, unit_scale=self.head_dim ** -0.5, heads=H, step_col=col + self.beta_col,
                       a_log=self.a_log, dt_bias=self.dt_bias, out=u, cu_seqlens=ctx.cu_seqlens, token_seq=ctx.token_seq,
                       seq_slot=ctx.seq_slot, n_seqs=ctx.n_seqs, longest_run=ctx.max_new)
-        gate, gate_col, decay = z, self.gate_col, None
+        gate, gate_col, decay = z, col + self.gate_col, None
         if self.decay_rank is None:
-            ops.scan_prepare(z, conv_bias=None, decay_col=self.a_col, **common)
+            ops.scan_prepare(z, conv_bias=None, decay_col=col + self.a_col, **common)
         else:
             decay = ctx.buffer("scan_decay", (n, H * self.head_dim), torch.float32)
             if self.gate_rank is not None:
                 gate, gate_col = ctx.buffer("scan_gate", (n, self.v_dim), torch.float32), 0
-            self._prepare_channels(z, decay, gate, n, ctx, common)
+            self._prepare_channels(z, col, decay, gate, n, ctx, common)
         o = ctx.buffer("scan_o", (n, self.v_dim), torch.float32)
         ops.state_scan(u, matrix.state, o, ctx.cu_seqlens, ctx.seq_slot, n_seqs=ctx.n_seqs, heads=H, groups=G,
                        dim=self.head_dim, vdim=self.v_head_dim, q_col=0, k_col=self.qk_dim, v_col=2 * self.qk_dim,
@@ -176,14 +188,14 @@ class GatedDeltaRule(Mixer):
         ops.low_rank_rows(z, col, rank, padded, rows)
         linear.logits(rows, wide, out, ctx)
 
-    def _prepare_channels(self, z, decay, gate, n, ctx, common):
+    def _prepare_channels(self, z, col, decay, gate, n, ctx, common):
         """Convolved channels, steps, decays per key channel and the low-rank gate."""
         low_gate = self.gate_rank is not None
         if n <= ops.LOW_RANK_FORMED_TOKENS:
-            gate_kw = dict(gate_w2=self.w_gate, gate_low_col=self.gate_col, gate_out=gate) if low_gate else {}
-            ops.scan_prepare_channels(z, head_dim=self.head_dim, decay=decay, w2=self.w_decay, low_col=self.a_col, **gate_kw, **common)
+            gate_kw = dict(gate_w2=self.w_gate, gate_low_col=col + self.gate_col, gate_out=gate) if low_gate else {}
+            ops.scan_prepare_channels(z, head_dim=self.head_dim, decay=decay, w2=self.w_decay, low_col=col + self.a_col, **gate_kw, **common)
             return
-        self._low_rank_product(z, self.a_col, self.decay_rank, self.w_decay_wide, decay, "scan_low_decay", ctx)
+        self._low_rank_product(z, col + self.a_col, self.decay_rank, self.w_decay_wide, decay, "scan_low_decay", ctx)
         if low_gate:
-            self._low_rank_product(z, self.gate_col, self.gate_rank, self.w_gate_wide, gate, "scan_low_gate", ctx)
+            self._low_rank_product(z, col + self.gate_col, self.gate_rank, self.w_gate_wide, gate, "scan_low_gate", ctx)
         ops.scan_prepare_channels(z, head_dim=self.head_dim, decay=decay, raw=decay, **common)

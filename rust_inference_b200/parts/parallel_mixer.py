@@ -3,7 +3,7 @@ from __future__ import annotations
 
 import torch
 
-from ..kernels import ops
+from ..kernels import linear, ops
 from .base import Mixer
 from .registry import lookup, register
 from .spec import PartSpec, TensorSpec
@@ -20,7 +20,9 @@ class ParallelMixers(Mixer):
     `member_norm` = {"eps": e, "weight_name": name}: every member's result is RMS-normed over the model width with a
     plain weight of its own (the tensor `name` below the member's prefix) before it is scaled and added:
     residual += sum_m scale_m * rmsnorm(mixer_m(x)) * w_m.  A member then writes into a zeroed float32 buffer of its
-    own, and one kernel norms and adds all of them (with the output bias of a member that can hand it over)."""
+    own, and one kernel norms and adds all of them (with the output bias of a member that can hand it over).
+    Members that all read their projections in float32 then have them as one product (their matrices lie one below the
+    other): a step of few tokens cuts it over K into a zeroed accumulator, which the kernel that adds the results zeroes again."""
 
     def __init__(self, *, members, member_norm: dict | None = None, hidden_size: int, dtype, device):
         super().__init__(hidden_size=hidden_size, dtype=dtype, device=device)
@@ -39,6 +41,8 @@ class ParallelMixers(Mixer):
                 part.hands_over_bias = True
             self.members.append((spec.prefix, part))
             self.scales.append(float(scale))
+        self.w_in = None                 # the members' projections as one matrix, and where each begins
+        self.cols = []
         if not self.members:
             raise ValueError("parallel_mixers: no members")
         self.graph_safe = all(getattr(p, "graph_safe", True) for _, p in self.members)
@@ -62,6 +66,14 @@ class ParallelMixers(Mixer):
             part.set_tensors({local: tensors[prefix + local] for local in part.tensor_specs()})
         if self.member_norm is not None:
             self.norm_weights = [tensors[prefix + self.member_norm["weight_name"]].contiguous() for prefix, _ in self.members]
+            if all(getattr(part, "float32_projection", False) for _, part in self.members):
+                mats = [part.projection().t for _, part in self.members]
+                self.w_in = linear.Weight(torch.cat(mats, dim=0))
+                self.cols, at = [], 0
+                for (_, part), m in zip(self.members, mats):
+                    part.set_projection(linear.Weight(self.w_in.t[at:at + m.shape[0]]))         # the same storage
+                    self.cols.append(at)
+                    at += m.shape[0]
 
     def get_tensors(self):
         out = {prefix + local: t for prefix, part in self.members for local, t in part.get_tensors().items()}
@@ -82,9 +94,20 @@ class ParallelMixers(Mixer):
             for (_, part), sub in zip(self.members, cache_layer.parts):
                 part.forward(x, residual, ctx, sub, writes_cache)
             return
-        joined = []
+        joined, z, cleared = [], None, None
+        if self.w_in is not None:
+            shape = (x.shape[0], self.w_in.n)
+            if linear.wants_split(x, self.w_in):
+                z = cleared = ctx.zeroed_buffer("members_z", shape, torch.float32)
+                linear.accumulate_split(x, self.w_in, z, ctx)
+            else:
+                z = ctx.buffer("members_z", shape, torch.float32)
+                linear.logits(x, self.w_in, z, ctx)
         for m, ((_, part), sub) in enumerate(zip(self.members, cache_layer.parts)):
             own = ctx.zeroed_buffer(f"member_result_{m}", tuple(residual.shape), torch.float32)
-            part.forward(x, own, ctx, sub, writes_cache)
+            if z is not None:
+                part.forward_projected(z, self.cols[m], own, ctx, sub, writes_cache)
+            else:
+                part.forward(x, own, ctx, sub, writes_cache)
             joined.append((own, part.b_o if getattr(part, "hands_over_bias", False) else None, self.norm_weights[m], self.scales[m]))
-        ops.normed_sum(joined, residual, self.member_norm["eps"], accumulate=True)
+        ops.normed_sum(joined, residual, self.member_norm["eps"], accumulate=True, clear=cleared)
