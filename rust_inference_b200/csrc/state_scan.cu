@@ -367,12 +367,14 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(Scan p) {
     if (t0 >= t1 || !RI_BLOCK_IN_LIMIT(slot, RI_LIMIT_SLOTS, RI_CHECK_SLOT)) return;
     float* S = MODE == WHOLE ? p.state + (((size_t)slot * p.heads + h) * p.dim) * p.vdim
                              : p.piece_state + ((((size_t)b * p.max_pieces + pc) * p.heads + h) * p.dim) * p.vdim;
-    float s[ROWS];
+    constexpr int PAIRS = ROWS / 2;                        // two neighbouring rows at a time through the packed float32 pipe
+    float2 s[PAIRS];
 #pragma unroll
-    for (int k = 0; k < ROWS; ++k) s[k] = (MODE != LOCAL && live && i0 + k < p.dim) ? S[(size_t)(i0 + k) * p.vdim + j] : 0.f;
-    float decays = 1.f, v_before = 0.f, q_before[ROWS];
+    for (int k = 0; k < ROWS; ++k) (k & 1 ? s[k / 2].y : s[k / 2].x) = (MODE != LOCAL && live && i0 + k < p.dim) ? S[(size_t)(i0 + k) * p.vdim + j] : 0.f;
+    float decays = 1.f, v_before = 0.f;
+    float2 q_before[PAIRS];
 #pragma unroll
-    for (int k = 0; k < ROWS; ++k) q_before[k] = 0.f;
+    for (int k = 0; k < PAIRS; ++k) q_before[k] = make_float2(0.f, 0.f);
     const float fixed = DECAY == FIXED ? p.decay[h] : 1.f;
     const int g = h / (p.heads / p.groups);
     const int q_off = p.q_col + g * p.dim, k_off = p.k_col + g * p.dim, v_off = p.v_col + h * p.vdim + j0;
@@ -380,20 +382,37 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(Scan p) {
     const int o_ld = p.heads * p.vdim;
     __syncthreads();                                      // the zeros are in place
 
+    // A token's 16-byte pieces are shared out among the threads once, and a thread copies its piece of every token: where it
+    // starts, how far the next token's lies, and its place in a token's part of the tile (-1: no piece).
+    constexpr int ITEMS = ROWS <= 16 ? 1 : 2;
+    const float* item_src[ITEMS];
+    int item_step[ITEMS], item_at[ITEMS];
+#pragma unroll
+    for (int m = 0; m < ITEMS; ++m) {
+        const int it = threadIdx.x + m * SCAN_THREADS;
+        const int dq = p.dim >> 2, parts = DECAY == CHANNELS ? 3 : 2;
+        const int part = dq > 0 ? it / dq : parts, c = 4 * (it - part * dq);
+        item_src[m] = p.u;
+        item_step[m] = p.ld;
+        item_at[m] = -1;
+        if (part < parts) {
+            item_at[m] = part * R * SLICE + c / ROWS * SLICE + c % ROWS;
+            item_src[m] = part == 0 ? p.u + k_off + c : part == 1 ? p.u + q_off + c : p.decay + (size_t)h * p.dim + c;
+            if (part == 2) item_step[m] = p.heads * p.dim;
+        } else if (it < parts * dq + (cols >> 2)) {
+            const int cc = 4 * (it - parts * dq);
+            item_at[m] = V_AT + cc;
+            item_src[m] = p.u + v_off + cc;
+        }
+    }
     // the copies of the tokens tb .. tb + n_tok - 1 into one of the two tiles; every thread commits one group
     auto fetch = [&](float* dst, int tb, int n_tok) {
         if (p.vec) {
-            const int dq = p.dim >> 2, cq = cols >> 2, parts = DECAY == CHANNELS ? 3 : 2, per = parts * dq + cq;
-            for (int tok = 0; tok < n_tok; ++tok) {
-                const float* row = p.u + (size_t)(tb + tok) * p.ld;
-                float* base = dst + tok * TOKEN;
-                for (int it = threadIdx.x; it < per; it += SCAN_THREADS) {
-                    if (it < dq) copy_async16(base + (4 * it / ROWS) * SLICE + 4 * it % ROWS, row + k_off + 4 * it);
-                    else if (it < 2 * dq) copy_async16(base + R * SLICE + (4 * (it - dq) / ROWS) * SLICE + 4 * (it - dq) % ROWS, row + q_off + 4 * (it - dq));
-                    else if (DECAY == CHANNELS && it < 3 * dq) copy_async16(base + 2 * R * SLICE + (4 * (it - 2 * dq) / ROWS) * SLICE + 4 * (it - 2 * dq) % ROWS, p.decay + ((size_t)(tb + tok) * p.heads + h) * p.dim + 4 * (it - 2 * dq));
-                    else copy_async16(base + V_AT + 4 * (it - parts * dq), row + v_off + 4 * (it - parts * dq));
-                }
-            }
+#pragma unroll
+            for (int m = 0; m < ITEMS; ++m)
+                if (item_at[m] >= 0)
+                    for (int tok = 0; tok < n_tok; ++tok)
+                        copy_async16(dst + tok * TOKEN + item_at[m], item_src[m] + (size_t)(tb + tok) * item_step[m]);
         } else {
             const int parts = DECAY == CHANNELS ? 3 : 2, per = parts * p.dim + cols;
             for (int tok = 0; tok < n_tok; ++tok) {
@@ -446,34 +465,30 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(Scan p) {
             const float v = base[V_AT + jj];
             const float a = DECAY == FIXED ? fixed : DECAY == CHANNELS ? 1.f : base[V_AT + COLS];
             const float step = DECAY == FIXED ? 1.f : base[V_AT + COLS + 1];
-            float kk[ROWS], qq[ROWS], aa[ROWS];
+            float2 kk[PAIRS], qq[PAIRS], aa[PAIRS];
 #pragma unroll
             for (int k = 0; k < ROWS / 4; ++k) {
                 const float4 kv = k4[k];
-                kk[4 * k] = kv.x; kk[4 * k + 1] = kv.y; kk[4 * k + 2] = kv.z; kk[4 * k + 3] = kv.w;
+                kk[2 * k] = make_float2(kv.x, kv.y); kk[2 * k + 1] = make_float2(kv.z, kv.w);
                 if (MODE != LOCAL) {
                     const float4 qv = q4[k];
-                    qq[4 * k] = qv.x; qq[4 * k + 1] = qv.y; qq[4 * k + 2] = qv.z; qq[4 * k + 3] = qv.w;
+                    qq[2 * k] = make_float2(qv.x, qv.y); qq[2 * k + 1] = make_float2(qv.z, qv.w);
                 }
                 if (DECAY == CHANNELS) {
                     const float4 av = a4[k];
-                    aa[4 * k] = av.x; aa[4 * k + 1] = av.y; aa[4 * k + 2] = av.z; aa[4 * k + 3] = av.w;
+                    aa[2 * k] = make_float2(av.x, av.y); aa[2 * k + 1] = make_float2(av.z, av.w);
                 }
             }
             if (MODE == LOCAL) decays *= a;
-            float d0 = 0.f, d1 = 0.f, e0 = 0.f, e1 = 0.f;
+            float2 d2[2] = {make_float2(0.f, 0.f), make_float2(0.f, 0.f)}, e2[2] = {make_float2(0.f, 0.f), make_float2(0.f, 0.f)};
 #pragma unroll
-            for (int k = 0; k < ROWS; k += 2) {
-                if (DELTA) {
-                    d0 = fmaf(s[k], DECAY == CHANNELS ? aa[k] * kk[k] : kk[k], d0);
-                    d1 = fmaf(s[k + 1], DECAY == CHANNELS ? aa[k + 1] * kk[k + 1] : kk[k + 1], d1);
-                }
-                if (MODE != LOCAL) {
-                    e0 = fmaf(s[k], q_before[k], e0);
-                    e1 = fmaf(s[k + 1], q_before[k + 1], e1);
-                }
+            for (int k = 0; k < PAIRS; ++k) {
+                if (DELTA) d2[k & 1] = __ffma2_rn(s[k], DECAY == CHANNELS ? __fmul2_rn(aa[k], kk[k]) : kk[k], d2[k & 1]);
+                if (MODE != LOCAL) e2[k & 1] = __ffma2_rn(s[k], q_before[k], e2[k & 1]);
             }
-            float dot = d0 + d1, acc = e0 + e1;
+            d2[0] = __fadd2_rn(d2[0], d2[1]);
+            e2[0] = __fadd2_rn(e2[0], e2[1]);
+            float dot = d2[0].x + d2[0].y, acc = e2[0].x + e2[0].y;
 #pragma unroll
             for (int o = R / 2; o > 0; o >>= 1) {
                 if (DELTA) dot += __shfl_xor_sync(0xffffffffu, dot, o);
@@ -484,30 +499,29 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(Scan p) {
                 v_before = v;
             }
             const float write = DELTA ? step * (v - (DECAY == CHANNELS ? dot : a * dot)) : step * v;
+            const float2 write2 = make_float2(write, write), keep2 = make_float2(a, a);
 #pragma unroll
-            for (int k = 0; k < ROWS; ++k) {
-                s[k] = fmaf(DECAY == CHANNELS ? aa[k] : a, s[k], kk[k] * write);
+            for (int k = 0; k < PAIRS; ++k) {
+                s[k] = __ffma2_rn(DECAY == CHANNELS ? aa[k] : keep2, s[k], __fmul2_rn(kk[k], write2));
                 if (MODE != LOCAL) q_before[k] = qq[k];
             }
         }
         __syncthreads();                                  // this tile may be overwritten by the fetch after next
     }
     if (MODE != LOCAL) {                                  // the last token's read-out
-        float e0 = 0.f, e1 = 0.f;
+        float2 e2 = make_float2(0.f, 0.f);
 #pragma unroll
-        for (int k = 0; k < ROWS; k += 2) {
-            e0 = fmaf(s[k], q_before[k], e0);
-            e1 = fmaf(s[k + 1], q_before[k + 1], e1);
-        }
-        float acc = e0 + e1;
+        for (int k = 0; k < PAIRS; ++k) e2 = __ffma2_rn(s[k], q_before[k], e2);
+        float acc = e2.x + e2.y;
 #pragma unroll
         for (int o = R / 2; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
         if (live && r == 0) p.o[(size_t)(t1 - 1) * o_ld + h * p.vdim + j] = fmaf(skip, v_before, acc);
     }
-    if (MODE == FINAL) return;                            // the carry kernel left the final state in the slot
+    if constexpr (MODE != FINAL) {                        // there the carry kernel left the final state in the slot
 #pragma unroll
-    for (int k = 0; k < ROWS; ++k)
-        if (live && i0 + k < p.dim) S[(size_t)(i0 + k) * p.vdim + j] = s[k];
+        for (int k = 0; k < ROWS; ++k)
+            if (live && i0 + k < p.dim) S[(size_t)(i0 + k) * p.vdim + j] = k & 1 ? s[k / 2].y : s[k / 2].x;
+    }
     if (MODE == LOCAL && blockIdx.z == 0 && threadIdx.x == 0) p.piece_decay[((size_t)b * p.max_pieces + pc) * p.heads + h] = decays;
 }
 
