@@ -43,6 +43,9 @@ beside a Lulisun-style model and a dense decoder of equal size (`rust_inference_
 `--arch belizen` does it for a Belizen-style model (window attention with kept first positions, normed and rotated heads and
 a gate on the result; gated linear attention; routed experts with pass-through ones; a run of layers passed again) beside the
 same two (`rust_inference_b200/kernels/belizen_bench.py`).
+`--arch gatarax` does it for a Gatarax-style model (window attention with a sink and convolved projections beside a delta rule with
+decays per key channel, linear attention with fixed decays, short convolutions in front of every sublayer, routed experts) beside a
+Redodra-style model, a Lulisun-style model and a dense decoder (`rust_inference_b200/kernels/gatarax_bench.py`).
 
 Prints ONE JSON line.  Only one GPU is used: for --gpus > 1 it says so and exits with 2.
 """

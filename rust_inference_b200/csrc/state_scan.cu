@@ -540,11 +540,24 @@ __global__ void __launch_bounds__(256) scan_carry_kernel(float* state, float* pi
     const int pieces = (n + piece - 1) / piece;
     float* dst = state + ((size_t)slot * heads + h) * per_head + e;
     float s = *dst;
-    for (int pc = 0; pc < pieces; ++pc) {
-        float* ps = piece_state + (((size_t)b * max_pieces + pc) * heads + h) * per_head + e;
-        const float local = *ps;
-        *ps = s;
-        s = fmaf(piece_decay[((size_t)b * max_pieces + pc) * heads + h], s, local);
+    // several pieces' loads are in flight before the first of their stores
+    constexpr int AHEAD = 8;
+    const size_t piece_step = (size_t)heads * per_head;
+    float* ps = piece_state + ((size_t)b * max_pieces * heads + h) * per_head + e;
+    const float* pd = piece_decay + (size_t)b * max_pieces * heads + h;
+    for (int pc = 0; pc < pieces; pc += AHEAD) {
+        float local[AHEAD], keep[AHEAD];
+#pragma unroll
+        for (int i = 0; i < AHEAD; ++i) {
+            local[i] = pc + i < pieces ? ps[(size_t)(pc + i) * piece_step] : 0.f;
+            keep[i] = pc + i < pieces ? pd[(size_t)(pc + i) * heads] : 1.f;
+        }
+#pragma unroll
+        for (int i = 0; i < AHEAD; ++i)
+            if (pc + i < pieces) {
+                ps[(size_t)(pc + i) * piece_step] = s;
+                s = fmaf(keep[i], s, local[i]);
+            }
     }
     *dst = s;
 }
@@ -635,17 +648,32 @@ __global__ void __launch_bounds__(1024) gated_group_norm_block_kernel(const floa
 }
 
 constexpr int SCAN_SMEM_LIMIT = 44 * 1024;
+constexpr int SCAN_SMEM_MOST = 216 * 1024;        // of an SM's 228 KB, with a kilobyte of the system's per block
+constexpr int SMS = 148;
 
 template <int ROWS, bool DELTA, int DECAY>
 int launch_scan(dim3 grid, cudaStream_t stream, Scan p, int longest, int n_seqs) {
     const int token_bytes = ((DECAY == CHANNELS ? 3 : 2) * R * (ROWS + 4) + COLS + 4) * (int)sizeof(float);
-    int tile_t = SCAN_SMEM_LIMIT / (2 * token_bytes);     // two tiles
-    if (tile_t > 16) tile_t = 16;
+    // A long one-pass scan is as slow as its most crowded SM.  Its blocks come onto the SMs while the kernel before still holds
+    // some of them, so blocks are kept apart by their shared memory: no more fit an SM than it gets when all are spread evenly
+    // (and the tiles are larger for it).
+    const long long blocks = (long long)grid.x * grid.y * grid.z;
+    const bool apart = p.piece <= 0 && longest >= 64 && blocks <= 4 * SMS;
+    const int per_sm = (int)((blocks + SMS - 1) / SMS);
+    const int budget = apart ? SCAN_SMEM_MOST / per_sm : SCAN_SMEM_LIMIT;
+    int tile_t = budget / (2 * token_bytes);              // two tiles
+    if (tile_t > (apart ? 32 : 16)) tile_t = apart ? 32 : 16;
     if (longest > 0 && tile_t > longest) tile_t = longest;
     if (tile_t < 1) tile_t = 1;
     p.tile_t = tile_t;
-    const size_t smem = (size_t)2 * tile_t * token_bytes;
+    size_t smem = (size_t)2 * tile_t * token_bytes;
     cudaError_t e;
+    if (apart) {
+        const size_t least = (size_t)(SCAN_SMEM_MOST / (per_sm + 1) + 8 * 1024);       // one block more would not fit
+        if (smem < least) smem = least;
+        static PerDeviceOnce once;
+        if (int rc = raise_dynamic_smem(state_scan_kernel<ROWS, DELTA, WHOLE, DECAY>, SCAN_SMEM_MOST, once, "state_scan")) return rc;
+    }
     if constexpr (!DELTA) {
         if (p.piece > 0) {
             const dim3 pieces(grid.x * p.max_pieces, grid.y, grid.z);
