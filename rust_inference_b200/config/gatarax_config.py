@@ -1,6 +1,6 @@
 """Typed configuration of the Gatarax decoder, read from config.json.
 
-config.json gives every size and every constant that can differ between models of the design:
+What config.json holds (sizes and constants come from nowhere else):
 
     {"architecture": "Gatarax", "vocab": V, "width": D, "norm": {"eps": e}, "canon": {"taps": K},
      "embedding": {"scale": s}, "logit_scale": c,
