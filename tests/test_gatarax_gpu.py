@@ -120,6 +120,28 @@ def test_input_convolutions(dtype, width, taps, two, normed):
     assert taps == 1 or float(carried[1].min()) == 7.0               # nobody else's slot was touched
 
 
+@pytest.mark.parametrize("width,taps", [(40, 4), (36, 2), (33, 3), (64, 6)])
+def test_input_convolutions_of_a_very_long_step(width, taps):
+    """A step of more than 4,096 tokens takes eight tokens per block: two sequences whose border lies inside a block."""
+    from rust_inference_b200.kernels import ops
+    g = torch.Generator().manual_seed(width)
+    w = 1.0 + 0.3 * torch.randn(width, generator=g)
+    fa, fb = (torch.randn(width, taps, generator=g) / math.sqrt(taps) for _ in range(2))
+    counts = [2803, 1402]
+    xs = [torch.randn(n, width, generator=g) for n in counts]
+    carried = torch.zeros(2, taps - 1, width, device=DEV)
+    a, b = (torch.empty(sum(counts), width, device=DEV) for _ in range(2))
+    seq = torch.repeat_interleave(torch.arange(2), torch.tensor(counts)).tolist()
+    ops.input_conv(d(torch.cat(xs)), d(w), 1e-5, d(fa.t().contiguous()), d(fb.t().contiguous()), carried, a, b, i32([0, 2803, 4205]), i32(seq),
+                   i32([1, 0]), n_seqs=2, longest_run=2803)
+    for k, (x, slot) in enumerate(zip(xs, (1, 0))):
+        h = pg.unit_rms(x.double(), 1e-5) * w.double()
+        part = slice(0, 2803) if k == 0 else slice(2803, 4205)
+        assert rel_err(a[part], pg.input_conv(h, fa.double())) < 1e-5
+        assert rel_err(b[part], pg.input_conv(h, fb.double())) < 1e-5
+        assert rel_err(carried[slot], h[-(taps - 1):]) < 1e-5
+
+
 @pytest.mark.parametrize("dtype", [F32, BF16])
 @pytest.mark.parametrize("n,width,ff", [(1, 72, 40), (5, 128, 200), (130, 128, 264), (600, 256, 520), (2100, 512, 1024), (9, 100, 36)])
 def test_relu_squared_in_the_product_s_epilogue(dtype, n, width, ff):
@@ -205,6 +227,50 @@ def test_delta_rule_with_channel_decays(dtype, heads, kv, dim, vdim, conv, ranks
     cache, ws = _cache(part, dtype), _workspace()
     for portions in ([n], [1], [2], [70, 1, 1, 3, 33, 16, 17, 2], [3, 1]):
         assert rel_err(_drive(part, cache, x, portions, dtype, ws), want) < PART_TOL[dtype], portions
+
+
+@pytest.mark.parametrize("heads,kv,dim,vdim,conv,ranks", [(4, 2, 16, 24, 3, (5, 3)), (1, 1, 40, 72, 1, (1, 1)), (6, 2, 8, 8, 5, (16, 8)),
+                                                          (2, 1, 128, 64, 2, (64, 7)), (3, 3, 9, 7, 4, (3, 4)), (5, 5, 48, 200, 4, (9, 32)),
+                                                          (2, 2, 256, 32, 4, (8, 8))])
+def test_delta_rule_of_a_long_prompt(heads, kv, dim, vdim, conv, ranks):
+    """Steps of 512 tokens and more prepare several tokens per block and keep the scan's blocks apart: a prompt of 700 tokens
+    whole, cut so that the second portion begins inside a block's tokens, and two prompts in one step whose border lies inside
+    one, each against the plain result."""
+    width, n = 96, 700
+    m = gm.right(heads=heads, kv=kv, dim=dim, vdim=vdim, conv=conv)
+    part, W, p = _part("right", m, F32, width, seed=dim + vdim, hot=1.5, ranks=lambda i: ranks)
+    x = torch.randn(n, width, generator=torch.Generator().manual_seed(conv))
+    want = pg.delta_rule(x.double(), W, p, m, 1e-5)
+    from rust_inference_b200.cache.sequence_cache import SequenceCache
+    cache = SequenceCache([part.cache_request()], max_tokens=4096, max_seq_len=1024, dtype=F32, device=DEV, n_slots=3)
+    ws = _workspace()
+    for portions in ([n], [533, 1, 3, 163]):
+        assert rel_err(_drive(part, cache, x, portions, F32, ws), want) < 5e-5, portions
+    slots = [cache.alloc_slot(), cache.alloc_slot()]
+    counts = [421, 3]
+    out = torch.zeros(sum(counts) + 200, width, device=DEV)
+    third = cache.alloc_slot()
+    ctx = make_ctx(cache, slots + [third], [0, 0, 0], counts + [200], F32, ws)
+    part.forward(d(torch.cat([x[:421], x[:3], x[:200]])), out, ctx, cache.layer(0), True)
+    for first, count in ((0, 421), (421, 3), (424, 200)):
+        assert rel_err(out[first:first + count], want[:count]) < 5e-5, count
+
+
+@pytest.mark.parametrize("heads,vdim,state,groups,conv,ng", [(3, 16, 8, 1, 4, 1), (4, 8, 24, 2, 2, 4), (2, 130, 20, 2, 5, 1), (6, 12, 20, 3, 1, 9)])
+def test_state_space_of_a_long_prompt(heads, vdim, state, groups, conv, ng):
+    """The state space's preparing kernel shares the path of several tokens per block, with a bias and without unit vectors."""
+    import plain_redodra
+    import redodra_models
+    from test_redodra_gpu import _mixer
+    width, n = 80, 640
+    m = redodra_models.ssm(heads=heads, vdim=vdim, state=state, groups=groups, conv=conv, norm_groups=ng)
+    part, W, p = _mixer("ssm", m, F32, width, seed=state + vdim, hot=1.5)
+    x = torch.randn(n, width, generator=torch.Generator().manual_seed(conv))
+    want = plain_redodra.state_space(x.double(), W, p, m, 1e-5)
+    from rust_inference_b200.cache.sequence_cache import SequenceCache
+    cache = SequenceCache([part.cache_request()], max_tokens=2048, max_seq_len=1024, dtype=F32, device=DEV, n_slots=2)
+    for portions in ([n], [517, 2, 121]):
+        assert rel_err(_drive(part, cache, x, portions, F32, _workspace()), want) < 5e-5, portions
 
 
 @pytest.mark.parametrize("dtype", [F32, BF16])
