@@ -8,18 +8,19 @@
 using namespace ri;
 
 // ----------------------------------------------------------------------------
-// embedding: out[t, :] = table[ids[t], :] * scale        (transformer.rs:74-75; the factor is 1 there)
+// embedding: out[t, :] = table[ids[t], :] * scale        (transformer.rs:74-75; the factor is 1 there), `copies` times
+// side by side (the parallel streams of a model that has several)
 // ----------------------------------------------------------------------------
 template <typename T>
 __global__ void embed_gather_kernel(const T* __restrict__ table, const int* __restrict__ ids,
-                                    float* __restrict__ out, int hidden, float scale) {
+                                    float* __restrict__ out, int hidden, int copies, float scale) {
     const int t = blockIdx.x;
     let_next_kernel_start();
     wait_for_previous_kernels();          // the ids may come from the previous step's sampler
     const int id = ids[t];
-    float* o = out + (size_t)t * hidden;
+    float* o = out + (size_t)t * copies * hidden;
     if (!RI_BLOCK_IN_LIMIT(id, RI_LIMIT_VOCAB, RI_CHECK_TOKEN_ID)) {           // checked build: recorded, the row left zero
-        for (int i = threadIdx.x; i < hidden; i += blockDim.x) o[i] = 0.f;
+        for (int i = threadIdx.x; i < copies * hidden; i += blockDim.x) o[i] = 0.f;
         return;
     }
     const T* row = table + (size_t)id * hidden;
@@ -42,25 +43,33 @@ __global__ void embed_gather_kernel(const T* __restrict__ table, const int* __re
                 const int i = base + j * blockDim.x;
                 if (i < n8) {
                     const T* e = reinterpret_cast<const T*>(&v[j]);
-                    float4* dst = reinterpret_cast<float4*>(o + 8 * (size_t)i);
-                    dst[0] = make_float4(to_f32<T>(e[0]) * scale, to_f32<T>(e[1]) * scale, to_f32<T>(e[2]) * scale, to_f32<T>(e[3]) * scale);
-                    dst[1] = make_float4(to_f32<T>(e[4]) * scale, to_f32<T>(e[5]) * scale, to_f32<T>(e[6]) * scale, to_f32<T>(e[7]) * scale);
+                    const float4 lo = make_float4(to_f32<T>(e[0]) * scale, to_f32<T>(e[1]) * scale, to_f32<T>(e[2]) * scale, to_f32<T>(e[3]) * scale);
+                    const float4 hi = make_float4(to_f32<T>(e[4]) * scale, to_f32<T>(e[5]) * scale, to_f32<T>(e[6]) * scale, to_f32<T>(e[7]) * scale);
+                    for (int c = 0; c < copies; ++c) {
+                        float4* dst = reinterpret_cast<float4*>(o + (size_t)c * hidden + 8 * (size_t)i);
+                        dst[0] = lo;
+                        dst[1] = hi;
+                    }
                 }
             }
         }
         return;
     }
-    for (int i = threadIdx.x; i < hidden; i += blockDim.x) o[i] = to_f32<T>(row[i]) * scale;
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
+        const float v = to_f32<T>(row[i]) * scale;
+        for (int c = 0; c < copies; ++c) o[(size_t)c * hidden + i] = v;
+    }
 }
 
 RI_API int ri_embed_gather(const void* table, int dtype, const int* ids, float* out, int n_tokens,
-                           int hidden, float scale, cudaStream_t stream) {
+                           int hidden, int copies, float scale, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
+    if (copies < 1) return fail("embed_gather: %d copies", copies);
     cudaError_t e = cudaSuccess;
     if (dtype == RI_F32)
-        e = launch_dependent(embed_gather_kernel<float>, n_tokens, 256, 0, stream, (const float*)table, ids, out, hidden, scale);
+        e = launch_dependent(embed_gather_kernel<float>, n_tokens, 256, 0, stream, (const float*)table, ids, out, hidden, copies, scale);
     else if (dtype == RI_BF16)
-        e = launch_dependent(embed_gather_kernel<__nv_bfloat16>, n_tokens, 256, 0, stream, (const __nv_bfloat16*)table, ids, out, hidden, scale);
+        e = launch_dependent(embed_gather_kernel<__nv_bfloat16>, n_tokens, 256, 0, stream, (const __nv_bfloat16*)table, ids, out, hidden, copies, scale);
     else
         return fail("embed_gather: unknown dtype %d", dtype);
     return check_launch(e, "embed_gather");
@@ -658,7 +667,8 @@ RI_API int ri_rope_cache_write(void* qkv, int dtype, int ld, const float* cos_t,
 // head is divided by its root mean square, sqrt(mean(x^2) + eps), and multiplied by a weight of hd values
 // that all heads share (q_w for queries, k_w for keys; null: the head is left as it is); then the first
 // `rot` channels are rotated as above.  q is rewritten in place, k goes to the cache.  The values are
-// either the columns after k (n_kv_heads * v_hd, copied), or, with `v_from_k`, the key heads as they were
+// either the columns after k (n_kv_heads * v_hd, copied; with `mix` v becomes (1 - mix[0]) v + mix[0] v_other, v_other a
+// row of the same values at v_other + t * v_other_ld, in float32 with one rounding), or, with `v_from_k`, the key heads as they were
 // projected, before norm and rotation (v_hd == hd; qkv then has no value columns).
 // A warp per (token, head): the head is read once into shared memory as float32.
 // ----------------------------------------------------------------------------
@@ -673,7 +683,8 @@ rope_normed_cache_write_kernel(T* __restrict__ qkv, int ld, const float* __restr
                                const int* __restrict__ token_seq, const int* __restrict__ seq_slot,
                                const int* __restrict__ page_table, int max_pages, T* __restrict__ kcache,
                                T* __restrict__ vcache, int n_tokens, int n_heads, int n_kv_heads, int hd, int page_size,
-                               int style, int write_kv, int rot, int v_hd, int v_from_k) {
+                               int style, int write_kv, int rot, int v_hd, int v_from_k, const float* __restrict__ mix,
+                               const T* __restrict__ v_other, int v_other_ld) {
     extern __shared__ float head_smem[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     float* x = head_smem + (size_t)warp * hd;
@@ -702,6 +713,12 @@ rope_normed_cache_write_kernel(T* __restrict__ qkv, int ld, const float* __restr
         const int kh = h - n_heads - n_kv_heads;
         const T* src = row + (size_t)(n_heads + n_kv_heads) * hd + (size_t)kh * v_hd;
         T* dst = vcache + (cache_row + (size_t)kh * page_size) * v_hd;
+        if (mix != nullptr) {
+            const float m = mix[0];
+            const T* other = v_other + (size_t)t * v_other_ld + (size_t)kh * v_hd;
+            for (int d = lane; d < v_hd; d += 32) dst[d] = from_f32<T>((1.f - m) * to_f32<T>(src[d]) + m * to_f32<T>(other[d]));
+            return;
+        }
         for (int d = lane; d < v_hd; d += 32) dst[d] = src[d];
         return;
     }
@@ -745,7 +762,8 @@ rope_normed_cache_write_vec_kernel(__nv_bfloat16* __restrict__ qkv, int ld, cons
                                    const int* __restrict__ token_seq, const int* __restrict__ seq_slot,
                                    const int* __restrict__ page_table, int max_pages, __nv_bfloat16* __restrict__ kcache,
                                    __nv_bfloat16* __restrict__ vcache, int n_tokens, int n_heads, int n_kv_heads, int hd,
-                                   int page_size, int style, int write_kv, int rot, int v_hd, int v_from_k) {
+                                   int page_size, int style, int write_kv, int rot, int v_hd, int v_from_k,
+                                   const float* __restrict__ mix, const __nv_bfloat16* __restrict__ v_other, int v_other_ld) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int heads = n_heads + n_kv_heads + (v_from_k ? 0 : n_kv_heads);
     const long long item = (long long)blockIdx.x * NORMED_ROPE_WARPS + warp;
@@ -796,9 +814,19 @@ rope_normed_cache_write_vec_kernel(__nv_bfloat16* __restrict__ qkv, int ld, cons
     __nv_bfloat16* row = qkv + (size_t)t * ld;
     if (h >= n_heads + n_kv_heads) {      // a value head of its own: copy
         const int kh = h - n_heads - n_kv_heads;
-        if (ch < v_hd)
-            *reinterpret_cast<uint4*>(vcache + (cache_row + (size_t)kh * page_size) * v_hd + ch) =
-                *reinterpret_cast<const uint4*>(row + (size_t)(n_heads + n_kv_heads) * hd + (size_t)kh * v_hd + ch);
+        if (ch < v_hd) {
+            uint4 v = *reinterpret_cast<const uint4*>(row + (size_t)(n_heads + n_kv_heads) * hd + (size_t)kh * v_hd + ch);
+            if (mix != nullptr) {
+                const float m = mix[0];
+                float a[8], b[8];
+                unpack8(v, a);
+                unpack8(*reinterpret_cast<const uint4*>(v_other + (size_t)t * v_other_ld + (size_t)kh * v_hd + ch), b);
+#pragma unroll
+                for (int i = 0; i < 8; ++i) a[i] = (1.f - m) * a[i] + m * b[i];
+                v = pack8(a);
+            }
+            *reinterpret_cast<uint4*>(vcache + (cache_row + (size_t)kh * page_size) * v_hd + ch) = v;
+        }
         return;
     }
     const int kh = h - n_heads;
@@ -848,7 +876,7 @@ RI_API int ri_rope_normed_cache_write(void* qkv, int dtype, int ld, const float*
                                       const int* token_seq, const int* seq_slot, const int* page_table, int max_pages,
                                       void* kcache, void* vcache, int n_tokens, int n_heads, int n_kv_heads, int hd,
                                       int page_size, int style, int write_kv, int rot, int v_hd, int v_from_k,
-                                      cudaStream_t stream) {
+                                      const float* mix, const void* v_other, int v_other_ld, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     const bool unrotated = rot < 0;       // rot < 0: nothing is rotated (no tables); 0: the whole head
     if (unrotated) rot = 0;
@@ -857,6 +885,8 @@ RI_API int ri_rope_normed_cache_write(void* qkv, int dtype, int ld, const float*
     if (rot % 2 || rot > hd) return fail("rope_normed_cache_write: %d rotated channels of a head of %d", rot, hd);
     if (!unrotated && (cos_t == nullptr || sin_t == nullptr)) return fail("rope_normed_cache_write: a rotation needs its tables");
     if (style != 0 && style != 1) return fail("rope_normed_cache_write: unknown style %d", style);
+    if (mix != nullptr && (v_from_k || v_other == nullptr || v_other_ld < n_kv_heads * v_hd))
+        return fail("rope_normed_cache_write: blended values need the rows they are blended with");
     if (v_from_k && v_hd != hd) return fail("rope_normed_cache_write: values taken from keys of %d have the size %d", hd, v_hd);
     const size_t smem = (size_t)NORMED_ROPE_WARPS * hd * sizeof(float);
     if (smem > 48 * 1024) return fail("rope_normed_cache_write: heads of %d exceed %d", hd, 48 * 1024 / 4 / NORMED_ROPE_WARPS);
@@ -869,17 +899,18 @@ RI_API int ri_rope_normed_cache_write(void* qkv, int dtype, int ld, const float*
     const bool aligned = hd % 8 == 0 && hd <= 256 && v_hd % 8 == 0 && v_hd <= 256 && rot % 8 == 0 && ld % 8 == 0 &&
                          (uintptr_t)qkv % 16 == 0 && (uintptr_t)kcache % 16 == 0 && (uintptr_t)vcache % 16 == 0 &&
                          (uintptr_t)cos_t % 16 == 0 && (uintptr_t)sin_t % 16 == 0 && (q_w == nullptr || (uintptr_t)q_w % 16 == 0) &&
-                         (k_w == nullptr || (uintptr_t)k_w % 16 == 0);
+                         (k_w == nullptr || (uintptr_t)k_w % 16 == 0) &&
+                         (mix == nullptr || ((uintptr_t)v_other % 16 == 0 && v_other_ld % 8 == 0));
     if (dtype == RI_BF16 && aligned && pairing_ok && !unrotated) {
         e = launch_dependent(rope_normed_cache_write_vec_kernel, blocks, NORMED_ROPE_WARPS * 32, 0, stream, (__nv_bfloat16*)qkv, ld,
                              cos_t, sin_t, q_w, k_w, eps, token_pos, token_seq, seq_slot, page_table, max_pages,
                              (__nv_bfloat16*)kcache, (__nv_bfloat16*)vcache, n_tokens, n_heads, n_kv_heads, hd, page_size, style,
-                             write_kv, rot, v_hd, v_from_k);
+                             write_kv, rot, v_hd, v_from_k, mix, (const __nv_bfloat16*)v_other, v_other_ld);
         return check_launch(e, "rope_normed_cache_write");
     }
 #define RI_NORMED_ROPE(T) launch_dependent(rope_normed_cache_write_kernel<T>, blocks, NORMED_ROPE_WARPS * 32, smem, stream, \
         (T*)qkv, ld, cos_t, sin_t, q_w, k_w, eps, token_pos, token_seq, seq_slot, page_table, max_pages, (T*)kcache, \
-        (T*)vcache, n_tokens, n_heads, n_kv_heads, hd, page_size, style, write_kv, rot, v_hd, v_from_k)
+        (T*)vcache, n_tokens, n_heads, n_kv_heads, hd, page_size, style, write_kv, rot, v_hd, v_from_k, mix, (const T*)v_other, v_other_ld)
     if (dtype == RI_F32) e = RI_NORMED_ROPE(float);
     else if (dtype == RI_BF16) e = RI_NORMED_ROPE(__nv_bfloat16);
     else return fail("rope_normed_cache_write: unknown dtype %d", dtype);

@@ -19,6 +19,10 @@
 // Steps of few rows (decoding) cut the keys into `n_splits` runs as well: every run writes an un-normalised
 // partial result with its (max, sum) to scratch, and a second kernel merges them by log-sum-exp.
 //
+// `window` > 0 limits a query at position p to the positions p - window + 1 .. p: a tile of rows starts at the key tile of
+// its first row's first visible position, and the positions before a row's own window are masked.  `sink`: the softmax's
+// denominator of head h also holds exp(sink[h]), without a value: the first run of keys starts its maximum and sum from it.
+//
 // Q and the key tiles sit in shared memory with rows padded by 16 bytes (conflict-free ldmatrix); key tiles are
 // double-buffered with cp.async.  The result is written head-major, [heads, tokens, RANK]: the rows of the
 // per-head up-projection that follows.
@@ -65,7 +69,7 @@ __global__ void __launch_bounds__(BM * 2 * NZ, 1)
 latent_attn_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ cache,
                    const int* __restrict__ page_table, int max_pages, const int* __restrict__ seq_slot,
                    const int* __restrict__ seq_start, const int* __restrict__ cu_seqlens, int n_heads, int n_tokens,
-                   float scale_log2, int n_splits, float* __restrict__ part_o, float* __restrict__ part_ml,
+                   float scale_log2, int window, const float* __restrict__ sink, int n_splits, float* __restrict__ part_o, float* __restrict__ part_ml,
                    __nv_bfloat16* __restrict__ out) {
     constexpr int KD = RANK + RD;
     constexpr int ROW = (KD + 8) * 2;                 // bytes of a padded row in shared memory
@@ -96,8 +100,10 @@ latent_attn_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
     const int last_row = min(n_rows, r0 + BM) - 1;
     const int n_keys = start + last_row / n_heads + 1;              // the keys the tile's last row sees
     const int n_kt = (n_keys + BN - 1) / BN;
-    const int per = (n_kt + n_splits - 1) / n_splits;
-    const int kt_begin = split * per, kt_end = min(n_kt, kt_begin + per);
+    const int seen_from = window > 0 ? max(0, start + r0 / n_heads - window + 1) : 0;      // by the tile's first row
+    const int kt_first = seen_from / BN;
+    const int per = (n_kt - kt_first + n_splits - 1) / n_splits;
+    const int kt_begin = kt_first + split * per, kt_end = min(n_kt, kt_begin + per);
     const int* pages = page_table + (size_t)seq_slot[b] * max_pages;
     const size_t row_base = (size_t)tok0 * n_heads + r0;            // first query row of the tile
 
@@ -130,6 +136,12 @@ latent_attn_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
     // the positions of this thread's two rows
     const int row_lo = r0 + rw * 16 + (lane >> 2), row_hi = row_lo + 8;
     const int pos_lo = start + row_lo / n_heads, pos_hi = start + row_hi / n_heads;
+    const int from_lo = window > 0 ? pos_lo - window + 1 : 0, from_hi = window > 0 ? pos_hi - window + 1 : 0;
+    if (sink != nullptr && split == 0) {
+        m_lo = sink[row_lo % n_heads] * 1.4426950408889634f;
+        m_hi = sink[row_hi % n_heads] * 1.4426950408889634f;
+        if (half == 0 && (lane & 3) == 0) l_lo = l_hi = 1.f;        // counted once: the sums of a row's lanes are added at the end
+    }
 
     for (int kt = kt_begin; kt < kt_end; ++kt) {
         const int stage = (kt - kt_begin) & 1;
@@ -172,7 +184,7 @@ latent_attn_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
                 s[i][0] += sx[i][0]; s[i][1] += sx[i][1]; s[i][2] += sx[i][2]; s[i][3] += sx[i][3];
             }
         }
-        // causal mask per row, in units of log2
+        // causal mask (and window) per row, in units of log2
         const int j0 = kt * BN + key0 + (lane & 3) * 2;
         float mx_lo = -INFINITY, mx_hi = -INFINITY;
 #pragma unroll
@@ -180,8 +192,8 @@ latent_attn_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
                 const int j = j0 + nt * 8 + e;
-                s[nt][e] = j <= pos_lo ? s[nt][e] * scale_log2 : -INFINITY;
-                s[nt][2 + e] = j <= pos_hi ? s[nt][2 + e] * scale_log2 : -INFINITY;
+                s[nt][e] = j <= pos_lo && j >= from_lo ? s[nt][e] * scale_log2 : -INFINITY;
+                s[nt][2 + e] = j <= pos_hi && j >= from_hi ? s[nt][2 + e] * scale_log2 : -INFINITY;
                 mx_lo = fmaxf(mx_lo, s[nt][e]);
                 mx_hi = fmaxf(mx_hi, s[nt][2 + e]);
             }
@@ -336,8 +348,8 @@ __global__ void latent_attn_combine_kernel(const float* __restrict__ part_o, con
 
 template <int RANK, int RD, int BM>
 int launch(const void* q, const void* cache, const int* page_table, int max_pages, const int* seq_slot, const int* seq_start,
-           const int* cu_seqlens, int n_seqs, int max_new, int n_heads, int n_tokens, float scale, int n_splits, float* part_o,
-           float* part_ml, void* out, cudaStream_t stream) {
+           const int* cu_seqlens, int n_seqs, int max_new, int n_heads, int n_tokens, float scale, int window, const float* sink,
+           int n_splits, float* part_o, float* part_ml, void* out, cudaStream_t stream) {
     constexpr int NZ = RANK > 256 ? 2 : 1;
     constexpr int KD = RANK + RD;
     constexpr int SMEM = (BM + 2 * BN) * (KD + 8) * 2;
@@ -349,7 +361,7 @@ int launch(const void* q, const void* cache, const int* page_table, int max_page
     dim3 grid(tiles, n_seqs * n_splits, 1);
     cudaError_t e = launch_dependent(kernel, grid, dim3(BM * 2 * NZ), (size_t)SMEM, stream, (const __nv_bfloat16*)q,
                                      (const __nv_bfloat16*)cache, page_table, max_pages, seq_slot, seq_start, cu_seqlens, n_heads,
-                                     n_tokens, scale * 1.4426950408889634f, n_splits, part_o, part_ml, (__nv_bfloat16*)out);
+                                     n_tokens, scale * 1.4426950408889634f, window, sink, n_splits, part_o, part_ml, (__nv_bfloat16*)out);
     if (int rc = check_launch(e, "latent_attention")) return rc;
     if (n_splits > 1) {
         e = launch_dependent(latent_attn_combine_kernel, dim3((unsigned)((long long)n_tokens * n_heads)), dim3(RANK >= 512 ? 128 : (RANK >= 256 ? 64 : 32)),
@@ -368,10 +380,10 @@ __host__ int tile_rows_for(long long rows, int rank) {
 
 template <int RANK, int RD>
 int pick(int bm, const void* q, const void* cache, const int* page_table, int max_pages, const int* seq_slot, const int* seq_start,
-         const int* cu_seqlens, int n_seqs, int max_new, int n_heads, int n_tokens, float scale, int n_splits, float* part_o,
-         float* part_ml, void* out, cudaStream_t stream) {
+         const int* cu_seqlens, int n_seqs, int max_new, int n_heads, int n_tokens, float scale, int window, const float* sink,
+         int n_splits, float* part_o, float* part_ml, void* out, cudaStream_t stream) {
 #define RI_TILE(BM) launch<RANK, RD, BM>(q, cache, page_table, max_pages, seq_slot, seq_start, cu_seqlens, n_seqs, max_new, n_heads, \
-                                         n_tokens, scale, n_splits, part_o, part_ml, out, stream)
+                                         n_tokens, scale, window, sink, n_splits, part_o, part_ml, out, stream)
     if constexpr (RANK <= 256) {
         if (bm == 128) return RI_TILE(128);
     }
@@ -397,16 +409,17 @@ RI_API int ri_latent_attention_mma_supports(int rank, int rd, int page_size) {
 // [n_tokens * n_heads * n_splits * rank], part_ml float32 [n_tokens * n_heads * n_splits * 2].
 RI_API int ri_latent_attention_mma(const void* q, const void* cache, const int* page_table, int max_pages, const int* seq_slot,
                                    const int* seq_start, const int* cu_seqlens, int n_seqs, int max_new, int n_heads,
-                                   int n_tokens, int rank, int rd, float scale, int n_splits, float* part_o, float* part_ml,
+                                   int n_tokens, int rank, int rd, float scale, int window, const float* sink, int n_splits, float* part_o, float* part_ml,
                                    void* out, cudaStream_t stream) {
     if (n_tokens <= 0 || n_seqs <= 0) return 0;
+    if (window < 0) return fail("latent_attention: window %d", window);
     if (n_splits > MAX_RUNS) return fail("latent_attention: %d runs of keys exceed %d", n_splits, MAX_RUNS);
     if (n_splits < 1 || (n_splits > 1 && (part_o == nullptr || part_ml == nullptr)))
         return fail("latent_attention: %d runs of keys need scratch for their partial results", n_splits);
     if ((long long)n_seqs * n_splits > 65535) return fail("latent_attention: %d sequences x %d runs exceed the grid limit", n_seqs, n_splits);
     const int bm = tile_rows_for((long long)max_new * n_heads, rank);
 #define RI_LATENT(R, D) if (rank == R && rd == D) return pick<R, D>(bm, q, cache, page_table, max_pages, seq_slot, seq_start, cu_seqlens, \
-        n_seqs, max_new, n_heads, n_tokens, scale, n_splits, part_o, part_ml, out, stream)
+        n_seqs, max_new, n_heads, n_tokens, scale, window, sink, n_splits, part_o, part_ml, out, stream)
     RI_LATENT(64, 32); RI_LATENT(64, 64); RI_LATENT(128, 32); RI_LATENT(128, 64);
     RI_LATENT(256, 32); RI_LATENT(256, 64); RI_LATENT(512, 32); RI_LATENT(512, 64);
 #undef RI_LATENT

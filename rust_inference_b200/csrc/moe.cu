@@ -9,7 +9,8 @@
 //             Optionally one more number per token: sigmoid(w_gate . h), the gate of a shared expert.
 //             Other forms: (`form` bit 0) s = softmax(W_router h) over all experts instead of the sigmoid; (bit 2) a
 //             group ranks by its largest c alone; no correction (a null pointer: c = s); and
-//             (bit 1) the weights are the taken s as they are, not divided by their sum.
+//             (bit 1) the weights are the taken s as they are, not divided by their sum; a bias (a pointer that may be null) is
+//             added to W_router h before the sigmoid or softmax.
 //   arrange   the (token, choice) pairs listed expert by expert, cut into tiles of rows that belong
 //             to one expert
 //   experts   the grouped contractions on the FFMA pipe with float32 accumulation, any sizes:
@@ -75,7 +76,7 @@ template <> __device__ __forceinline__ void load4_f32<__nv_bfloat16>(const __nv_
 // ticket reads all sums back and makes the token's choice.
 template <typename T, bool VEC, int TOK>
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
-moe_route_kernel(const T* x, const float* __restrict__ router, const float* __restrict__ correction,
+moe_route_kernel(const T* x, const float* __restrict__ router, const float* __restrict__ correction, const float* __restrict__ bias,
                  const float* __restrict__ gate_w, int* __restrict__ ids, float* __restrict__ weights,
                  float* __restrict__ gate_out, int n_tokens, int width, int experts, int top, int groups, int keep,
                  int per_block, int form, float* split_sums, int* split_count) {
@@ -94,6 +95,7 @@ moe_route_kernel(const T* x, const float* __restrict__ router, const float* __re
     const int row_lo = split ? (int)blockIdx.y * rows_each : 0, row_hi = split ? min(n_rows, row_lo + rows_each) : n_rows;
     // what a row's sum becomes: the score (or, for the softmax, the logit) and the choice score; the gate's sigmoid
     auto place = [&](int k, int e, float a) {
+        if (bias != nullptr && e < experts) a += bias[e];
         const float s = sigmoid_f32(a);
         if (e < experts) {
             smem[k * stride + e] = (form & 1) ? a : s;           // softmax: the logit, turned into a score below
@@ -403,10 +405,10 @@ __global__ void moe_combine_kernel(float* residual, const float* y, const float*
 }  // namespace
 
 // form: bit 0 softmax scores instead of sigmoid ones, bit 1 weights not divided by their sum, bit 2 a group counts by its
-// largest score instead of the sum of its two largest.  correction may be null.
+// largest score instead of the sum of its two largest.  correction and bias may be null.
 // split > 1 (steps of up to ROUTE_SPLIT_TOKENS tokens): the router's rows are cut over that many blocks per token;
 // split_sums: float32 [n_tokens, experts + 1] scratch, split_count: int32 [n_tokens], zero before the call and after it.
-RI_API int ri_moe_route(const void* x, int dtype, const float* router, const float* correction, const float* gate_w,
+RI_API int ri_moe_route(const void* x, int dtype, const float* router, const float* correction, const float* bias, const float* gate_w,
                         int* ids, float* weights, float* gate_out, int n_tokens, int width, int experts, int top,
                         int groups, int keep, int form, int split, float* split_sums, int* split_count,
                         cudaStream_t stream) {
@@ -427,7 +429,7 @@ RI_API int ri_moe_route(const void* x, int dtype, const float* router, const flo
                      (gate_w == nullptr || (uintptr_t)gate_w % 16 == 0);
     cudaError_t e;
 #define RI_ROUTE_N(T, V, N) launch_dependent(moe_route_kernel<T, V, N>, blocks, ROUTE_WARPS * 32, smem, stream, (const T*)x, \
-                                             router, correction, gate_w, ids, weights, gate_out, n_tokens, width, experts, top,   \
+                                             router, correction, bias, gate_w, ids, weights, gate_out, n_tokens, width, experts, top,   \
                                              groups, keep, per_block, form, split_sums, split_count)
 #define RI_ROUTE(T, V) (per_block == 1 ? RI_ROUTE_N(T, V, 1) : per_block == 2 ? RI_ROUTE_N(T, V, 2) : RI_ROUTE_N(T, V, ROUTE_TOKENS))
     if (dtype == RI_F32) e = vec ? RI_ROUTE(float, true) : RI_ROUTE(float, false);

@@ -91,6 +91,20 @@ class StepContext:
     def zeroed_buffer(self, name: str, shape, dtype: torch.dtype) -> torch.Tensor:
         return self.workspace.get_zeroed(name, shape, dtype)
 
+    # A layer may leave the end of its work (an object with `apply(stream)`) to the layer after it, whose first pass over
+    # the stream takes it along.
+    def leave_pending(self, work) -> None:
+        self.extras["pending"] = work
+
+    def take_pending(self):
+        return self.extras.pop("pending", None)
+
+    def settle(self, stream: torch.Tensor) -> None:
+        """Finish what the layer before has left, because something other than a layer looks at the stream now."""
+        work = self.take_pending()
+        if work is not None:
+            work.apply(stream)
+
 
 _pack = None
 

@@ -81,6 +81,8 @@ class DecoderModel:
         self.spec = spec
         self.dtype = dtype
         self.device = torch.device(device)
+        if spec.streams < 1 or (spec.streams > 1 and spec.stream_parts):
+            raise ValueError(f"{spec.streams} parallel streams (at least one; more than one without parts that act on a single stream)")
         kw = dict(hidden_size=spec.hidden_size, dtype=dtype, device=device)
         self._embedding_spec, self._head_spec = spec.embedding_part(), spec.head_part()
         self.embedding = _build("embedding", self._embedding_spec, **kw)
@@ -228,20 +230,25 @@ class DecoderModel:
     # ---- the step --------------------------------------------------------------
     def forward(self, ctx, cache, logits_out: torch.Tensor | None = None, probe: "LayerProbe | None" = None):
         """Run the step's tokens: the embedding part fills the float32 hidden stream, the scheduled
-        layers add to it, the head part turns the wanted rows into float32 logits [wanted rows, vocab]
+        layers add to it (several streams: [T, streams * hidden], a token's streams side by side), the head part turns the wanted rows into float32 logits [wanted rows, vocab]
         (None when nothing is wanted).  `probe` (a debugging aid, never inside a captured step)
         records statistics of the hidden state after every layer."""
-        residual = ctx.buffer("residual", (ctx.n_tokens, self.spec.hidden_size), torch.float32)
+        streams = self.spec.streams
+        residual = ctx.buffer("residual", (ctx.n_tokens, streams * self.spec.hidden_size), torch.float32)
+        ctx.take_pending()                       # of a step that did not finish
         self.embedding.forward(ctx, residual)
         for part in self.stream_parts:
             part.begin(residual, ctx)
         for run, (layer, cache_index, writes) in enumerate(self.schedule):
             before = self._before[run]
             if before is not None:
+                ctx.settle(residual)
                 self.stream_parts[before[0]].forward(residual, ctx, before[1])
             self.layers[layer].block.forward(residual, ctx, cache.layer(cache_index), writes)
             if probe is not None:
-                probe.record(f"L{run}", residual)
+                ctx.settle(residual)
+                probe.record(f"L{run}", residual if streams == 1 else residual.view(len(residual), streams, -1).sum(dim=1))
+        ctx.settle(residual)
         if probe is not None:
             normed = self.head.normalised(residual, torch.tensor(probe.rows, dtype=torch.int32, device=self.device))
             if normed is not None:

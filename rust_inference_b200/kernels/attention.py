@@ -191,10 +191,11 @@ def latent_splits(n_ctas: int, longest: int, tile_rows: int) -> int:
     return max(1, min(most, per_sm * _sm_count() // max(1, n_ctas), -(-longest // LATENT_TILE_KEYS)))
 
 
-def latent_attention(q_wide, cache_layer, out, ctx, *, n_heads, key_dim, rank, scale):
+def latent_attention(q_wide, cache_layer, out, ctx, *, n_heads, key_dim, rank, scale, window=0, sink=None):
     """Attention of n_heads query heads over ONE kv head whose keys are the cached rows [key_dim] and whose
     values are the rows' first `rank` channels (no storage of their own); causal.  q_wide is
-    [T, n_heads * key_dim]; out is head-major, [n_heads, T, rank].  bfloat16 with a latent the tensor-core kernel
+    [T, n_heads * key_dim]; out is head-major, [n_heads, T, rank].  `window`: only the last so many positions (0: all);
+    `sink` (float32 [n_heads]): one more term exp(sink_h) in the softmax's denominator.  bfloat16 with a latent the tensor-core kernel
     is built for: `latent_attention_mma` (steps of few rows cut the keys into runs); anything else: the generic
     kernel."""
     rd = key_dim - rank
@@ -205,6 +206,8 @@ def latent_attention(q_wide, cache_layer, out, ctx, *, n_heads, key_dim, rank, s
         tiles = -(-rows // tile_rows)
         # a decode step's grid may depend on the batch size and the cache geometry only (captured steps)
         longest = ctx.page_table.shape[1] * ctx.page_size if ctx.all_single else ctx.max_len
+        if window:                        # the positions that a tile of rows sees
+            longest = min(longest, window + -(-tile_rows // n_heads) + LATENT_TILE_KEYS)
         splits = latent_splits(tiles * ctx.n_seqs, longest, tile_rows)
         part_o = part_ml = None
         if splits > 1:
@@ -212,8 +215,8 @@ def latent_attention(q_wide, cache_layer, out, ctx, *, n_heads, key_dim, rank, s
             part_ml = ctx.buffer("latent_part_ml", (n * n_heads * splits * 2,), torch.float32)
         return ops.latent_attention_mma(q_wide, cache_layer.k, ctx.page_table, ctx.seq_slot, ctx.seq_start, ctx.cu_seqlens,
                                         out, n_seqs=ctx.n_seqs, max_new=ctx.max_new, n_heads=n_heads, rank=rank, rot_dim=rd,
-                                        scale=scale, n_splits=splits, part_o=part_o, part_ml=part_ml)
+                                        scale=scale, window=window, sink=sink, n_splits=splits, part_o=part_o, part_ml=part_ml)
     return ops.attention_generic(
         q_wide, q_wide.shape[1], cache_layer.k, cache_layer.k, ctx.page_table, ctx.token_pos, ctx.token_seq,
         ctx.seq_slot, out, n_tokens=q_wide.shape[0], n_heads=n_heads, n_kv_heads=1, head_dim=key_dim,
-        page_size=ctx.page_size, scale=scale, v_head_dim=rank, values_in_keys=True, head_major=True)
+        page_size=ctx.page_size, scale=scale, window=window, sink=sink, v_head_dim=rank, values_in_keys=True, head_major=True)

@@ -36,6 +36,7 @@ MODULES = {
     "latent": "latent.cu",
     "latent_attention_mma": "latent_attention_mma.cu",
     "stream": "stream.cu",
+    "parallel_streams": "parallel_streams.cu",
     "state_scan": "state_scan.cu",
     "short_conv": "short_conv.cu",
     "wait_probe": "wait_probe.cu",

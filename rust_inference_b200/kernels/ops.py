@@ -164,14 +164,15 @@ def timeline_read(strict: bool = True) -> list:
 
 # ----------------------------------------------------------------------------
 def embed_gather(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, scale: float = 1.0) -> torch.Tensor:
-    """out[t, :] = table[ids[t], :] * scale, widened to float32 first.  ids: int32 [T]; out: float32 [T, H]."""
+    """out[t, :] = table[ids[t], :] * scale, widened to float32 first.  ids: int32 [T]; out: float32 [T, H], or
+    [T, S * H]: S copies of the row side by side."""
     _need_cuda(table, ids, out)
-    n, hidden = out.shape
+    n, hidden = out.shape[0], table.shape[1]
     _need(ids.dtype == torch.int32 and ids.numel() == n, "embed_gather: ids must be int32 [T]")
     _need(out.dtype == torch.float32 and out.is_contiguous() and table.is_contiguous()
-          and table.shape[1] == hidden, "embed_gather: bad out/table")
+          and out.shape[1] % hidden == 0, "embed_gather: bad out/table")
     _call("elementwise", "ri_embed_gather", _p(table), c_int(dtype_code(table.dtype)), _p(ids), _p(out),
-          c_int(n), c_int(hidden), c_float(scale), _stream())
+          c_int(n), c_int(hidden), c_int(out.shape[1] // hidden), c_float(scale), _stream())
     return out
 
 
@@ -228,11 +229,13 @@ def layernorm(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tens
 def rope_normed_cache_write(qkv: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor, q_weight, k_weight, eps: float,
                             token_pos, token_seq, seq_slot, page_table: torch.Tensor, kcache, vcache, *, n_heads: int,
                             n_kv_heads: int, head_dim: int, page_size: int, style: int, write_kv: bool,
-                            rot_dims: int | None = None, v_head_dim: int | None = None, values_from_keys: bool = False) -> None:
+                            rot_dims: int | None = None, v_head_dim: int | None = None, values_from_keys: bool = False,
+                            value_mix: tuple | None = None) -> None:
     """`rope_cache_write` for heads that are RMS-normalised before they are rotated: every q head times
     q_weight / rms (float32 [head_dim], shared by the heads; None: not normalised), every k head likewise
     with k_weight.  With values_from_keys qkv holds no values: the cache's values are the key heads as
-    projected, before norm and rotation."""
+    projected, before norm and rotation.  value_mix = (lambda float32 [1], other [T, .] in the run dtype, column): the
+    values that go into the cache are (1 - lambda) v + lambda other[:, column : column + n_kv_heads * v_head_dim]."""
     _need_cuda(qkv, cos, sin, q_weight, k_weight, token_pos, token_seq, seq_slot, page_table, kcache, vcache)
     n = qkv.shape[0]
     rot = head_dim if rot_dims is None else int(rot_dims)
@@ -252,11 +255,19 @@ def rope_normed_cache_write(qkv: torch.Tensor, cos: torch.Tensor, sin: torch.Ten
               and vcache.is_contiguous(), "rope_normed_cache_write: cache dtype/layout")
         _need(tuple(kcache.shape[1:]) == (n_kv_heads, page_size, head_dim)
               and tuple(vcache.shape[1:]) == (n_kv_heads, page_size, v_hd), "rope_normed_cache_write: cache shape")
+    lam = other = None
+    if value_mix is not None:
+        lam, rows, col = value_mix
+        _need_cuda(lam, rows)
+        _need(not values_from_keys and lam.dtype == torch.float32 and lam.numel() == 1 and rows.dtype == qkv.dtype and rows.dim() == 2
+              and rows.is_contiguous() and rows.shape[0] >= n and 0 <= col and rows.shape[1] >= col + n_kv_heads * v_hd,
+              "rope_normed_cache_write: the values to blend in")
+        other = rows[:, col:]
     _call("elementwise", "ri_rope_normed_cache_write", _p(qkv), c_int(dtype_code(qkv.dtype)), c_int(qkv.shape[1]),
           _p(cos), _p(sin), _p(q_weight), _p(k_weight), c_float(eps), _p(token_pos), _p(token_seq), _p(seq_slot),
           _p(page_table), c_int(page_table.shape[1]), _p(kcache), _p(vcache), c_int(n), c_int(n_heads), c_int(n_kv_heads),
           c_int(head_dim), c_int(page_size), c_int(style), c_int(1 if write_kv else 0), c_int(rot if rot else -1), c_int(v_hd),
-          c_int(1 if values_from_keys else 0), _stream())
+          c_int(1 if values_from_keys else 0), _p(lam), _p(other), c_int(0 if other is None else other.stride(0)), _stream())
 
 
 def rope_cache_write(qkv: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor, token_pos, token_seq,
@@ -784,20 +795,23 @@ def moe_route(x: torch.Tensor, router: torch.Tensor, correction: torch.Tensor | 
               weights: torch.Tensor, *, top: int, groups: int = 1, keep: int = 1,
               gate_weight: torch.Tensor | None = None, gate_out: torch.Tensor | None = None,
               softmax: bool = False, normalise: bool = True, split: int = 1, split_sums: torch.Tensor | None = None,
-              split_count: torch.Tensor | None = None, group_max: bool = False) -> None:
+              split_count: torch.Tensor | None = None, group_max: bool = False, bias: torch.Tensor | None = None) -> None:
     """Per token the `top` experts with the largest sigmoid(router x) + correction among the `keep` best of
     `groups` groups (a group's score: the sum of its two largest, or with group_max its largest alone; correction None:
     zero), ids int32 [T, top], and their weights
     float32 [T, top] (the plain sigmoid scores, normalised).  gate_weight float32 [width]: gate_out[t] =
     sigmoid(gate_weight . x_t) as well.  softmax: the scores are softmax(router x) over all experts instead of
-    sigmoids; normalise False: the weights are the chosen scores as they are.  split > 1 (steps of fewer than 296
+    sigmoids; normalise False: the weights are the chosen scores as they are.  bias float32 [experts]: added to
+    router x before the sigmoid or softmax.  split > 1 (steps of fewer than 296
     tokens): the router's rows are cut over that many blocks per token, which leave their sums in split_sums (float32
     [T, experts + 1]) and count themselves in split_count (int32 [T], zero before the call and after it)."""
-    _need_cuda(x, router, correction, ids, weights, gate_weight, gate_out)
+    _need_cuda(x, router, correction, ids, weights, gate_weight, gate_out, bias)
     n, width = x.shape
     experts = router.shape[0]
     _need(x.is_contiguous() and router.dtype == torch.float32 and router.is_contiguous() and router.shape[1] == width
           and (correction is None or (correction.dtype == torch.float32 and correction.numel() == experts)), "moe_route: router and correction")
+    if bias is not None:
+        _f32_vec(bias, experts, "moe_route: bias")
     _need(ids.dtype == torch.int32 and ids.is_contiguous() and ids.numel() >= n * top and weights.dtype == torch.float32
           and weights.is_contiguous() and weights.numel() >= n * top, "moe_route: ids int32 and weights float32 [T, top]")
     _need((gate_weight is None) == (gate_out is None), "moe_route: gate weight and output go together")
@@ -809,7 +823,7 @@ def moe_route(x: torch.Tensor, router: torch.Tensor, correction: torch.Tensor | 
         _need(n < 296 and split_sums is not None and split_sums.dtype == torch.float32 and split_sums.is_contiguous()
               and split_sums.numel() >= n * (experts + 1) and split_count is not None and split_count.dtype == torch.int32
               and split_count.numel() >= n, "moe_route: rows cut over blocks need few tokens, float32 sums and int32 counters")
-    _call("moe", "ri_moe_route", _p(x), c_int(dtype_code(x.dtype)), _p(router), _p(correction), _p(gate_weight), _p(ids),
+    _call("moe", "ri_moe_route", _p(x), c_int(dtype_code(x.dtype)), _p(router), _p(correction), _p(bias), _p(gate_weight), _p(ids),
           _p(weights), _p(gate_out), c_int(n), c_int(width), c_int(experts), c_int(top), c_int(groups), c_int(keep),
           c_int((1 if softmax else 0) | (0 if normalise else 2) | (4 if group_max else 0)), c_int(max(1, split)), _p(split_sums if split > 1 else None),
           _p(split_count if split > 1 else None), _stream())
@@ -975,13 +989,18 @@ def latent_attention_mma_tile_rows(rows: int, rank: int) -> int:
 
 def latent_attention_mma(q_wide: torch.Tensor, cache: torch.Tensor, page_table, seq_slot, seq_start, cu_seqlens,
                          out: torch.Tensor, *, n_seqs: int, max_new: int, n_heads: int, rank: int, rot_dim: int, scale: float,
-                         n_splits: int = 1, part_o: torch.Tensor | None = None, part_ml: torch.Tensor | None = None) -> torch.Tensor:
+                         window: int = 0, sink: torch.Tensor | None = None, n_splits: int = 1, part_o: torch.Tensor | None = None,
+                         part_ml: torch.Tensor | None = None) -> torch.Tensor:
     """Causal attention of n_heads query heads over one cached row per position on the tensor cores (bfloat16):
     q_wide [T, n_heads * (rank + rot_dim)], cache [pages, 1, 64, rank + rot_dim] (keys: the rows; values: their
-    first `rank` channels), out head-major [n_heads, T, rank].  n_splits > 1 cuts every sequence's keys into runs
+    first `rank` channels), out head-major [n_heads, T, rank].  window > 0: only the last so many positions; sink (float32
+    [n_heads]): one more term exp(sink_h) in the softmax's denominator.  n_splits > 1 cuts every sequence's keys into runs
     whose partial results (part_o float32 [T * n_heads * n_splits * rank], part_ml float32 [T * n_heads * n_splits
     * 2]) a second kernel merges."""
-    _need_cuda(q_wide, cache, page_table, seq_slot, seq_start, cu_seqlens, out, part_o, part_ml)
+    _need_cuda(q_wide, cache, page_table, seq_slot, seq_start, cu_seqlens, out, part_o, part_ml, sink)
+    _need(window >= 0, "latent_attention: a window is not negative")
+    if sink is not None:
+        _f32_vec(sink, n_heads, "latent_attention: sink")
     n = q_wide.shape[0]
     wide = rank + rot_dim
     _need(q_wide.dtype == torch.bfloat16 and cache.dtype == torch.bfloat16 and out.dtype == torch.bfloat16
@@ -994,7 +1013,7 @@ def latent_attention_mma(q_wide: torch.Tensor, cache: torch.Tensor, page_table, 
               "latent_attention: scratch for the runs' partial results")
     _call("latent_attention_mma", "ri_latent_attention_mma", _p(q_wide), _p(cache), _p(page_table), c_int(page_table.shape[1]),
           _p(seq_slot), _p(seq_start), _p(cu_seqlens), c_int(n_seqs), c_int(max_new), c_int(n_heads), c_int(n), c_int(rank),
-          c_int(rot_dim), c_float(scale), c_int(n_splits), _p(part_o), _p(part_ml), _p(out), _stream())
+          c_int(rot_dim), c_float(scale), c_int(window), _p(sink), c_int(n_splits), _p(part_o), _p(part_ml), _p(out), _stream())
     if n_splits > 1:
         global _launches
         _launches += 1                       # the merge is a kernel of its own
@@ -1056,6 +1075,43 @@ def stream_update(stream_x: torch.Tensor, *, branch=None, branch_bias=None, post
     _call("stream", "ri_stream_update", _p(stream_x), _p(branch), _p(branch_bias), _p(pw), _p(pb), _p(pa), _p(history),
           _p(depth_w), c_int(depth_index), c_int(1 if store_result else 0), _p(nw), _p(nb), _p(na),
           _p(next_out if next_norm is not None else None), c_int(next_dtype), c_int(t), c_int(n), _stream())
+
+
+MAX_STREAMS = 16             # parallel streams `streams_step` takes
+
+
+def streams_step(x: torch.Tensor, streams: int, *, branch=None, scale=None, mix=None, write=None, read=None, norm=None,
+                 eps: float = 0.0, out=None, rows=None) -> None:
+    """One pass over `streams` parallel hidden streams x (float32 [T, streams * n], a token's streams side by side).  With
+    `branch` (float32 [T, n], left zeroed): x_t <- sum_s mix[s, t] x_s + write[t] * branch * scale, all streams at once from
+    the old ones (mix float32 [from, to], write float32 [streams], scale float32 [n] or None).  With `out`:
+    out = u / sqrt(mean(u^2) + eps) * norm of u = sum_s read[s] x_s, the streams as just written (read None: the plain sum;
+    norm None: u itself); `rows` (int32, without a branch) picks the tokens that are read."""
+    _need_cuda(x, branch, scale, mix, write, read, norm, out, rows)
+    t = x.shape[0]
+    _need(x.dtype == torch.float32 and x.is_contiguous() and x.shape[1] % streams == 0, "streams_step: x must be float32 [T, streams * n]")
+    n = x.shape[1] // streams
+    if branch is not None:
+        _need(branch.dtype == torch.float32 and branch.is_contiguous() and tuple(branch.shape) == (t, n) and rows is None,
+              "streams_step: branch must be float32 [T, n], without chosen rows")
+        _f32_vec(mix, streams * streams, "streams_step: mix"); _f32_vec(write, streams, "streams_step: write")
+        if scale is not None:
+            _f32_vec(scale, n, "streams_step: scale")
+    n_rows, dtype = t, RI_F32
+    if out is not None:
+        n_rows = out.shape[0]
+        _need(out.is_contiguous() and out.shape[1] == n, "streams_step: out must be [rows, n]")
+        dtype = dtype_code(out.dtype)
+        if rows is not None:
+            _need(rows.dtype == torch.int32 and rows.numel() == n_rows, "streams_step: rows must be int32 [R]")
+        else:
+            _need(n_rows == t, "streams_step: out has a row per token")
+    if read is not None:
+        _f32_vec(read, streams, "streams_step: read")
+    if norm is not None:
+        _f32_vec(norm, n, "streams_step: norm")
+    _call("parallel_streams", "ri_streams_step", _p(x), _p(branch), _p(scale), _p(mix), _p(write), _p(read), _p(norm), c_float(eps),
+          _p(rows), _p(out), c_int(dtype), c_int(n_rows), c_int(streams), c_int(n), _stream())
 
 
 def normed_sum(members: list, out: torch.Tensor, eps: float, accumulate: bool = False, clear: torch.Tensor | None = None) -> torch.Tensor:

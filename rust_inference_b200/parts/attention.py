@@ -41,12 +41,15 @@ class GQAttention(Mixer):
     # per channel right after the projection and its bias (so many taps, no activation; `names`: q_conv, k_conv, v_conv,
     # [channels, taps], the last column the current token's); the projection's last conv - 1 rows, biases included, are a
     # state of the sequence beside its keys and values.  `fixed_sink`: a sink that is the same number for every head and
-    # no tensor.
+    # no tensor.  `qk_norm_weights` False: the heads' norm has no weights (with a rotation that keeps lengths it is then
+    # the same before and after it).  `value_mix`: the layer's values are blended with those of another layer of the same
+    # step, v <- (1 - lambda) v + lambda v_first: "first" is the layer whose projected values are kept for the others (its own stay
+    # as they are), "mixed" one that blends them in with its learned number lambda (`names`: value_mix); what is cached is blended.
     _NAMES = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o": "o_proj.weight",
               "q_bias": "q_proj.bias", "k_bias": "k_proj.bias", "v_bias": "v_proj.bias",
               "q_norm": "q_norm.weight", "k_norm": "k_norm.weight", "o_bias": "o_proj.bias", "sink": "sinks",
               "gate": "gate_proj.weight", "r1": "distance_r1", "r2": "distance_r2", "out_gate": "out_gate_proj.weight",
-              "q_conv": "q_conv1d.weight", "k_conv": "k_conv1d.weight", "v_conv": "v_conv1d.weight"}
+              "q_conv": "q_conv1d.weight", "k_conv": "k_conv1d.weight", "v_conv": "v_conv1d.weight", "value_mix": "value_mix"}
 
     def __init__(self, *, n_heads: int, n_kv_heads: int, head_dim: int, qkv_bias: bool,
                  position: PartSpec, window: int | None = None, v_head_dim: int | None = None,
@@ -54,8 +57,8 @@ class GQAttention(Mixer):
                  names: dict | None = None, qk_norm_eps: float | None = None, values_from_keys: bool = False,
                  softcap: float = 0.0, distance_bias: bool = False, keep_first: int = 0, sink: bool = False,
                  head_gate: bool = False, o_bias: bool = False, own_kv: bool = True, out_gate: bool = False,
-                 conv: int | None = None, fixed_sink: float | None = None,
-                 hidden_size: int, dtype, device):
+                 conv: int | None = None, fixed_sink: float | None = None, qk_norm_weights: bool = True,
+                 value_mix: str | None = None, hidden_size: int, dtype, device):
         super().__init__(hidden_size=hidden_size, dtype=dtype, device=device)
         if n_heads % n_kv_heads:
             raise ValueError(f"{n_heads} heads are not a multiple of {n_kv_heads} kv heads")
@@ -69,6 +72,12 @@ class GQAttention(Mixer):
         if window is not None and window <= 0:
             raise ValueError(f"a window holds at least one position, found {window}")
         self.qk_norm_eps = None if qk_norm_eps is None else float(qk_norm_eps)
+        self.qk_norm_weights = bool(qk_norm_weights)
+        if value_mix not in (None, "first", "mixed"):
+            raise ValueError(f"value_mix must be 'first' or 'mixed', found {value_mix!r}")
+        if value_mix is not None and (values_from_keys or not own_kv or qkv_bias or conv is not None):
+            raise ValueError("blended values go with value projections of the layer's own, without biases and convolutions")
+        self.value_mix, self.value_lambda = value_mix, None
         self.q_dim, self.kv_dim = n_heads * head_dim, n_kv_heads * head_dim
         self.v_dim, self.o_dim = n_kv_heads * self.v_head_dim, n_heads * self.v_head_dim
         self.qkv_bias = bool(qkv_bias)
@@ -139,7 +148,9 @@ class GQAttention(Mixer):
         if self.conv is not None:
             for name, rows in (("q_conv", self.q_dim), ("k_conv", self.kv_dim), ("v_conv", self.v_dim)):
                 specs[nm[name]] = TensorSpec((rows, self.conv), role="vector")
-        if self.qk_norm_eps is not None:
+        if self.value_mix == "mixed":
+            specs[nm["value_mix"]] = TensorSpec((), role="vector", init="zeros")
+        if self.qk_norm_eps is not None and self.qk_norm_weights:
             specs[nm["q_norm"]] = TensorSpec((self.head_dim,), role="vector", init="ones")
             specs[nm["k_norm"]] = TensorSpec((self.head_dim,), role="vector", init="ones")
         if self.qkv_bias:
@@ -173,7 +184,11 @@ class GQAttention(Mixer):
         if self.o_bias:
             self.b_o = tensors[nm["o_bias"]].contiguous()
             self.b_o_scaled = self.b_o if self.out_scale == 1.0 else self.b_o * self.out_scale
-        if self.qk_norm_eps is not None:
+        if self.value_mix == "mixed":
+            self.value_lambda = tensors[nm["value_mix"]].reshape(1).contiguous()
+        if self.qk_norm_eps is not None and not self.qk_norm_weights:
+            self.q_norm = self.k_norm = torch.ones(self.head_dim, dtype=torch.float32, device=self.device)
+        elif self.qk_norm_eps is not None:
             self.q_norm, self.k_norm = tensors[nm["q_norm"]].contiguous(), tensors[nm["k_norm"]].contiguous()
         if self.qkv_bias:
             biases = [tensors[nm["q_bias"]]] + ([tensors[nm["k_bias"]], tensors[nm["v_bias"]]] if self.own_kv else [])
@@ -203,7 +218,9 @@ class GQAttention(Mixer):
             out[nm["r1"]], out[nm["r2"]] = self.dist[0], self.dist[1]
         if self.o_bias:
             out[nm["o_bias"]] = self.b_o
-        if self.qk_norm_eps is not None:
+        if self.value_mix == "mixed":
+            out[nm["value_mix"]] = self.value_lambda.reshape(())
+        if self.qk_norm_eps is not None and self.qk_norm_weights:
             out[nm["q_norm"]], out[nm["k_norm"]] = self.q_norm, self.k_norm
         if self.conv is not None:
             taps = self.w_conv.t()
@@ -264,7 +281,7 @@ class GQAttention(Mixer):
         kv_width = (self.kv_dim + (0 if self.values_from_keys else self.v_dim)) if self.own_kv else 0
         gate_col = self.q_dim + kv_width
         width = self.w_qkv.n                           # with gates: one more column per head, padded to a multiple of 8
-        special = self.values_from_keys or self.qk_norm_eps is not None
+        special = self.values_from_keys or self.qk_norm_eps is not None or self.value_mix is not None
         usual = (self.v_head_dim == self.head_dim and not getattr(self.position, "partial", False) and not special
                  and not self.extended)
         from_acc = getattr(self.position, "apply_and_store_from_accumulators", None) if usual else None
@@ -277,9 +294,17 @@ class GQAttention(Mixer):
             from_acc(acc, self.b_qkv, qkv, ctx, cache_layer, n_heads=self.n_heads, n_kv_heads=self.n_kv_heads,
                      head_dim=self.head_dim, write_kv=writes_cache)
         else:
-            qkv = ctx.buffer("qkv", (n, width), self.dtype)
+            # values that later layers of the step blend in stay where they were projected: in a buffer that layers do not share
+            qkv = ctx.buffer("qkv" if self.value_mix != "first" else "qkv_first_values", (n, width), self.dtype)
             linear.project(x, self.w_qkv, qkv, ctx, bias=self.b_qkv)
             extra = {} if usual else {"v_head_dim": self.v_head_dim}
+            if self.value_mix == "first":
+                ctx.extras["first_values"] = (qkv, self.q_dim + self.kv_dim, self.v_dim)
+            elif self.value_mix == "mixed":
+                first = ctx.extras.get("first_values")
+                if first is None or first[0].shape[0] != n or first[2] != self.v_dim:
+                    raise RuntimeError("blended values: no layer before this one has kept values of the same size in this step")
+                extra["value_mix"] = (self.value_lambda, first[0], first[1])
             if special:
                 # norm of the heads, rotation and cache write as one kernel (the position encoding's)
                 self.position.apply_normed_and_store(

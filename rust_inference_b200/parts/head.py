@@ -1,7 +1,7 @@
 """The output head: final norm, then logits = W h in float32, on the wanted rows only
 (transformer.rs:89, :97).  The matrix is the embedding's when the model ties them: the same
 storage, where the reference clones it (model.rs:221-226).  `scale`: logits = scale * W h (with the final norm where that can
-take the factor, otherwise on the logits).  `softcap` > 0: logits <- softcap * tanh(logits / softcap)."""
+take the factor, otherwise on the logits).  Of several parallel streams the head reads the sum.  `softcap` > 0: logits <- softcap * tanh(logits / softcap)."""
 from __future__ import annotations
 
 import torch
@@ -57,18 +57,34 @@ class LinearHead(Head):
     def matrix_bytes(self):
         return self.weight.t.numel() * self.weight.t.element_size()
 
+    def _normed(self, residual, out, rows, factor=None, ctx=None):
+        """out = the norm of the stream's (or the streams' summed) rows, times `factor` where one is given."""
+        streams = residual.shape[1] // self.hidden_size
+        if streams == 1:
+            if factor is None:
+                self.norm.forward(residual, out, rows=rows)
+            else:
+                self.norm.forward_times(factor, residual, out, rows=rows)
+            return
+        weight = getattr(self.norm, "factor", None)
+        if weight is not None and factor is None:               # an RMS norm: sum and norm in one pass
+            ops.streams_step(residual, streams, norm=weight, eps=self.norm.eps, out=out, rows=rows)
+            return
+        shape = tuple(out.shape)
+        plain = (torch.empty(shape, dtype=torch.float32, device=out.device) if ctx is None
+                 else ctx.buffer("head_streams", shape, torch.float32))
+        ops.streams_step(residual, streams, out=plain, rows=rows)
+        self._normed(plain, out, None, factor)
+
     def normalised(self, residual, rows):
         out = torch.empty((rows.numel(), self.hidden_size), dtype=self.dtype, device=residual.device)
-        self.norm.forward(residual, out, rows=rows)
+        self._normed(residual, out, rows)
         return out
 
     def forward(self, residual, ctx, logits_out=None):
         normed = ctx.buffer("head_in", (ctx.n_logit_rows, self.hidden_size), self.dtype)
         with_norm = self.scale != 1.0 and hasattr(self.norm, "forward_times")
-        if with_norm:
-            self.norm.forward_times(self.scale, residual, normed, rows=ctx.logit_rows)
-        else:
-            self.norm.forward(residual, normed, rows=ctx.logit_rows)
+        self._normed(residual, normed, ctx.logit_rows, self.scale if with_norm else None, ctx)
         if logits_out is None:
             logits_out = torch.empty((ctx.n_logit_rows, self.vocab_size), dtype=torch.float32, device=residual.device)
         linear.logits(normed, self.weight, logits_out, ctx)

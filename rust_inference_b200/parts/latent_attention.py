@@ -35,14 +35,16 @@ class LatentAttention(Mixer):
     channels over a latent of kv_rank channels.  `position`: the rotary encoding of the rot_dim part (its
     tables, pairing and rotated channels).  `own_latent` false: the layer has no down-projection and reads
     the cache of the layer the schedule names.  `gated`: an output gate per head.  `scale`: on the scores
-    (default 1 / sqrt(head_dim + rot_dim)).  `names`: q, dkv, dkv_norm, uk, uv, gate, o below the prefix."""
+    (default 1 / sqrt(head_dim + rot_dim)).  `window`: a query sees itself and the window - 1
+    positions before it (None: all).  `sink`: the softmax's denominator also holds exp(sink_h), a learned number per head
+    without key or value.  `names`: q, dkv, dkv_norm, uk, uv, gate, sink, o below the prefix."""
 
     _NAMES = {"q": "q_proj.weight", "dkv": "kv_a_proj.weight", "dkv_norm": "kv_a_norm.weight",
-              "uk": "k_b_proj.weight", "uv": "v_b_proj.weight", "gate": "g_proj.weight", "o": "o_proj.weight"}
+              "uk": "k_b_proj.weight", "uv": "v_b_proj.weight", "gate": "g_proj.weight", "sink": "sinks", "o": "o_proj.weight"}
 
     def __init__(self, *, n_heads: int, head_dim: int, rot_dim: int, v_head_dim: int, kv_rank: int, eps: float,
                  position: PartSpec, scale: float | None = None, own_latent: bool = True, gated: bool = True,
-                 names: dict | None = None, hidden_size: int, dtype, device):
+                 window: int | None = None, sink: bool = False, names: dict | None = None, hidden_size: int, dtype, device):
         super().__init__(hidden_size=hidden_size, dtype=dtype, device=device)
         self.n_heads, self.head_dim, self.rot_dim = int(n_heads), int(head_dim), int(rot_dim)
         self.v_head_dim, self.kv_rank = int(v_head_dim), int(kv_rank)
@@ -51,6 +53,9 @@ class LatentAttention(Mixer):
         self.eps = float(eps)
         self.scale = 1.0 / math.sqrt(float(head_dim + rot_dim)) if scale is None else float(scale)
         self.own_latent, self.gated = bool(own_latent), bool(gated)
+        if window is not None and window <= 0:
+            raise ValueError(f"a window holds at least one position, found {window}")
+        self.window, self.sink, self.sinks = window, bool(sink), None
         self.names = dict(self._NAMES, **(names or {}))
         self.position = lookup("position", position.kind)(hidden_size=hidden_size, dtype=dtype, device=device,
                                                           **position.params)
@@ -71,6 +76,8 @@ class LatentAttention(Mixer):
         specs[nm["uv"]] = TensorSpec((H * self.v_head_dim, self.kv_rank))
         if self.gated:
             specs[nm["gate"]] = TensorSpec((H, h))
+        if self.sink:
+            specs[nm["sink"]] = TensorSpec((H,), role="vector", init="zeros")
         specs[nm["o"]] = TensorSpec((h, H * self.v_head_dim))
         return specs
 
@@ -84,6 +91,8 @@ class LatentAttention(Mixer):
         if self.gated:
             mats.append(tensors[nm["gate"]])
         self.w_in = linear.Weight(torch.cat(mats, dim=0))
+        if self.sink:
+            self.sinks = tensors[nm["sink"]].contiguous()
         # Uk per head, transposed: q_lat_h = Uk_h^T q_nope_h is x W^T with W = Uk_h^T [kv_rank, head_dim]
         self.w_uk_t = tensors[nm["uk"]].view(H, self.head_dim, self.kv_rank).transpose(1, 2).contiguous()
         self.w_uv = tensors[nm["uv"]].view(H, self.v_head_dim, self.kv_rank).contiguous()
@@ -100,6 +109,8 @@ class LatentAttention(Mixer):
             at += self.wide
         if self.gated:
             out[nm["gate"]] = w[at:at + H]
+        if self.sink:
+            out[nm["sink"]] = self.sinks
         out[nm["uk"]] = self.w_uk_t.transpose(1, 2).reshape(H * self.head_dim, self.kv_rank)
         out[nm["uv"]] = self.w_uv.view(H * self.v_head_dim, self.kv_rank)
         out[nm["o"]] = self.w_o.t
@@ -109,7 +120,7 @@ class LatentAttention(Mixer):
         self.position.prepare(max_positions)
 
     def cache_request(self):
-        return KVRequest(1, self.wide, None, self.kv_rank, True)
+        return KVRequest(1, self.wide, self.window, self.kv_rank, True)
 
     # ---- the step ------------------------------------------------------------------------------------------
     def _grouped(self, x, w, out, lists, n_rows):
@@ -163,7 +174,7 @@ class LatentAttention(Mixer):
         # attention of all heads over the one cached row per position; the weighted latents head by head
         o_lat = ctx.buffer("latent_o_lat", (rows, kr), self.dtype)              # [heads, T, kv_rank]
         attn_kernels.latent_attention(q_wide, cache_layer, o_lat, ctx, n_heads=H, key_dim=self.wide, rank=kr,
-                                      scale=self.scale)
+                                      scale=self.scale, window=self.window or 0, sink=self.sinks)
         v = ctx.buffer("latent_v", (rows, vd), torch.float32)                    # [heads, T, v_head_dim]
         self._grouped(o_lat, self.w_uv, v, lists, rows)
         gated = ctx.buffer("attn_out", (n, H * vd), self.dtype)

@@ -13,6 +13,8 @@ Interfaces (see `parts.base`):
   embedding         Embedding (token ids -> hidden stream)
   head              Head (hidden stream -> logits)
   depth             DepthMix (what a layer hands on, as a function of the results of all layers so far)
+  stream_link       how a sublayer reads and writes several parallel streams (wired by an arrangement)
+  branch_scale      a vector on a sublayer's result before it joins the stream (wired by an arrangement)
   input_conv        a short convolution in front of a sublayer (wired and run by an arrangement)
   stream            StreamStep (something that happens to the whole stream between layer runs the schedule names)
 """
@@ -20,7 +22,7 @@ from __future__ import annotations
 
 _REGISTRIES: dict[str, dict] = {
     "norm": {}, "position": {}, "mixer": {}, "feed_forward": {}, "arrangement": {}, "embedding": {}, "head": {},
-    "depth": {}, "stream": {}, "input_conv": {},
+    "depth": {}, "stream": {}, "input_conv": {}, "stream_link": {}, "branch_scale": {},
 }
 
 
@@ -61,3 +63,4 @@ def _ensure_builtin() -> None:
     from . import depth, state_space, delta_rule  # noqa: F401
     from . import linear_attention, loop  # noqa: F401
     from . import input_conv, fixed_decay_attention  # noqa: F401
+    from . import streams  # noqa: F401

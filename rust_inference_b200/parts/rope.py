@@ -30,15 +30,31 @@ def interpolated_frequencies(rot_dims: int, base: float, *, factor: float, origi
     return f / np.float64(factor) * ramp + f * (1.0 - ramp), 0.1 * float(np.log(np.float64(factor))) + 1.0
 
 
+def stretched_frequencies(rot_dims: int, base: float, *, factor: float, low: float, high: float, original: float):
+    """Frequencies float64 [rot_dims / 2] of a rotation whose long waves are stretched (the form Llama 3.1 uses).  With
+    f_i = base^(-2i/rot_dims) and t_i = original f_i / (2 pi), how often the channel's wave turns over the original context:
+    f_i where t_i > high, f_i / factor where t_i < low, and between the two bounds, with s = (t_i - low) / (high - low),
+    (1 - s) f_i / factor + s f_i."""
+    f = np.power(np.float64(base), -2.0 * np.arange(rot_dims // 2, dtype=np.float64) / np.float64(rot_dims))
+    turns = np.float64(original) * f / (2.0 * np.pi)
+    s = (turns - low) / (high - low)
+    return np.where(turns > high, f, np.where(turns < low, f / factor, (1.0 - s) * f / factor + s * f))
+
+
 def rope_tables(head_dim: int, base: float, n_positions: int, exact_angles: bool = False, scaling_factor: float = 1.0,
-                interpolation: dict | None = None):
+                interpolation: dict | None = None, wave_scaling: dict | None = None):
     """cos, sin as float32 [n_positions, head_dim/2], built the way rope.rs:47-55 does:
     exponent = 2i/dim, theta = 1/base^exponent and angle = pos*theta are 32-bit numbers
     (the power is taken in float64 and rounded once); cos and sin are taken of the 32-bit
     angle in float64 and rounded once.  With exact_angles frequency and angle stay float64 and
     only cos and sin are rounded.  Every frequency is divided by scaling_factor (linear position scaling).
-    `interpolation` (factor, original, fast, slow): the frequencies and the magnitude of `interpolated_frequencies`."""
+    `interpolation` (factor, original, fast, slow): the frequencies and the magnitude of `interpolated_frequencies`.
+    `wave_scaling` (factor, low, high, original): the frequencies of `stretched_frequencies`, exact angles."""
     half = head_dim // 2
+    if wave_scaling is not None:
+        theta = stretched_frequencies(head_dim, base, **wave_scaling) / np.float64(scaling_factor)
+        angle = np.arange(n_positions, dtype=np.float64)[:, None] * theta[None, :]
+        return np.cos(angle).astype(np.float32), np.sin(angle).astype(np.float32)
     if interpolation is not None:
         # frequencies of their own per channel and a magnitude on cos and sin; angles in float64, rounded once
         theta, magnitude = interpolated_frequencies(head_dim, base, **interpolation)
@@ -68,11 +84,12 @@ class RotaryEncoding(PositionEncoding):
     the first rot_dims channels of every head (frequencies base^(-2i/rot_dims), pairs within
     them) and lets the rest pass.  `scaling_factor` divides every frequency (linear position scaling).
     `interpolation` (a dict factor, original, fast, slow): slow channels are interpolated and cos and sin get a
-    magnitude (`interpolated_frequencies`); the tables hold it, the kernels are the same."""
+    magnitude (`interpolated_frequencies`); the tables hold it, the kernels are the same.  `wave_scaling` (a dict factor, low,
+    high, original): long waves are stretched (`stretched_frequencies`)."""
 
     def __init__(self, *, head_dim: int, base: float, style: str = "half", rot_dims: int | None = None,
                  exact_angles: bool = False, scaling_factor: float = 1.0, interpolation: dict | None = None,
-                 hidden_size: int, dtype, device):
+                 wave_scaling: dict | None = None, hidden_size: int, dtype, device):
         super().__init__(hidden_size=hidden_size, dtype=dtype, device=device)
         if style not in _STYLES:
             raise ValueError(f"rope style must be one of {sorted(_STYLES)}, found {style!r}")
@@ -96,6 +113,17 @@ class RotaryEncoding(PositionEncoding):
             if not (self.interpolation["factor"] > 0 and self.interpolation["original"] > 0 and
                     self.interpolation["fast"] > 0 and self.interpolation["slow"] > 0 and self.base > 1):
                 raise ValueError(f"rope interpolation needs positive constants and a base above 1, found {interpolation}")
+        self.wave_scaling = None
+        if wave_scaling is not None:
+            missing = [k for k in ("factor", "low", "high", "original") if k not in wave_scaling]
+            if missing:
+                raise ValueError(f"rope wave scaling lacks {missing}")
+            if interpolation is not None:
+                raise ValueError("a rotation is interpolated or its long waves are stretched, not both")
+            self.wave_scaling = {k: float(wave_scaling[k]) for k in ("factor", "low", "high", "original")}
+            if not (self.wave_scaling["factor"] > 0 and self.wave_scaling["original"] > 0
+                    and self.wave_scaling["high"] > self.wave_scaling["low"]):
+                raise ValueError(f"rope wave scaling needs a positive factor and context and high above low, found {wave_scaling}")
         self.cos = self.sin = None
 
     @property
@@ -105,7 +133,7 @@ class RotaryEncoding(PositionEncoding):
     def prepare(self, max_positions: int) -> None:
         if self.cos is None or self.cos.shape[0] < max_positions:
             cos, sin = rope_tables(self.rot_dims, self.base, max_positions, self.exact_angles, self.scaling_factor,
-                                   self.interpolation)
+                                   self.interpolation, self.wave_scaling)
             self.cos = torch.from_numpy(cos).contiguous().to(self.device)
             self.sin = torch.from_numpy(sin).contiguous().to(self.device)
 
@@ -118,16 +146,17 @@ class RotaryEncoding(PositionEncoding):
                              style=self.style, write_kv=write_kv, rot_dims=self.rot_dims, v_head_dim=v_head_dim)
 
     def apply_normed_and_store(self, qkv, ctx, cache_layer, *, n_heads, n_kv_heads, head_dim, write_kv, q_weight,
-                               k_weight, eps, values_from_keys=False, v_head_dim=None):
+                               k_weight, eps, values_from_keys=False, v_head_dim=None, value_mix=None):
         """The same after an RMS norm of every q and k head (weights shared by the heads; None: no norm); with
-        values_from_keys the cached values are the keys as projected, before norm and rotation."""
+        values_from_keys the cached values are the keys as projected, before norm and rotation.  value_mix = (lambda, other, column): the
+        cached values are (1 - lambda) v + lambda other's columns from there on."""
         if self.cos is None or self.cos.shape[0] < ctx.max_len:
             raise RuntimeError("rope tables do not cover the step's positions; call prepare() first")
         ops.rope_normed_cache_write(qkv, self.cos, self.sin, q_weight, k_weight, eps, ctx.token_pos, ctx.token_seq,
                                     ctx.seq_slot, ctx.page_table, cache_layer.k, cache_layer.v, n_heads=n_heads,
                                     n_kv_heads=n_kv_heads, head_dim=head_dim, page_size=ctx.page_size, style=self.style,
                                     write_kv=write_kv, rot_dims=self.rot_dims, v_head_dim=v_head_dim,
-                                    values_from_keys=values_from_keys)
+                                    values_from_keys=values_from_keys, value_mix=value_mix)
 
     def apply_and_store_from_accumulators(self, acc, bias, q_out, ctx, cache_layer, *, n_heads, n_kv_heads,
                                           head_dim, write_kv):
@@ -156,10 +185,10 @@ class Unrotated(PositionEncoding):
                              page_size=ctx.page_size, style=0, write_kv=True, rot_dims=0, v_head_dim=v_head_dim)
 
     def apply_normed_and_store(self, qkv, ctx, cache_layer, *, n_heads, n_kv_heads, head_dim, write_kv, q_weight,
-                               k_weight, eps, values_from_keys=False, v_head_dim=None):
+                               k_weight, eps, values_from_keys=False, v_head_dim=None, value_mix=None):
         """The RMS norm of every q and k head (weights shared by the heads; None: no norm) without any rotation; keys
         and values go into the cache."""
         ops.rope_normed_cache_write(qkv, None, None, q_weight, k_weight, eps, ctx.token_pos, ctx.token_seq, ctx.seq_slot,
                                     ctx.page_table, cache_layer.k, cache_layer.v, n_heads=n_heads, n_kv_heads=n_kv_heads,
                                     head_dim=head_dim, page_size=ctx.page_size, style=0, write_kv=write_kv, rot_dims=0,
-                                    v_head_dim=v_head_dim, values_from_keys=values_from_keys)
+                                    v_head_dim=v_head_dim, values_from_keys=values_from_keys, value_mix=value_mix)

@@ -26,13 +26,15 @@ class RoutedExperts(FeedForward):
     g' sigmoid(alpha g') (u' + shift) of `bounded_glu` instead of SiLU); `shared_gate` False (the shared expert has no
     learned gate and is added as it is); `out_scale` (a factor on the part's whole result, applied in float32 as it
     joins the stream); `correction` False (no such tensor: the scores rank the experts by themselves); `group_score` "max" (a
-    group is ranked by its largest c alone instead of the sum of its two largest).
+    group is ranked by its largest c alone instead of the sum of its two largest); `router_bias` (a vector of its own added
+    to W_router x before the sigmoid or softmax: it moves the ranking and the weights alike.  Softmax scores of all experts
+    divided by the sum of the chosen ones are the softmax over the chosen logits).
 
     Everything from the router to the sum runs on the device (`csrc/moe.cu`), so decode steps stay
     inside captured graphs.  Experts are kept stacked: gate, up [experts, ff, hidden], down [experts,
     hidden, ff].  `names` gives the tensors' names below the part's prefix; "{e}" is the expert's number."""
 
-    _NAMES = {"router": "router.weight", "correction": "router.correction", "gate": "experts.{e}.gate_proj.weight",
+    _NAMES = {"router": "router.weight", "correction": "router.correction", "router_bias": "router.bias", "gate": "experts.{e}.gate_proj.weight",
               "up": "experts.{e}.up_proj.weight", "down": "experts.{e}.down_proj.weight",
               "shared_gate": "shared.gate_proj.weight", "shared_up": "shared.up_proj.weight",
               "shared_down": "shared.down_proj.weight", "shared_mix": "shared.mix.weight"}
@@ -44,12 +46,13 @@ class RoutedExperts(FeedForward):
                  shared_size: int | None = None, names: dict | None = None, router_kind: str = "sigmoid",
                  normalise: bool = True, identity: int = 0, expert_form: dict | None = None,
                  shared_form: dict | None = None, shared_gate: bool = True, out_scale: float = 1.0,
-                 correction: bool = True, group_score: str = "top2_sum", hidden_size: int, dtype, device):
+                 correction: bool = True, group_score: str = "top2_sum", router_bias: bool = False, hidden_size: int, dtype, device):
         super().__init__(hidden_size=hidden_size, dtype=dtype, device=device)
         if router_kind not in self.ROUTERS:
             raise ValueError(f"routed_experts: unknown router {router_kind!r}; known: {', '.join(self.ROUTERS)}")
         if group_score not in self.GROUP_SCORES:
             raise ValueError(f"routed_experts: unknown group score {group_score!r}; known: {', '.join(self.GROUP_SCORES)}")
+        self.has_router_bias, self.router_bias = bool(router_bias), None
         self.has_correction, self.group_max = bool(correction), group_score == "max"
         if identity < 0 or (identity and n_groups != 1):
             raise ValueError(f"{identity} experts without tensors (not negative; not combined with groups)")
@@ -87,6 +90,8 @@ class RoutedExperts(FeedForward):
         specs = {nm["router"]: TensorSpec((outputs, h), role="vector")}
         if self.has_correction:
             specs[nm["correction"]] = TensorSpec((outputs,), role="vector", init="zeros")
+        if self.has_router_bias:
+            specs[nm["router_bias"]] = TensorSpec((outputs,), role="vector", init="zeros")
         for e in range(self.n_experts):
             specs[nm["gate"].format(e=e)] = TensorSpec((f, h))
             specs[nm["up"].format(e=e)] = TensorSpec((f, h))
@@ -104,6 +109,7 @@ class RoutedExperts(FeedForward):
         nm, n = self.names, self.n_experts
         self.router = tensors[nm["router"]].contiguous()
         self.correction = tensors[nm["correction"]].contiguous() if self.has_correction else None
+        self.router_bias = tensors[nm["router_bias"]].contiguous() if self.has_router_bias else None
         self.w_gate = torch.stack([tensors[nm["gate"].format(e=e)] for e in range(n)]).contiguous()
         self.w_up = torch.stack([tensors[nm["up"].format(e=e)] for e in range(n)]).contiguous()
         self.w_down = torch.stack([tensors[nm["down"].format(e=e)] for e in range(n)]).contiguous()
@@ -117,6 +123,8 @@ class RoutedExperts(FeedForward):
         out = {nm["router"]: self.router}
         if self.has_correction:
             out[nm["correction"]] = self.correction
+        if self.has_router_bias:
+            out[nm["router_bias"]] = self.router_bias
         for e in range(self.n_experts):
             out[nm["gate"].format(e=e)] = self.w_gate[e]
             out[nm["up"].format(e=e)] = self.w_up[e]
@@ -163,7 +171,7 @@ class RoutedExperts(FeedForward):
         cut = self.route_cut(n, ctx)
         ops.moe_route(x, self.router, self.correction, ids, weights, top=top, groups=self.n_groups,
                       keep=self.group_keep, gate_weight=self.shared_mix, gate_out=gate,
-                      softmax=self.router_kind == "softmax", normalise=self.normalise, group_max=self.group_max, **cut)
+                      softmax=self.router_kind == "softmax", normalise=self.normalise, group_max=self.group_max, bias=self.router_bias, **cut)
         fast = self._on_tensor_cores(x)
         if fast:
             from ..kernels import tcgen05

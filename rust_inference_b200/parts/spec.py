@@ -91,6 +91,9 @@ class ModelSpec:
     head: PartSpec | None = None
     # parts of the category "stream" that act on the whole stream between layer runs (`ScheduleEntry.before`)
     stream_parts: tuple = ()
+    # parallel hidden streams, all equal to the embedding's output at the start and summed for the head; more than one goes
+    # with layers whose arrangement reads and writes them all
+    streams: int = 1
 
     def embedding_part(self) -> PartSpec:
         if self.embedding is not None:
@@ -128,7 +131,8 @@ class TensorSpec:
 
     role  "matrix" (kept in the run dtype), "vector" (norm weights and biases: kept in
           float32 on the device whatever they were stored as) or "table" (integers, int32);
-    init  how the random-weights mode fills it: "normal", "ones", "zeros" or "unit_last" (zeros, the last entry 1).
+    init  how the random-weights mode fills it: "normal", "ones", "zeros", "unit_last" (zeros, the last entry 1) or
+          "identity" (a square matrix with ones on its diagonal).
     """
     shape: tuple
     role: str = "matrix"
