@@ -7,6 +7,7 @@
     python bench.py --arch redodra [--arch-sizes 1k|2k|4k]     (likewise, beside a Lulisun-style model too)
     python bench.py --arch belizen [--arch-sizes 1k|2k|4k]     (likewise)
     python bench.py --arch gatarax [--arch-sizes 1k|2k|4k]     (likewise)
+    python bench.py --arch pagulix [--arch-sizes 1k|2k|4k]     (likewise)
 
 Default run: a Qwen2.5-7B-sized dense decoder (28 layers, hidden 3584, 28 heads, 4 kv
 heads, head_dim 128, intermediate 18944, vocabulary 152064, q/k/v biases, untied head)
@@ -46,6 +47,9 @@ same two (`rust_inference_b200/kernels/belizen_bench.py`).
 `--arch gatarax` does it for a Gatarax-style model (window attention with a sink and convolved projections beside a delta rule with
 decays per key channel, linear attention with fixed decays, short convolutions in front of every sublayer, routed experts) beside a
 Redodra-style model, a Lulisun-style model and a dense decoder (`rust_inference_b200/kernels/gatarax_bench.py`).
+`--arch pagulix` does it for a Pagulix-style model (latent attention over a window with sinks, attention whose values are blended across
+layers, the gated delta rule, routed experts, several parallel streams) beside a Vadodra-style, a Redodra-style and a Lulisun-style
+model and a dense decoder (`rust_inference_b200/kernels/pagulix_bench.py`).
 
 Prints ONE JSON line.  Only one GPU is used: for --gpus > 1 it says so and exits with 2.
 """
@@ -205,10 +209,10 @@ def main() -> int:
     ap.add_argument("--tokens", type=int, default=8, help="with --kernel: tokens in the step")
     ap.add_argument("--context", type=int, default=1024, help="with --kernel: cached positions per sequence")
     ap.add_argument("--once", action="store_true", help="with --kernel: launch the workload once, untimed (for ncu)")
-    ap.add_argument("--arch", default="dense", choices=["dense", "lulisun", "vadodra", "redodra", "belizen", "gatarax"],
-                    help="lulisun / vadodra / redodra / belizen / gatarax: prefill and decode throughput of a model of that design beside a dense decoder of "
+    ap.add_argument("--arch", default="dense", choices=["dense", "lulisun", "vadodra", "redodra", "belizen", "gatarax", "pagulix"],
+                    help="lulisun / vadodra / redodra / belizen / gatarax / pagulix: prefill and decode throughput of a model of that design beside a dense decoder of "
                          "equal size, kernel by kernel against the rooflines, instead of the default workload")
-    ap.add_argument("--arch-sizes", default="2k", choices=["1k", "2k", "4k"], help="with --arch lulisun / vadodra / redodra / belizen / gatarax: the layer sizes")
+    ap.add_argument("--arch-sizes", default="2k", choices=["1k", "2k", "4k"], help="with --arch lulisun / vadodra / redodra / belizen / gatarax / pagulix: the layer sizes")
     args = ap.parse_args()
 
     if args.impl == "reference":
@@ -251,6 +255,12 @@ def main() -> int:
         from rust_inference_b200.kernels import gatarax_bench
         peaks, peak_source = load_peaks()
         return gatarax_bench.main(args.arch_sizes, peaks, peak_source, prefill_tokens=max(1, args.prefill_tokens),
+                                  batch=args.batch, context=args.context if args.context != 1024 else None,
+                                  steps=max(1, min(args.steps, 64)))
+    if args.arch == "pagulix":
+        from rust_inference_b200.kernels import pagulix_bench
+        peaks, peak_source = load_peaks()
+        return pagulix_bench.main(args.arch_sizes, peaks, peak_source, prefill_tokens=max(1, args.prefill_tokens),
                                   batch=args.batch, context=args.context if args.context != 1024 else None,
                                   steps=max(1, min(args.steps, 64)))
     warmup = max(3, args.warmup)

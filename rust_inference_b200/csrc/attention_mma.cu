@@ -501,7 +501,8 @@ __device__ __forceinline__ void pv_16keys_atoms(const uint32_t* p, uint32_t vtil
     }
 }
 
-template <int HD, bool CLUSTER>
+// VD: the size of a value head; 32 takes tiles of 64 columns whose upper half the copy fills with zeros
+template <int HD, int VD, bool CLUSTER>
 __global__ void __launch_bounds__(DECODE_TMA_THREADS)
 attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                        const __nv_bfloat16* __restrict__ q, int q_ld, const int* __restrict__ page_table,
@@ -509,14 +510,15 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
                        const int* __restrict__ cu_seqlens, int n_heads, int n_kv_heads, float scale, int window,
                        int n_splits, float* __restrict__ part_o, float* __restrict__ part_ml,
                        __nv_bfloat16* __restrict__ out, int out_ld, int* status) {
-    constexpr int TILE = PAGE * HD * 2;                 // bytes of one K or V page tile
-    constexpr int ATOMS = HD / 64;
+    constexpr int ATOMS = HD / 64, V_ATOMS = (VD + 63) / 64;
+    constexpr int K_TILE = PAGE * HD * 2, V_TILE = V_ATOMS * PAGE * 128;      // bytes of a K and of a V page tile
+    constexpr int STAGE = K_TILE + V_TILE;
     extern __shared__ uint8_t smem_raw[];
     __shared__ __align__(8) uint64_t full_bar[RING], empty_bar[RING];
     __shared__ volatile int abort_flag;
     uint8_t* smem = smem_raw + ((1024u - (smem_u32(smem_raw) & 1023u)) & 1023u);      // swizzled tiles: 1024-byte aligned
     const uint32_t kv_base = smem_u32(smem);            // [RING][K tile, V tile], then the Q tile [16][HD]
-    const uint32_t q_tile = kv_base + 2 * RING * TILE;
+    const uint32_t q_tile = kv_base + RING * STAGE;
 
     const int b = blockIdx.x, kvh = blockIdx.y, split = blockIdx.z;
     const int n_rep = n_heads / n_kv_heads;
@@ -543,9 +545,9 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
     const int pg_begin = pg_lo + split * per, pg_end = min(pg_hi, pg_begin + per);
 
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
-    float o[HD / 8][4];
+    float o[VD / 8][4];
 #pragma unroll
-    for (int t = 0; t < HD / 8; ++t) o[t][0] = o[t][1] = o[t][2] = o[t][3] = 0.f;
+    for (int t = 0; t < VD / 8; ++t) o[t][0] = o[t][1] = o[t][2] = o[t][3] = 0.f;
 
     if (warp == 4) {
         // ---------------- producer ----------------
@@ -565,11 +567,11 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
                 }
                 const int row = (page_now * n_kv_heads + kvh) * PAGE;
                 const uint32_t bar = smem_u32(&full_bar[s]);
-                tc::mbar_expect_tx(bar, 2 * TILE);
+                tc::mbar_expect_tx(bar, STAGE);
 #pragma unroll
-                for (int a = 0; a < ATOMS; ++a) {
-                    tc::tma_load_2d(kv_base + (2 * s) * TILE + a * PAGE * 128, &map_k, bar, a * 64, row);
-                    tc::tma_load_2d(kv_base + (2 * s + 1) * TILE + a * PAGE * 128, &map_v, bar, a * 64, row);
+                for (int a = 0; a < (ATOMS > V_ATOMS ? ATOMS : V_ATOMS); ++a) {
+                    if (a < ATOMS) tc::tma_load_2d(kv_base + s * STAGE + a * PAGE * 128, &map_k, bar, a * 64, row);
+                    if (a < V_ATOMS) tc::tma_load_2d(kv_base + s * STAGE + K_TILE + a * PAGE * 128, &map_v, bar, a * 64, row);
                 }
                 issued = j + 1;
             }
@@ -584,7 +586,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
             const int r = idx / (HD / 8), c = idx % (HD / 8);
             uint4 v = make_uint4(0, 0, 0, 0);
             if (r < n_rep) v = *reinterpret_cast<const uint4*>(q + (size_t)token * q_ld + (size_t)(kvh * n_rep + r) * HD + c * 8);
-            *reinterpret_cast<uint4*>(smem + 2 * RING * TILE + tile_off<HD>(r, c)) = v;
+            *reinterpret_cast<uint4*>(smem + RING * STAGE + tile_off<HD>(r, c)) = v;
         }
         asm volatile("bar.sync 1, 128;" ::: "memory");          // the four compute warps: Q tile written
         RI_PHASE(0);
@@ -601,7 +603,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
                 if (lane == 0) { tc::report(status, 22); abort_flag = 1; }
                 break;
             }
-            const uint32_t ktile = kv_base + (2 * s) * TILE, vtile = ktile + TILE;
+            const uint32_t ktile = kv_base + s * STAGE, vtile = ktile + K_TILE;
             const int kbase = warp * 16;
             const int key0 = pg * PAGE + kbase;
             if (key0 < n_keys && key0 + 16 > first_key) {
@@ -614,10 +616,10 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
                         const int key = key0 + t * 8 + 2 * tq + (e & 1);
                         sc[t][e] = (key < n_keys && key >= first_key) ? sc[t][e] * scale : -INFINITY;
                     }
-                softmax_update<2, HD / 8>(sc, m, l, o);
+                softmax_update<2, VD / 8>(sc, m, l, o);
                 uint32_t pf[4] = {pack_bf16(sc[0][0], sc[0][1]), pack_bf16(sc[0][2], sc[0][3]),
                                   pack_bf16(sc[1][0], sc[1][1]), pack_bf16(sc[1][2], sc[1][3])};
-                pv_16keys_atoms<HD>(pf, vtile, kbase, o);
+                pv_16keys_atoms<VD>(pf, vtile, kbase, o);
             }
             __syncwarp();
             if (lane == 0) tc::mbar_arrive(smem_u32(&empty_bar[s]));       // this warp is done with the stage
@@ -628,12 +630,12 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
     RI_PHASE_LATEST(2);
 
     // ---- merge the 4 compute warps (each saw a quarter of the keys) through shared memory ----
-    constexpr int SO_LD = HD + 4;                         // padded rows: the 8 rows a warp stores at once hit 8 bank groups
+    constexpr int SO_LD = VD + 4;                         // padded rows: the 8 rows a warp stores at once hit 8 bank groups
     float* so = reinterpret_cast<float*>(smem);           // [4][16][SO_LD]
     float* sml = so + 4 * 16 * SO_LD;                     // [4][16][2]
     if (warp < 4) {
 #pragma unroll
-        for (int t = 0; t < HD / 8; ++t) {
+        for (int t = 0; t < VD / 8; ++t) {
             const int d = t * 8 + 2 * tq;
             *reinterpret_cast<float2*>(so + (warp * 16 + g) * SO_LD + d) = make_float2(o[t][0], o[t][1]);
             *reinterpret_cast<float2*>(so + (warp * 16 + g + 8) * SO_LD + d) = make_float2(o[t][2], o[t][3]);
@@ -648,14 +650,14 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
     __syncthreads();
     if constexpr (CLUSTER) {
         // the splits of this (sequence, kv head) are the CTAs of one cluster: merged here, no scratch, no second kernel
-        float* recv = reinterpret_cast<float*>(smem + 2 * RING * TILE + 16 * HD * 2);
-        cluster_merge<HD, DECODE_TMA_THREADS>(so, sml, recv, n_rep, n_splits, split, token, kvh, out, out_ld, !abort_flag);
+        float* recv = reinterpret_cast<float*>(smem + RING * STAGE + 16 * HD * 2);
+        cluster_merge<VD, DECODE_TMA_THREADS>(so, sml, recv, n_rep, n_splits, split, token, kvh, out, out_ld, !abort_flag);
         return;
     }
     if (abort_flag) return;
-    for (int it = threadIdx.x; it < n_rep * (HD / 4); it += DECODE_TMA_THREADS) {
-        const int r = it / (HD / 4), d = (it % (HD / 4)) * 4;
-        write_merged<HD>(so, sml, r, d, b, kvh * n_rep + r, token, n_heads, n_splits, split, part_o, part_ml, out, out_ld);
+    for (int it = threadIdx.x; it < n_rep * (VD / 4); it += DECODE_TMA_THREADS) {
+        const int r = it / (VD / 4), d = (it % (VD / 4)) * 4;
+        write_merged<VD>(so, sml, r, d, b, kvh * n_rep + r, token, n_heads, n_splits, split, part_o, part_ml, out, out_ld);
     }
 }
 
@@ -1196,24 +1198,28 @@ int launch_decode(const void* q, int q_ld, const void* kc, const void* vc, const
     return 0;
 }
 
-template <int HD>
+// bytes of the ring of K and V page tiles
+template <int HD, int VD>
+constexpr int decode_ring_bytes() { return RING * (PAGE * HD * 2 + (VD + 63) / 64 * PAGE * 128); }
+
+template <int HD, int VD>
 int launch_decode_tma(const CUtensorMap& mk, const CUtensorMap& mv, const void* q, int q_ld, const int* page_table,
                       int max_pages, const int* seq_slot, const int* seq_len, const int* cu_seqlens, int n_seqs,
                       int n_heads, int n_kv_heads, float scale, int window, int n_splits, float* part_o,
                       float* part_ml, void* out, int out_ld, int* status, cudaStream_t stream) {
-    constexpr int SMEM = 2 * RING * PAGE * HD * 2 + 16 * HD * 2 + 1024;
-    static_assert((4 * 16 * (HD + 4) + 4 * 16 * 2 + 4 * 16 + 16 * 2) * 4 <= 2 * RING * PAGE * HD * 2, "merge area must fit the ring");
+    constexpr int SMEM = decode_ring_bytes<HD, VD>() + 16 * HD * 2 + 1024;
+    static_assert((4 * 16 * (VD + 4) + 4 * 16 * 2 + 4 * 16 + 16 * 2) * 4 <= decode_ring_bytes<HD, VD>(), "merge area must fit the ring");
     static PerDeviceOnce configured;       // per device: the attribute belongs to a device's copy of the kernel
-    if (int rc = raise_dynamic_smem(attn_decode_tma_kernel<HD, false>, SMEM, configured, "attention")) return rc;
+    if (int rc = raise_dynamic_smem(attn_decode_tma_kernel<HD, VD, false>, SMEM, configured, "attention")) return rc;
     dim3 grid(n_seqs, n_kv_heads, n_splits);
     cudaError_t e = launch_dependent(
-        attn_decode_tma_kernel<HD, false>, grid, dim3(DECODE_TMA_THREADS), (size_t)SMEM, stream, mk, mv, (const __nv_bfloat16*)q,
+        attn_decode_tma_kernel<HD, VD, false>, grid, dim3(DECODE_TMA_THREADS), (size_t)SMEM, stream, mk, mv, (const __nv_bfloat16*)q,
         q_ld, page_table, max_pages, seq_slot, seq_len, cu_seqlens, n_heads, n_kv_heads, scale, window, n_splits, part_o,
         part_ml, (__nv_bfloat16*)out, out_ld, status);
     if (int rc = check_launch(e, "attn_decode_tma")) return rc;
     if (n_splits > 1) {
-        e = launch_dependent(attn_combine_kernel, dim3(n_seqs, n_heads), dim3(HD >= 128 ? 128 : 64), (size_t)0, stream,
-                             (const float*)part_o, (const float*)part_ml, cu_seqlens, n_heads, (int)HD, n_splits,
+        e = launch_dependent(attn_combine_kernel, dim3(n_seqs, n_heads), dim3(VD >= 128 ? 128 : 64), (size_t)0, stream,
+                             (const float*)part_o, (const float*)part_ml, cu_seqlens, n_heads, (int)VD, n_splits,
                              (__nv_bfloat16*)out, out_ld);
         return check_launch(e, "attn_combine");
     }
@@ -1221,24 +1227,24 @@ int launch_decode_tma(const CUtensorMap& mk, const CUtensorMap& mv, const void* 
 }
 
 // The TMA-fed kernel with the splits of a (sequence, kv head) as one cluster.
-template <int HD>
+template <int HD, int VD>
 constexpr int tma_cluster_smem_bytes() {
-    return 2 * RING * PAGE * HD * 2 + 16 * HD * 2 + CLUSTER_RECV_FLOATS<HD> * 4 + 1024;
+    return decode_ring_bytes<HD, VD>() + 16 * HD * 2 + CLUSTER_RECV_FLOATS<VD> * 4 + 1024;
 }
 
-template <int HD>
+template <int HD, int VD>
 PerDeviceOnce& tma_cluster_configured() {
     static PerDeviceOnce once;
     return once;
 }
 
-template <int HD>
+template <int HD, int VD>
 void tma_cluster_config(cudaLaunchConfig_t& cfg, cudaLaunchAttribute* attr, int n_seqs, int n_kv_heads, int n_splits,
                         cudaStream_t stream) {
     cfg = {};
     cfg.gridDim = dim3(n_seqs, n_kv_heads, n_splits);
     cfg.blockDim = dim3(DECODE_TMA_THREADS);
-    cfg.dynamicSmemBytes = tma_cluster_smem_bytes<HD>();
+    cfg.dynamicSmemBytes = tma_cluster_smem_bytes<HD, VD>();
     cfg.stream = stream;
     attr[0].id = cudaLaunchAttributeClusterDimension;
     attr[0].val.clusterDim.x = 1;
@@ -1250,16 +1256,16 @@ void tma_cluster_config(cudaLaunchConfig_t& cfg, cudaLaunchAttribute* attr, int 
     cfg.numAttrs = pdl_enabled() ? 2 : 1;
 }
 
-template <int HD>
+template <int HD, int VD>
 int launch_decode_tma_cluster(const CUtensorMap& mk, const CUtensorMap& mv, const void* q, int q_ld, const int* page_table,
                               int max_pages, const int* seq_slot, const int* seq_len, const int* cu_seqlens, int n_seqs,
                               int n_heads, int n_kv_heads, float scale, int window, int n_splits, void* out, int out_ld,
                               int* status, cudaStream_t stream) {
-    auto kernel = attn_decode_tma_kernel<HD, true>;
-    if (int rc = raise_dynamic_smem(kernel, tma_cluster_smem_bytes<HD>(), tma_cluster_configured<HD>(), "attention")) return rc;
+    auto kernel = attn_decode_tma_kernel<HD, VD, true>;
+    if (int rc = raise_dynamic_smem(kernel, tma_cluster_smem_bytes<HD, VD>(), tma_cluster_configured<HD, VD>(), "attention")) return rc;
     cudaLaunchConfig_t cfg;
     cudaLaunchAttribute attr[2];
-    tma_cluster_config<HD>(cfg, attr, n_seqs, n_kv_heads, n_splits, stream);
+    tma_cluster_config<HD, VD>(cfg, attr, n_seqs, n_kv_heads, n_splits, stream);
     cudaError_t e = cudaLaunchKernelEx(&cfg, kernel, mk, mv, (const __nv_bfloat16*)q, q_ld, page_table, max_pages, seq_slot,
                                        seq_len, cu_seqlens, n_heads, n_kv_heads, scale, window, n_splits, (float*)nullptr,
                                        (float*)nullptr, (__nv_bfloat16*)out, out_ld, status);
@@ -1267,13 +1273,13 @@ int launch_decode_tma_cluster(const CUtensorMap& mk, const CUtensorMap& mv, cons
 }
 
 // How many clusters of n_splits CTAs of that kernel the device holds at once.
-template <int HD>
+template <int HD, int VD>
 int decode_tma_cluster_capacity(int n_splits, int* clusters) {
-    auto kernel = attn_decode_tma_kernel<HD, true>;
-    if (int rc = raise_dynamic_smem(kernel, tma_cluster_smem_bytes<HD>(), tma_cluster_configured<HD>(), "attention")) return rc;
+    auto kernel = attn_decode_tma_kernel<HD, VD, true>;
+    if (int rc = raise_dynamic_smem(kernel, tma_cluster_smem_bytes<HD, VD>(), tma_cluster_configured<HD, VD>(), "attention")) return rc;
     cudaLaunchConfig_t cfg;
     cudaLaunchAttribute attr[2];
-    tma_cluster_config<HD>(cfg, attr, 1, 1, n_splits, nullptr);
+    tma_cluster_config<HD, VD>(cfg, attr, 1, 1, n_splits, nullptr);
     cfg.numAttrs = 1;
     cudaError_t e = cudaOccupancyMaxActiveClusters(clusters, kernel, &cfg);
     if (e != cudaSuccess) return fail("attention_decode: cannot ask how many clusters fit: %s", cudaGetErrorString(e));
@@ -1323,6 +1329,20 @@ int check_common(int hd, int page_size, int n_heads, int n_kv_heads, int q_ld, i
 
 }  // namespace
 
+// 1 if the TMA-fed decode kernels take heads of these sizes (keys hd, values v_hd)
+RI_API int ri_attention_decode_tma_supports(int hd, int v_hd) {
+    return (hd == 64 || hd == 128) && (v_hd == 32 || v_hd == 64 || v_hd == 128);
+}
+#define RI_VALUE_SIZES(H, CALL) \
+    if (v_hd == 32) return CALL<H, 32> ARGS; \
+    if (v_hd == 64) return CALL<H, 64> ARGS; \
+    return CALL<H, 128> ARGS
+#define RI_HEAD_SIZES(CALL) \
+    if (hd == 64) { RI_VALUE_SIZES(64, CALL); } \
+    RI_VALUE_SIZES(128, CALL)
+#define RI_CHECK_VALUES() \
+    if (!ri_attention_decode_tma_supports(hd, v_hd)) return fail("attention_decode: heads of %d with values of %d", hd, v_hd)
+
 // 1 if the tensor-core kernels take this shape (the caller falls back to the generic kernel otherwise)
 RI_API int ri_attention_mma_supports(int hd, int page_size, int n_heads, int n_kv_heads, int decode) {
     if (hd != 64 && hd != 128) return 0;
@@ -1353,12 +1373,13 @@ RI_API int ri_attention_decode(const void* q, int q_ld, const void* kcache, cons
 }
 
 // The same with the cache pages brought in by TMA.  map_k / map_v: tensor maps (128 bytes each) of the
-// layer's K and V viewed as [pages * kv heads * 64, head_dim] with a {64, 64} box and 128-byte swizzle.
+// layer's K and V viewed as [pages * kv heads * 64, head size] with a {64, 64} box and 128-byte swizzle (v_hd: the
+// values' head size; out and the scratch then have heads of that size).
 // `status` (may be null) is a host-visible int that receives a code if a bounded wait ran out.
 RI_API int ri_attention_decode_tma(const void* map_k, const void* map_v, const void* q, int q_ld,
                                    const int* page_table, int max_pages, const int* seq_slot, const int* seq_len,
                                    const int* cu_seqlens, void* out, int out_ld, int n_seqs, int n_heads,
-                                   int n_kv_heads, int hd, int page_size, float scale, int window, int n_splits,
+                                   int n_kv_heads, int hd, int v_hd, int page_size, float scale, int window, int n_splits,
                                    float* part_o, float* part_ml, int* status, cudaStream_t stream) {
     if (n_seqs <= 0) return 0;
     if (int rc = check_common(hd, page_size, n_heads, n_kv_heads, q_ld, out_ld, q, out)) return rc;
@@ -1366,13 +1387,13 @@ RI_API int ri_attention_decode_tma(const void* map_k, const void* map_v, const v
     if (n_splits < 1 || n_splits > 65535) return fail("attention_decode: %d splits", n_splits);
     if (n_splits > 1 && (part_o == nullptr || part_ml == nullptr)) return fail("attention_decode: splits need scratch");
     if (n_kv_heads > 65535) return fail("attention_decode: %d kv heads exceed the grid limit", n_kv_heads);
+    RI_CHECK_VALUES();
     const CUtensorMap& mk = *reinterpret_cast<const CUtensorMap*>(map_k);
     const CUtensorMap& mv = *reinterpret_cast<const CUtensorMap*>(map_v);
-    if (hd == 64)
-        return launch_decode_tma<64>(mk, mv, q, q_ld, page_table, max_pages, seq_slot, seq_len, cu_seqlens, n_seqs, n_heads,
-                                     n_kv_heads, scale, window, n_splits, part_o, part_ml, out, out_ld, status, stream);
-    return launch_decode_tma<128>(mk, mv, q, q_ld, page_table, max_pages, seq_slot, seq_len, cu_seqlens, n_seqs, n_heads,
-                                  n_kv_heads, scale, window, n_splits, part_o, part_ml, out, out_ld, status, stream);
+#define ARGS (mk, mv, q, q_ld, page_table, max_pages, seq_slot, seq_len, cu_seqlens, n_seqs, n_heads, n_kv_heads, \
+              scale, window, n_splits, part_o, part_ml, out, out_ld, status, stream)
+    RI_HEAD_SIZES(launch_decode_tma);
+#undef ARGS
 }
 
 // The same with the 2..8 splits of a (sequence, kv head) as one thread-block cluster that merges its own partial
@@ -1380,7 +1401,7 @@ RI_API int ri_attention_decode_tma(const void* map_k, const void* map_v, const v
 RI_API int ri_attention_decode_tma_cluster(const void* map_k, const void* map_v, const void* q, int q_ld,
                                            const int* page_table, int max_pages, const int* seq_slot,
                                            const int* seq_len, const int* cu_seqlens, void* out, int out_ld, int n_seqs,
-                                           int n_heads, int n_kv_heads, int hd, int page_size, float scale, int window,
+                                           int n_heads, int n_kv_heads, int hd, int v_hd, int page_size, float scale, int window,
                                            int n_splits, int* status, cudaStream_t stream) {
     if (n_seqs <= 0) return 0;
     if (int rc = check_common(hd, page_size, n_heads, n_kv_heads, q_ld, out_ld, q, out)) return rc;
@@ -1388,21 +1409,23 @@ RI_API int ri_attention_decode_tma_cluster(const void* map_k, const void* map_v,
     if (n_splits < 2 || n_splits > MAX_CLUSTER_SPLITS)
         return fail("attention_decode: a cluster takes 2 to %d splits, not %d", MAX_CLUSTER_SPLITS, n_splits);
     if (n_kv_heads > 65535) return fail("attention_decode: %d kv heads exceed the grid limit", n_kv_heads);
+    RI_CHECK_VALUES();
     const CUtensorMap& mk = *reinterpret_cast<const CUtensorMap*>(map_k);
     const CUtensorMap& mv = *reinterpret_cast<const CUtensorMap*>(map_v);
-    if (hd == 64)
-        return launch_decode_tma_cluster<64>(mk, mv, q, q_ld, page_table, max_pages, seq_slot, seq_len, cu_seqlens, n_seqs,
-                                             n_heads, n_kv_heads, scale, window, n_splits, out, out_ld, status, stream);
-    return launch_decode_tma_cluster<128>(mk, mv, q, q_ld, page_table, max_pages, seq_slot, seq_len, cu_seqlens, n_seqs,
-                                          n_heads, n_kv_heads, scale, window, n_splits, out, out_ld, status, stream);
+#define ARGS (mk, mv, q, q_ld, page_table, max_pages, seq_slot, seq_len, cu_seqlens, n_seqs, n_heads, n_kv_heads, \
+              scale, window, n_splits, out, out_ld, status, stream)
+    RI_HEAD_SIZES(launch_decode_tma_cluster);
+#undef ARGS
 }
 
 // clusters[0] = how many clusters of n_splits CTAs of that kernel the current device holds at the same time
-RI_API int ri_attention_decode_tma_cluster_capacity(int hd, int n_splits, int* clusters) {
-    if (hd != 64 && hd != 128) return fail("attention_mma: head_dim %d is not 64 or 128", hd);
+RI_API int ri_attention_decode_tma_cluster_capacity(int hd, int v_hd, int n_splits, int* clusters) {
+    RI_CHECK_VALUES();
     if (n_splits < 2 || n_splits > MAX_CLUSTER_SPLITS)
         return fail("attention_decode: a cluster takes 2 to %d splits, not %d", MAX_CLUSTER_SPLITS, n_splits);
-    return hd == 64 ? decode_tma_cluster_capacity<64>(n_splits, clusters) : decode_tma_cluster_capacity<128>(n_splits, clusters);
+#define ARGS (n_splits, clusters)
+    RI_HEAD_SIZES(decode_tma_cluster_capacity);
+#undef ARGS
 }
 
 RI_API int ri_attention_prefill(const void* q, int q_ld, const void* kcache, const void* vcache, const int* page_table,

@@ -16,7 +16,7 @@
 //                 accumulator is rescaled rarely (exactness is kept: the final division by the
 //                 row sum uses the same scaling).
 //   O += P V      P goes back to tensor memory as bf16, over the scores it was made from, and is the
-//                 A operand; the V page, [keys][head_dim] as the cache holds it, is the B operand
+//                 A operand; the V page, [keys][value head size] as the cache holds it, is the B operand
 //                 in MN-major form; O accumulates in tensor memory in float32.
 // Warp 0 issues the TMA loads, warp 1 the MMAs, warps 2-5 are the softmax rows.  There are two score
 // buffers in tensor memory: S of page j+1 is computed while the softmax of page j runs, and the
@@ -90,7 +90,8 @@ __device__ __forceinline__ uint32_t pack2(float lo, float hi) {
     return *reinterpret_cast<uint32_t*>(&v);
 }
 
-template <int HD, bool FORMS>
+// VD: the size of a value head; one below 64 takes a tile of 64 columns that the copy fills up with zeros, and so does the product
+template <int HD, int VD, bool FORMS>
 __global__ void __launch_bounds__(THREADS, 2)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                        const __grid_constant__ CUtensorMap map_v, const int* __restrict__ page_table, int max_pages,
@@ -101,11 +102,12 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
     constexpr int ATOMS = HD / 64;                       // 64-wide (128-byte) column tiles per row of head_dim
     constexpr int Q_BYTES = ATOMS * BM * 128;            // [atom][128 queries][64]
     constexpr int K_BYTES = ATOMS * BN * 128;            // one buffer: [atom][64 keys][64]
-    constexpr int V_BYTES = ATOMS * BN * 128;
+    constexpr int V_ATOMS = (VD + 63) / 64;
+    constexpr int V_BYTES = V_ATOMS * BN * 128;
     constexpr int S_COL = 0, O_COL = 2 * BN;             // two score buffers, then the output accumulator
     constexpr int TMEM_COLS = 256;
     constexpr uint32_t IDESC_S = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(BN >> 3) << 17) | ((uint32_t)(BM >> 4) << 24);
-    constexpr uint32_t IDESC_PV = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | ((uint32_t)(HD >> 3) << 17) |
+    constexpr uint32_t IDESC_PV = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | ((uint32_t)(V_ATOMS * 64 >> 3) << 17) |
                                   ((uint32_t)(BM >> 4) << 24);
 
     // Everything lives in dynamic shared memory: the tiles (1024-byte aligned for the 128-byte swizzle) and,
@@ -199,7 +201,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
                     report(status, ST_ATTN_PRODUCER); abort_flag = 1; break;
                 }
                 mbar_expect_tx(smem_u32(&v_full[kb]), V_BYTES);
-                for (int a = 0; a < ATOMS; ++a)
+                for (int a = 0; a < V_ATOMS; ++a)
                     tma_load_2d(v_smem + kb * V_BYTES + a * BN * 128, &map_v, smem_u32(&v_full[kb]), a * 64, row);
                 v_issued = j + 1;
             }
@@ -337,7 +339,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
                 tc_fence_after();
                 if (__any_sync(0xffffffffu, move)) {            // rescale the accumulator (uniform over the warp)
 #pragma unroll 1
-                    for (int c = 0; c < HD; c += 16) {
+                    for (int c = 0; c < VD; c += 16) {
                         uint32_t o[16];
                         tmem_ld16(trow + O_COL + c, o);
                         tmem_wait_ld();
@@ -371,9 +373,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
             // FORMS: a sink joins the row's sum as one more term exp(sink_h) without a value (2^x may overflow to infinity when
             // the sink outweighs every score: the result is then 0, as it should be)
             const float inv = out_scale / ((FORMS && sink != nullptr) ? l + fast_exp2(fmaf(sink[h], 1.4426950408889634f, -m_used)) : l);
-            __nv_bfloat16* dst = out + (size_t)(tok0 + q0 + r) * out_ld + (size_t)h * HD;
+            __nv_bfloat16* dst = out + (size_t)(tok0 + q0 + r) * out_ld + (size_t)h * VD;
 #pragma unroll 1
-            for (int c = 0; c < HD; c += 16) {
+            for (int c = 0; c < VD; c += 16) {
                 uint32_t o[16];
                 tmem_ld16(trow + O_COL + c, o);
                 tmem_wait_ld();
@@ -402,7 +404,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
     }
 }
 
-template <int HD, bool FORMS>
+template <int HD, int VD, bool FORMS>
 int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const int* page_table, int max_pages,
            const int* seq_slot, const int* seq_start, const int* cu_seqlens, int n_seqs, int max_new, int n_heads,
            int n_kv_heads, float scale, int window, float out_scale, void* out, int out_ld, int* status, cudaStream_t stream,
@@ -410,9 +412,9 @@ int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, 
     constexpr int ATOMS = HD / 64;
     // Q, two K and two V pages, P, the barriers; with head_dim 128 no room for alignment padding is left if
     // two CTAs are to share an SM (the kernel refuses, with a status code, a shared window that needs any)
-    constexpr int TILES = ATOMS * BM * 128 + 4 * ATOMS * BN * 128;
-    constexpr int SMEM = TILES + (HD >= 128 ? 256 : 1024 + 256);
-    auto kernel = attn_prefill_tc_kernel<HD, FORMS>;
+    constexpr int TILES = ATOMS * BM * 128 + 2 * (ATOMS + (VD + 63) / 64) * BN * 128;
+    constexpr int SMEM = TILES + (HD >= 128 && VD >= 128 ? 256 : 1024 + 256);
+    auto kernel = attn_prefill_tc_kernel<HD, VD, FORMS>;
     static PerDeviceOnce configured;       // per device: the attribute belongs to a device's copy of the kernel
     if (int rc = raise_dynamic_smem(kernel, SMEM, configured, "attention_tcgen05")) return rc;
     // blocks are handed out x fastest: every head and sequence of the longest query tiles first, the short
@@ -428,8 +430,8 @@ int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, 
 
 }  // namespace
 
-RI_API int ri_attention_tcgen05_supports(int hd, int page_size, int n_heads, int n_kv_heads, int q_ld, int out_ld) {
-    if (hd != 64 && hd != 128) return 0;
+RI_API int ri_attention_tcgen05_supports(int hd, int v_hd, int page_size, int n_heads, int n_kv_heads, int q_ld, int out_ld) {
+    if ((hd != 64 && hd != 128) || (v_hd != 32 && v_hd != 64 && v_hd != 128)) return 0;
     if (page_size != BN) return 0;
     if (n_kv_heads <= 0 || n_heads % n_kv_heads) return 0;
     if (q_ld % 8 || out_ld % 8) return 0;
@@ -438,7 +440,7 @@ RI_API int ri_attention_tcgen05_supports(int hd, int page_size, int n_heads, int
 
 // Tensor maps (128 bytes each, 64-byte aligned storage):
 //   which 0: the query rows, a matrix [rows, cols] with row stride ld (the packed q/k/v buffer); box of 128 rows
-//   which 1: one cache layer viewed as [pages * kv heads * 64, head_dim]; box of 64 rows (keys or values)
+//   which 1: one cache layer viewed as [pages * kv heads * 64, head size]; box of 64 rows (keys or values)
 RI_API int ri_attention_tcgen05_encode(void* map_out, int which, const void* ptr, long long rows, long long cols,
                                        long long ld) {
     if ((uintptr_t)map_out % 64) return fail("attention_tcgen05: tensor map storage must be 64-byte aligned");
@@ -449,10 +451,10 @@ RI_API int ri_attention_tcgen05_encode(void* map_out, int which, const void* ptr
 RI_API int ri_attention_tcgen05_prefill(const void* map_q, const void* map_k, const void* map_v, const int* page_table,
                                         int max_pages, const int* seq_slot, const int* seq_start,
                                         const int* cu_seqlens, void* out, int out_ld, int n_seqs, int max_new,
-                                        int n_heads, int n_kv_heads, int hd, int page_size, float scale, int window,
+                                        int n_heads, int n_kv_heads, int hd, int v_hd, int page_size, float scale, int window,
                                         float out_scale, int* status, cudaStream_t stream) {
     if (n_seqs <= 0 || max_new <= 0) return 0;
-    if (!ri_attention_tcgen05_supports(hd, page_size, n_heads, n_kv_heads, 8, out_ld))
+    if (!ri_attention_tcgen05_supports(hd, v_hd, page_size, n_heads, n_kv_heads, 8, out_ld))
         return fail("attention_tcgen05: head_dim %d, pages of %d, %d heads over %d kv heads, out rows of %d are not supported",
                     hd, page_size, n_heads, n_kv_heads, out_ld);
     if ((uintptr_t)out % 16) return fail("attention_tcgen05: out is not 16-byte aligned");
@@ -460,11 +462,11 @@ RI_API int ri_attention_tcgen05_prefill(const void* map_q, const void* map_k, co
     const CUtensorMap& mq = *reinterpret_cast<const CUtensorMap*>(map_q);
     const CUtensorMap& mk = *reinterpret_cast<const CUtensorMap*>(map_k);
     const CUtensorMap& mv = *reinterpret_cast<const CUtensorMap*>(map_v);
-    if (hd == 64)
-        return launch<64, false>(mq, mk, mv, page_table, max_pages, seq_slot, seq_start, cu_seqlens, n_seqs, max_new, n_heads,
-                                 n_kv_heads, scale, window, out_scale, out, out_ld, status, stream);
-    return launch<128, false>(mq, mk, mv, page_table, max_pages, seq_slot, seq_start, cu_seqlens, n_seqs, max_new, n_heads,
-                              n_kv_heads, scale, window, out_scale, out, out_ld, status, stream);
+#define RI_LAUNCH(H, V) if (hd == H && v_hd == V) return launch<H, V, false>(mq, mk, mv, page_table, max_pages, seq_slot, seq_start, cu_seqlens, n_seqs, max_new, \
+        n_heads, n_kv_heads, scale, window, out_scale, out, out_ld, status, stream)
+    RI_LAUNCH(64, 32); RI_LAUNCH(64, 64); RI_LAUNCH(64, 128); RI_LAUNCH(128, 32); RI_LAUNCH(128, 64); RI_LAUNCH(128, 128);
+#undef RI_LAUNCH
+    return fail("attention_tcgen05: no kernel for heads of %d with values of %d", hd, v_hd);
 }
 
 // The same with capped scores (softcap > 0: s <- softcap tanh(s scale / softcap)) and, with a window (> 0 only: the last
@@ -473,11 +475,11 @@ RI_API int ri_attention_tcgen05_prefill(const void* map_q, const void* map_k, co
 RI_API int ri_attention_tcgen05_prefill_forms(const void* map_q, const void* map_k, const void* map_v, const int* page_table,
                                               int max_pages, const int* seq_slot, const int* seq_start,
                                               const int* cu_seqlens, void* out, int out_ld, int n_seqs, int max_new,
-                                              int n_heads, int n_kv_heads, int hd, int page_size, float scale, int window,
+                                              int n_heads, int n_kv_heads, int hd, int v_hd, int page_size, float scale, int window,
                                               float out_scale, float softcap, int keep_first, const float* sink, int* status,
                                               cudaStream_t stream) {
     if (n_seqs <= 0 || max_new <= 0) return 0;
-    if (!ri_attention_tcgen05_supports(hd, page_size, n_heads, n_kv_heads, 8, out_ld))
+    if (!ri_attention_tcgen05_supports(hd, v_hd, page_size, n_heads, n_kv_heads, 8, out_ld))
         return fail("attention_tcgen05: head_dim %d, pages of %d, %d heads over %d kv heads, out rows of %d are not supported",
                     hd, page_size, n_heads, n_kv_heads, out_ld);
     if (softcap < 0.f || keep_first < 0 || window < 0 || (keep_first > 0 && window == 0))
@@ -487,11 +489,11 @@ RI_API int ri_attention_tcgen05_prefill_forms(const void* map_q, const void* map
     const CUtensorMap& mq = *reinterpret_cast<const CUtensorMap*>(map_q);
     const CUtensorMap& mk = *reinterpret_cast<const CUtensorMap*>(map_k);
     const CUtensorMap& mv = *reinterpret_cast<const CUtensorMap*>(map_v);
-    if (hd == 64)
-        return launch<64, true>(mq, mk, mv, page_table, max_pages, seq_slot, seq_start, cu_seqlens, n_seqs, max_new, n_heads,
-                                n_kv_heads, scale, window, out_scale, out, out_ld, status, stream, softcap, keep_first, sink);
-    return launch<128, true>(mq, mk, mv, page_table, max_pages, seq_slot, seq_start, cu_seqlens, n_seqs, max_new, n_heads,
-                             n_kv_heads, scale, window, out_scale, out, out_ld, status, stream, softcap, keep_first, sink);
+#define RI_LAUNCH(H, V) if (hd == H && v_hd == V) return launch<H, V, true>(mq, mk, mv, page_table, max_pages, seq_slot, seq_start, cu_seqlens, n_seqs, max_new, \
+        n_heads, n_kv_heads, scale, window, out_scale, out, out_ld, status, stream, softcap, keep_first, sink)
+    RI_LAUNCH(64, 32); RI_LAUNCH(64, 64); RI_LAUNCH(64, 128); RI_LAUNCH(128, 32); RI_LAUNCH(128, 64); RI_LAUNCH(128, 128);
+#undef RI_LAUNCH
+    return fail("attention_tcgen05: no kernel for heads of %d with values of %d", hd, v_hd);
 }
 
 RI_DEFINE_LAST_ERROR()

@@ -7,13 +7,14 @@
   further forms of the score     gate per head: single tokens and prompts on mma.sync kernels with those forms
                                  (`attention_decode_forms`, `attention_prefill_forms`); prompts without a bias and
                                  a gate on the tcgen05 kernel
+  bfloat16, head_dim 64 or 128,  values of 32, 64 or 128: the TMA-fed decode kernel and the tcgen05 prefill kernel, in their
+  values of another size         instances for both sizes
   anything else                  the generic kernel (`attention_generic`): any head size, any
                                  dtype, float32 arithmetic
 
 Besides causality a mixer may limit a query's keys to the last `window` keys or to the query's own
 chunk of positions.  The tensor-core kernels take either as one signed span (`csrc/common.cuh:
-first_visible_key`); both at once, or values of another head size than the keys', go to the
-generic kernel.
+first_visible_key`); both at once go to the generic kernel.
 """
 from __future__ import annotations
 
@@ -52,7 +53,8 @@ def decode_splits(n_seqs: int, n_kv_heads: int, max_seq_len: int, page_size: int
     return max(1, min(want, limit, -(-max_seq_len // page_size)))
 
 
-def decode_plan(n_seqs: int, n_kv_heads: int, max_seq_len: int, page_size: int, head_dim: int | None = None):
+def decode_plan(n_seqs: int, n_kv_heads: int, max_seq_len: int, page_size: int, head_dim: int | None = None,
+                v_head_dim: int | None = None):
     """Which decode kernel a step of n_seqs sequences takes, and into how many runs of pages it
     cuts a sequence: ("cluster" | "tma" | "cp_async", splits).  Left to itself it answers "cluster"
     (the TMA-fed kernel with the 2..8 runs of a sequence as one thread-block cluster) while a step's
@@ -69,7 +71,8 @@ def decode_plan(n_seqs: int, n_kv_heads: int, max_seq_len: int, page_size: int, 
         splits = decode_splits(n_seqs, n_kv_heads, max_seq_len, page_size, CLUSTER_SPLITS)
         if head_dim is not None:
             from . import attention_tc
-            while splits >= 2 and attention_tc.decode_cluster_capacity(head_dim, splits) < n_seqs * n_kv_heads:
+            sizes = {} if v_head_dim is None else {"v_head_dim": v_head_dim}
+            while splits >= 2 and attention_tc.decode_cluster_capacity(head_dim, splits, **sizes) < n_seqs * n_kv_heads:
                 splits -= 1
         if splits >= 2:
             return "cluster", splits
@@ -95,16 +98,21 @@ def attention(qkv, cache_layer, out, ctx, *, n_heads, n_kv_heads, head_dim, scal
     leading n_heads*head_dim columns of `qkv`, already rotated.  `window`: only the last so many
     keys; `chunk`: only the keys of the query's own block of that many positions (counted from the
     start of the sequence); `v_head_dim`: values of another head size than keys; `out_scale`: a
-    factor on the result.  The tensor-core kernels take a window or a chunk (as one signed span) and
-    equal head sizes; values of their own size, or both limits at once, are the generic kernel's.
+    factor on the result.  The tensor-core kernels take a window or a chunk (as one signed span);
+    both limits at once are the generic kernel's.
     `softcap`, `keep_first`, `sink`, `dist`, `gate`: a cap on the scores, first positions that stay visible beyond
     the window, a term without key in the softmax's denominator, a bias by distance and a gate per head on the
     result (see `ops.attention_generic`)."""
     q_ld = qkv.shape[1]
     same_sizes = v_head_dim is None or v_head_dim == head_dim
     plain = not (softcap or keep_first or sink is not None or dist is not None or gate is not None)
+    span = window if window else -int(chunk or 0)
+    if qkv.dtype == torch.bfloat16 and not same_sizes and not (window and chunk) and plain:
+        done = _own_value_size(qkv, cache_layer, out, ctx, n_heads=n_heads, n_kv_heads=n_kv_heads, head_dim=head_dim,
+                               v_head_dim=v_head_dim, scale=scale, span=span, out_scale=out_scale)
+        if done is not None:
+            return done
     if qkv.dtype == torch.bfloat16 and same_sizes and not (window and chunk) and plain:
-        span = window if window else -int(chunk or 0)
         decode = ctx.all_single
         if ops.attention_mma_supports(head_dim, ctx.page_size, n_heads, n_kv_heads, decode):
             if decode:
@@ -177,6 +185,34 @@ def attention(qkv, cache_layer, out, ctx, *, n_heads, n_kv_heads, head_dim, scal
         head_dim=head_dim, page_size=ctx.page_size, scale=scale, window=window, chunk=chunk or 0,
         v_head_dim=v_head_dim, out_scale=out_scale, softcap=softcap, keep_first=keep_first, sink=sink, dist=dist,
         gate=gate)
+
+
+def _own_value_size(qkv, cache_layer, out, ctx, *, n_heads, n_kv_heads, head_dim, v_head_dim, scale, span, out_scale):
+    """`attention` on the tensor cores for values of another head size than the keys'; None where no kernel takes the sizes."""
+    from . import attention_tc
+    q_ld = qkv.shape[1]
+    if ctx.all_single:
+        if not (ops.attention_mma_supports(head_dim, ctx.page_size, n_heads, n_kv_heads, True) and q_ld % 8 == 0
+                and attention_tc.decode_supports(head_dim, v_head_dim)):
+            return None
+        name, splits = decode_plan(ctx.n_seqs, n_kv_heads, ctx.page_table.shape[1] * ctx.page_size, ctx.page_size, head_dim, v_head_dim)
+        part_o = part_ml = None
+        if splits > 1 and name != "cluster":
+            part_o = ctx.buffer("attn_part_o", (ctx.n_seqs * n_heads * splits * v_head_dim,), torch.float32)
+            part_ml = ctx.buffer("attn_part_ml", (ctx.n_seqs * n_heads * splits * 2,), torch.float32)
+        kernel = attention_tc.decode_cluster if name == "cluster" else attention_tc.decode
+        kernel(qkv, q_ld, cache_layer.k, cache_layer.v, ctx.page_table, ctx.seq_slot, ctx.seq_len, ctx.cu_seqlens, out,
+               n_seqs=ctx.n_seqs, n_heads=n_heads, n_kv_heads=n_kv_heads, head_dim=head_dim, page_size=ctx.page_size, scale=scale,
+               window=span, n_splits=splits, part_o=part_o, part_ml=part_ml)
+        if out_scale != 1.0:
+            ops.scale_(out, out_scale)
+        return out
+    if not attention_tc.supports(head_dim, ctx.page_size, n_heads, n_kv_heads, q_ld, out.shape[1], v_head_dim):
+        return None
+    return attention_tc.prefill(
+        qkv, cache_layer.k, cache_layer.v, ctx.page_table, ctx.seq_slot, ctx.seq_start, ctx.cu_seqlens, out, n_seqs=ctx.n_seqs,
+        max_new=ctx.max_new, n_heads=n_heads, n_kv_heads=n_kv_heads, head_dim=head_dim, page_size=ctx.page_size, scale=scale,
+        window=span, out_scale=out_scale)
 
 
 # RI_B200_LATENT_ATTENTION=generic keeps the generic kernel for attention over a shared latent (for comparisons)
