@@ -869,7 +869,115 @@ rope_normed_cache_write_vec_kernel(__nv_bfloat16* __restrict__ qkv, int ld, cons
         *reinterpret_cast<uint4*>(dst + ch) = pack8(y);
     }
 }
+
+// The same from float32 accumulators of a K-split projection [n_tokens, ld] (q, k and value columns; `bias`, one number per
+// column or null, not yet added): the queries go to q_out [n_tokens, n_heads * hd], the values are rounded to T first, as a
+// projection in T would leave them, and kept in v_keep [n_tokens, n_kv_heads * v_hd] as well where one is given, and the
+// accumulators are left zeroed.  For steps of few tokens.
+template <typename T>
+__global__ void __launch_bounds__(NORMED_ROPE_WARPS * 32)
+rope_normed_cache_write_acc_kernel(float* __restrict__ acc, int ld, const float* __restrict__ bias, T* __restrict__ q_out,
+                                   T* __restrict__ v_keep, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
+                                   const float* __restrict__ q_w, const float* __restrict__ k_w, float eps,
+                                   const int* __restrict__ token_pos, const int* __restrict__ token_seq,
+                                   const int* __restrict__ seq_slot, const int* __restrict__ page_table, int max_pages,
+                                   T* __restrict__ kcache, T* __restrict__ vcache, int n_tokens, int n_heads, int n_kv_heads, int hd,
+                                   int page_size, int style, int rot, int v_hd, const float* __restrict__ mix,
+                                   const T* v_other, int v_other_ld) {
+    extern __shared__ float head_smem[];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    float* x = head_smem + (size_t)warp * hd;
+    const int heads = n_heads + 2 * n_kv_heads;
+    const long long item = (long long)blockIdx.x * NORMED_ROPE_WARPS + warp;
+    let_next_kernel_start();
+    if (item >= (long long)n_tokens * heads) return;
+    const int t = (int)(item / heads), h = (int)(item % heads);
+    const int pos = token_pos[t];                     // positions, slots, pages and angles: fixed before the step
+    const int half = rot >> 1;
+    const float* c = cos_t + (size_t)pos * half;
+    const float* s = sin_t + (size_t)pos * half;
+    size_t cache_row = 0;
+    bool store = true;
+    if (h >= n_heads) {
+        const int slot = seq_slot[token_seq[t]];
+        if (!RI_IN_LIMIT(slot, RI_LIMIT_SLOTS, RI_CHECK_SLOT) || !RI_IN_RANGE(pos / page_size, max_pages, RI_CHECK_PAGE_INDEX)) {
+            store = false;
+        } else {
+            const int page = page_table[(size_t)slot * max_pages + pos / page_size];
+            if (!RI_IN_LIMIT(page, RI_LIMIT_PAGES, RI_CHECK_PAGE)) store = false;
+            cache_row = (size_t)page * n_kv_heads * page_size + (pos % page_size);
+        }
+    }
+    wait_for_previous_kernels();          // the projections come from the previous kernel
+    const int kh = h - n_heads, vh = kh - n_kv_heads;
+    const bool is_v = vh >= 0;
+    const int col = is_v ? (n_heads + n_kv_heads) * hd + vh * v_hd : h * hd;
+    float* src = acc + (size_t)t * ld + col;
+    if (is_v) {
+        const float m = mix != nullptr ? mix[0] : 0.f;
+        for (int d = lane; d < v_hd; d += 32) {
+            const T own = from_f32<T>(src[d] + (bias != nullptr ? bias[col + d] : 0.f));
+            src[d] = 0.f;
+            float v = to_f32<T>(own);
+            if (v_keep != nullptr) v_keep[((size_t)t * n_kv_heads + vh) * v_hd + d] = own;
+            if (mix != nullptr) v = (1.f - m) * v + m * to_f32<T>(v_other[(size_t)t * v_other_ld + (size_t)vh * v_hd + d]);
+            if (store) vcache[(cache_row + (size_t)vh * page_size) * v_hd + d] = from_f32<T>(v);
+        }
+        return;
+    }
+    float ss = 0.f;
+    for (int d = lane; d < hd; d += 32) {
+        const float v = src[d] + (bias != nullptr ? bias[col + d] : 0.f);
+        src[d] = 0.f;
+        x[d] = v;
+        ss += v * v;
+    }
+    const float* w = kh < 0 ? q_w : k_w;
+    if (w != nullptr) {
+        ss = warp_sum(ss);
+        const float scale = 1.0f / sqrtf(ss / (float)hd + eps);
+        for (int d = lane; d < hd; d += 32) x[d] = x[d] * scale * w[d];
+    }
+    __syncwarp();
+    if (!store) return;
+    T* dst = kh < 0 ? q_out + ((size_t)t * n_heads + h) * hd : kcache + (cache_row + (size_t)kh * page_size) * hd;
+    for (int i = lane; i < half; i += 32) {
+        const int i0 = style == 0 ? i : 2 * i;
+        const int i1 = style == 0 ? i + half : 2 * i + 1;
+        const float x0 = x[i0], x1 = x[i1];
+        dst[i0] = from_f32<T>(x0 * c[i] - x1 * s[i]);
+        dst[i1] = from_f32<T>(x0 * s[i] + x1 * c[i]);
+    }
+    for (int d = rot + lane; d < hd; d += 32) dst[d] = from_f32<T>(x[d]);
+}
 }  // namespace
+
+// Every layer writes its keys and values here (there is no reading form).
+RI_API int ri_rope_normed_cache_write_acc(float* acc, int ld, const float* bias, void* q_out, void* v_keep, int dtype, const float* cos_t,
+                                          const float* sin_t, const float* q_w, const float* k_w, float eps, const int* token_pos,
+                                          const int* token_seq, const int* seq_slot, const int* page_table, int max_pages, void* kcache,
+                                          void* vcache, int n_tokens, int n_heads, int n_kv_heads, int hd, int page_size, int style, int rot,
+                                          int v_hd, const float* mix, const void* v_other, int v_other_ld, cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    if (rot < 0 || rot % 2 || rot > hd) return fail("rope_normed_cache_write_acc: %d rotated channels of a head of %d", rot, hd);
+    if (rot > 0 && (cos_t == nullptr || sin_t == nullptr)) return fail("rope_normed_cache_write_acc: a rotation needs its tables");
+    if (style != 0 && style != 1) return fail("rope_normed_cache_write_acc: unknown style %d", style);
+    if (mix != nullptr && (v_other == nullptr || v_other_ld < n_kv_heads * v_hd))
+        return fail("rope_normed_cache_write_acc: blended values need the rows they are blended with");
+    const size_t smem = (size_t)NORMED_ROPE_WARPS * hd * sizeof(float);
+    if (smem > 48 * 1024) return fail("rope_normed_cache_write_acc: heads of %d exceed %d", hd, 48 * 1024 / 4 / NORMED_ROPE_WARPS);
+    const long long items = (long long)n_tokens * (n_heads + 2 * n_kv_heads);
+    const unsigned blocks = (unsigned)((items + NORMED_ROPE_WARPS - 1) / NORMED_ROPE_WARPS);
+    cudaError_t e;
+#define RI_NORMED_ROPE_ACC(T) launch_dependent(rope_normed_cache_write_acc_kernel<T>, blocks, NORMED_ROPE_WARPS * 32, smem, stream, acc, ld, \
+        bias, (T*)q_out, (T*)v_keep, cos_t, sin_t, q_w, k_w, eps, token_pos, token_seq, seq_slot, page_table, max_pages, (T*)kcache, \
+        (T*)vcache, n_tokens, n_heads, n_kv_heads, hd, page_size, style, rot, v_hd, mix, (const T*)v_other, v_other_ld)
+    if (dtype == RI_F32) e = RI_NORMED_ROPE_ACC(float);
+    else if (dtype == RI_BF16) e = RI_NORMED_ROPE_ACC(__nv_bfloat16);
+    else return fail("rope_normed_cache_write_acc: unknown dtype %d", dtype);
+#undef RI_NORMED_ROPE_ACC
+    return check_launch(e, "rope_normed_cache_write_acc");
+}
 
 RI_API int ri_rope_normed_cache_write(void* qkv, int dtype, int ld, const float* cos_t, const float* sin_t,
                                       const float* q_w, const float* k_w, float eps, const int* token_pos,

@@ -26,10 +26,12 @@ namespace {
 
 constexpr int PREPARE_HEADS = 4;    // query heads per block of the preparing kernel
 
-// grid (tokens, groups of PREPARE_HEADS heads); the first group's block also writes the cache row and the lists
-template <typename T>
+// grid (tokens, groups of PREPARE_HEADS heads); the first group's block also writes the cache row and the lists.
+// TI: what the projection is held in; float beside a 16-bit T: accumulators of a K-split projection, left zeroed (every
+// element by the thread that read it last)
+template <typename T, typename TI>
 __global__ void __launch_bounds__(128)
-latent_prepare_kernel(const T* __restrict__ proj, int ld, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
+latent_prepare_kernel(TI* __restrict__ proj, int ld, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
                       const float* __restrict__ c_w, float eps, const int* __restrict__ token_pos,
                       const int* __restrict__ token_seq, const int* __restrict__ seq_slot,
                       const int* __restrict__ page_table, int max_pages, T* __restrict__ cache, T* __restrict__ q_nope,
@@ -45,11 +47,17 @@ latent_prepare_kernel(const T* __restrict__ proj, int ld, const float* __restric
     const float* s = sin_t + (size_t)pos * half;
     let_next_kernel_start();
     wait_for_previous_kernels();                      // the projection; and the lists may still be read by the layer before
-    const T* row = proj + (size_t)t * ld;
+    constexpr bool ZERO = sizeof(TI) != sizeof(T);
+    TI* row = proj + (size_t)t * ld;
     const int qh = d + rd, wide = rank + rd;
 
     // queries: the unrotated parts head by head, the rotated parts into the wide rows
-    if (vec) {                                        // 2-byte values, 16 bytes at a time
+    auto take = [&](int i) {                          // the projection's element i of this token
+        const float v = to_f32<TI>(row[i]);
+        if (ZERO) row[i] = from_f32<TI>(0.f);
+        return v;
+    };
+    if (!ZERO && vec) {                               // 2-byte values, 16 bytes at a time
         const int d8 = d >> 3;
         for (int i = tid; i < nh * d8; i += blockDim.x) {
             const int h = h0 + i / d8, j = (i % d8) * 8;
@@ -58,21 +66,20 @@ latent_prepare_kernel(const T* __restrict__ proj, int ld, const float* __restric
     } else {
         for (int i = tid; i < nh * d; i += blockDim.x) {
             const int h = h0 + i / d, j = i % d;
-            q_nope[((size_t)h * n_tokens + t) * d + j] = row[h * qh + j];
+            q_nope[((size_t)h * n_tokens + t) * d + j] = from_f32<T>(take(h * qh + j));
         }
     }
     for (int i = tid; i < nh * half; i += blockDim.x) {
         const int h = h0 + i / half, k = i % half;
         const int i0 = style == 0 ? k : 2 * k, i1 = style == 0 ? k + half : 2 * k + 1;
-        const T* v = row + h * qh + d;
-        const float x0 = to_f32<T>(v[i0]), x1 = to_f32<T>(v[i1]);
+        const float x0 = take(h * qh + d + i0), x1 = take(h * qh + d + i1);
         T* dst = q_wide + ((size_t)t * n_heads + h) * wide + rank;
         dst[i0] = from_f32<T>(x0 * c[k] - x1 * s[k]);
         dst[i1] = from_f32<T>(x0 * s[k] + x1 * c[k]);
     }
     for (int i = tid; i < nh * (rd - rot); i += blockDim.x) {
         const int h = h0 + i / (rd - rot), j = rot + i % (rd - rot);
-        q_wide[((size_t)t * n_heads + h) * wide + rank + j] = row[h * qh + d + j];
+        q_wide[((size_t)t * n_heads + h) * wide + rank + j] = from_f32<T>(take(h * qh + d + j));
     }
     if (blockIdx.y != 0) return;
 
@@ -91,27 +98,28 @@ latent_prepare_kernel(const T* __restrict__ proj, int ld, const float* __restric
     if (!write_kv) return;
 
     // the cache row: normalised latent, rotated key part
-    const T* lat = row + (size_t)n_heads * qh;
+    const int lat = n_heads * qh;
     float ss = 0.f;
     for (int j = tid; j < rank; j += blockDim.x) {
-        const float v = to_f32<T>(lat[j]);
+        const float v = to_f32<TI>(row[lat + j]);
         ss += v * v;
     }
     ss = block_sum(ss, scratch);
     const float scale = 1.0f / sqrtf(ss / (float)rank + eps);
     const int slot = seq_slot[token_seq[t]];
+    // checked build: a slot, a page index or a page outside its range is recorded and nothing is written
     if (!RI_BLOCK_IN_LIMIT(slot, RI_LIMIT_SLOTS, RI_CHECK_SLOT) || !RI_BLOCK_IN_RANGE(pos / page_size, max_pages, RI_CHECK_PAGE_INDEX)) return;
     const int page = page_table[(size_t)slot * max_pages + pos / page_size];
     if (!RI_BLOCK_IN_LIMIT(page, RI_LIMIT_PAGES, RI_CHECK_PAGE)) return;
     T* dst = cache + ((size_t)page * page_size + (pos % page_size)) * wide;
-    for (int j = tid; j < rank; j += blockDim.x) dst[j] = from_f32<T>(to_f32<T>(lat[j]) * scale * c_w[j]);
+    for (int j = tid; j < rank; j += blockDim.x) dst[j] = from_f32<T>(take(lat + j) * scale * c_w[j]);
     for (int k = tid; k < half; k += blockDim.x) {
         const int i0 = style == 0 ? k : 2 * k, i1 = style == 0 ? k + half : 2 * k + 1;
-        const float x0 = to_f32<T>(lat[rank + i0]), x1 = to_f32<T>(lat[rank + i1]);
+        const float x0 = take(lat + rank + i0), x1 = take(lat + rank + i1);
         dst[rank + i0] = from_f32<T>(x0 * c[k] - x1 * s[k]);
         dst[rank + i1] = from_f32<T>(x0 * s[k] + x1 * c[k]);
     }
-    for (int j = rot + tid; j < rd; j += blockDim.x) dst[rank + j] = lat[rank + j];
+    for (int j = rot + tid; j < rd; j += blockDim.x) dst[rank + j] = from_f32<T>(take(lat + rank + j));
 }
 
 template <typename T>
@@ -187,11 +195,11 @@ int blocks_for(size_t total) {
 
 }  // namespace
 
-// proj: [T, ld], the heads' queries from column 0, then (write_kv) the latent and its key part.  cache: one layer,
+// proj: [T, ld] in dtype, or with proj_is_acc float32 accumulators that are left zeroed; the heads' queries from column 0, then (write_kv) the latent and its key part.  cache: one layer,
 // [pages, 1, page_size, rank + rd].  q_nope [heads, T, d], q_wide [T, heads, rank + rd] (its last rd channels are
 // written here).  offsets int32 [heads + 1], order int32 [heads * T], tiles int32 [2 * heads * ceil(T / tile_rows)],
 // n_tiles int32 [1].
-RI_API int ri_latent_prepare(const void* proj, int dtype, int ld, const float* cos_t, const float* sin_t, const float* c_w,
+RI_API int ri_latent_prepare(void* proj, int proj_is_acc, int dtype, int ld, const float* cos_t, const float* sin_t, const float* c_w,
                              float eps, const int* token_pos, const int* token_seq, const int* seq_slot,
                              const int* page_table, int max_pages, void* cache, void* q_nope, void* q_wide, int* offsets,
                              int* order, int* tiles, int* n_tiles, int n_tokens, int n_heads, int d, int rd, int rank,
@@ -204,14 +212,15 @@ RI_API int ri_latent_prepare(const void* proj, int dtype, int ld, const float* c
     if ((long long)n_heads * n_tokens > 0x7fffffffLL) return fail("latent_prepare: %d heads x %d tokens exceed 2^31", n_heads, n_tokens);
     const int groups = (n_heads + PREPARE_HEADS - 1) / PREPARE_HEADS;
     if (groups > 65535) return fail("latent_prepare: %d heads exceed the grid limit", n_heads);
-    const int vec = dtype == RI_BF16 && d % 8 == 0 && rd % 8 == 0 && ld % 8 == 0 && (uintptr_t)proj % 16 == 0 && (uintptr_t)q_nope % 16 == 0;
+    const int vec = dtype == RI_BF16 && !proj_is_acc && d % 8 == 0 && rd % 8 == 0 && ld % 8 == 0 && (uintptr_t)proj % 16 == 0 && (uintptr_t)q_nope % 16 == 0;
     const dim3 grid(n_tokens, groups);
     cudaError_t e;
-#define RI_PREPARE(T) launch_dependent(latent_prepare_kernel<T>, grid, dim3(128), (size_t)0, stream, (const T*)proj, ld, cos_t, sin_t, \
+#define RI_PREPARE(T, TI) launch_dependent(latent_prepare_kernel<T, TI>, grid, dim3(128), (size_t)0, stream, (TI*)proj, ld, cos_t, sin_t, \
         c_w, eps, token_pos, token_seq, seq_slot, page_table, max_pages, (T*)cache, (T*)q_nope, (T*)q_wide, offsets, order, \
         tiles, n_tiles, n_tokens, n_heads, d, rd, rank, rot, style, page_size, write_kv, tile_rows, vec)
-    if (dtype == RI_F32) e = RI_PREPARE(float);
-    else if (dtype == RI_BF16) e = RI_PREPARE(__nv_bfloat16);
+    if (dtype == RI_F32) e = RI_PREPARE(float, float);
+    else if (dtype == RI_BF16 && proj_is_acc) e = RI_PREPARE(__nv_bfloat16, float);
+    else if (dtype == RI_BF16) e = RI_PREPARE(__nv_bfloat16, __nv_bfloat16);
     else return fail("latent_prepare: unknown dtype %d", dtype);
 #undef RI_PREPARE
     return check_launch(e, "latent_prepare");

@@ -79,7 +79,7 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32)
 moe_route_kernel(const T* x, const float* __restrict__ router, const float* __restrict__ correction, const float* __restrict__ bias,
                  const float* __restrict__ gate_w, int* __restrict__ ids, float* __restrict__ weights,
                  float* __restrict__ gate_out, int n_tokens, int width, int experts, int top, int groups, int keep,
-                 int per_block, int form, float* split_sums, int* split_count) {
+                 int per_block, int form, int always, float* split_sums, int* split_count) {
     extern __shared__ float smem[];
     __shared__ int last_ticket;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -200,7 +200,12 @@ moe_route_kernel(const T* x, const float* __restrict__ router, const float* __re
         __syncwarp();
     }
 
-    // `top` rounds of taking the best remaining expert
+    // `top` rounds of taking the best remaining expert; behind them the ids that every token has
+    const int ld = top + always;
+    for (int c = lane; c < always; c += 32) {
+        ids[(size_t)t * ld + top + c] = experts + c;
+        weights[(size_t)t * ld + top + c] = 1.f;
+    }
     float sum = 0.f;
     for (int c = 0; c < top; ++c) {
         float bv = -INFINITY;
@@ -214,15 +219,15 @@ moe_route_kernel(const T* x, const float* __restrict__ router, const float* __re
         const float s = score[bi];
         sum += s;
         if (lane == 0) {
-            ids[(size_t)t * top + c] = bi;
-            weights[(size_t)t * top + c] = s;
+            ids[(size_t)t * ld + c] = bi;
+            weights[(size_t)t * ld + c] = s;
             choice[bi] = NAN;                    // taken
         }
         __syncwarp();
     }
     if (form & 2) return;                        // the weights are the scores as they are
     const float inv = 1.0f / (sum + 1e-20f);
-    for (int c = lane; c < top; c += 32) weights[(size_t)t * top + c] *= inv;
+    for (int c = lane; c < top; c += 32) weights[(size_t)t * ld + c] *= inv;
 }
 
 // ---- arrange ---------------------------------------------------------------------------------
@@ -406,13 +411,16 @@ __global__ void moe_combine_kernel(float* residual, const float* y, const float*
 
 // form: bit 0 softmax scores instead of sigmoid ones, bit 1 weights not divided by their sum, bit 2 a group counts by its
 // largest score instead of the sum of its two largest.  correction and bias may be null.
+// always > 0: a token's ids are its top chosen ones and then experts, experts + 1, .. (so many, with weight 1): rows of ids and
+// weights hold top + always entries.
 // split > 1 (steps of up to ROUTE_SPLIT_TOKENS tokens): the router's rows are cut over that many blocks per token;
 // split_sums: float32 [n_tokens, experts + 1] scratch, split_count: int32 [n_tokens], zero before the call and after it.
 RI_API int ri_moe_route(const void* x, int dtype, const float* router, const float* correction, const float* bias, const float* gate_w,
                         int* ids, float* weights, float* gate_out, int n_tokens, int width, int experts, int top,
-                        int groups, int keep, int form, int split, float* split_sums, int* split_count,
+                        int groups, int keep, int form, int always, int split, float* split_sums, int* split_count,
                         cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
+    if (always < 0) return fail("moe_route: %d ids that every token has", always);
     if (experts <= 0 || top <= 0 || top > experts) return fail("moe_route: top %d of %d experts", top, experts);
     if (groups <= 0 || experts % groups || keep <= 0 || keep > groups)
         return fail("moe_route: %d experts in %d groups, %d kept", experts, groups, keep);
@@ -430,7 +438,7 @@ RI_API int ri_moe_route(const void* x, int dtype, const float* router, const flo
     cudaError_t e;
 #define RI_ROUTE_N(T, V, N) launch_dependent(moe_route_kernel<T, V, N>, blocks, ROUTE_WARPS * 32, smem, stream, (const T*)x, \
                                              router, correction, bias, gate_w, ids, weights, gate_out, n_tokens, width, experts, top,   \
-                                             groups, keep, per_block, form, split_sums, split_count)
+                                             groups, keep, per_block, form, always, split_sums, split_count)
 #define RI_ROUTE(T, V) (per_block == 1 ? RI_ROUTE_N(T, V, 1) : per_block == 2 ? RI_ROUTE_N(T, V, 2) : RI_ROUTE_N(T, V, ROUTE_TOKENS))
     if (dtype == RI_F32) e = vec ? RI_ROUTE(float, true) : RI_ROUTE(float, false);
     else if (dtype == RI_BF16) e = vec ? RI_ROUTE(__nv_bfloat16, true) : RI_ROUTE(__nv_bfloat16, false);

@@ -270,6 +270,45 @@ def rope_normed_cache_write(qkv: torch.Tensor, cos: torch.Tensor, sin: torch.Ten
           c_int(1 if values_from_keys else 0), _p(lam), _p(other), c_int(0 if other is None else other.stride(0)), _stream())
 
 
+def rope_normed_cache_write_acc(acc: torch.Tensor, bias, q_out: torch.Tensor, cos, sin, q_weight, k_weight, eps: float, token_pos, token_seq,
+                                seq_slot, page_table: torch.Tensor, kcache, vcache, *, n_heads: int, n_kv_heads: int, head_dim: int,
+                                page_size: int, style: int, rot_dims: int | None = None, v_head_dim: int | None = None,
+                                value_mix: tuple | None = None, v_keep: torch.Tensor | None = None) -> None:
+    """`rope_normed_cache_write` from float32 accumulators [T, columns] of a K-split projection (`bias` float32 [columns] or
+    None, not yet added): the queries go to q_out, keys and values to the cache, the projected values into v_keep
+    [T, n_kv_heads * v_head_dim] as well where one is given; `acc` is left zeroed."""
+    _need_cuda(acc, bias, q_out, cos, sin, q_weight, k_weight, token_pos, token_seq, seq_slot, page_table, kcache, vcache, v_keep)
+    n = acc.shape[0]
+    rot = head_dim if rot_dims is None else int(rot_dims)
+    v_hd = head_dim if v_head_dim is None else int(v_head_dim)
+    cols = (n_heads + n_kv_heads) * head_dim + n_kv_heads * v_hd
+    _need(acc.dtype == torch.float32 and acc.is_contiguous() and acc.shape[1] == cols, "rope_normed_cache_write_acc: accumulators")
+    _need(q_out.is_contiguous() and tuple(q_out.shape) == (n, n_heads * head_dim), "rope_normed_cache_write_acc: q_out")
+    _need(0 <= rot <= head_dim and rot % 2 == 0, "rope_normed_cache_write_acc: rotated channels must be even and at most head_dim")
+    _need(rot == 0 or (cos.dtype == torch.float32 and sin.dtype == torch.float32 and cos.shape[1] == rot // 2 and cos.is_contiguous()
+                       and sin.is_contiguous()), "rope_normed_cache_write_acc: tables must be float32 [positions, rotated channels / 2]")
+    for w, size in ((q_weight, head_dim), (k_weight, head_dim), (bias, cols)):
+        if w is not None:
+            _f32_vec(w, size, "rope_normed_cache_write_acc: norm weights and bias")
+    _need(kcache.dtype == q_out.dtype and vcache.dtype == q_out.dtype and kcache.is_contiguous() and vcache.is_contiguous()
+          and tuple(kcache.shape[1:]) == (n_kv_heads, page_size, head_dim) and tuple(vcache.shape[1:]) == (n_kv_heads, page_size, v_hd),
+          "rope_normed_cache_write_acc: cache")
+    _need(v_keep is None or (v_keep.dtype == q_out.dtype and v_keep.is_contiguous() and tuple(v_keep.shape) == (n, n_kv_heads * v_hd)),
+          "rope_normed_cache_write_acc: v_keep")
+    lam = other = None
+    if value_mix is not None:
+        lam, rows, col = value_mix
+        _need_cuda(lam, rows)
+        _need(lam.dtype == torch.float32 and lam.numel() == 1 and rows.dtype == q_out.dtype and rows.dim() == 2 and rows.is_contiguous()
+              and rows.shape[0] >= n and 0 <= col and rows.shape[1] >= col + n_kv_heads * v_hd, "rope_normed_cache_write_acc: the values to blend in")
+        other = rows[:, col:]
+    _call("elementwise", "ri_rope_normed_cache_write_acc", _p(acc), c_int(acc.shape[1]), _p(bias), _p(q_out), _p(v_keep),
+          c_int(dtype_code(q_out.dtype)), _p(cos), _p(sin), _p(q_weight), _p(k_weight), c_float(eps), _p(token_pos), _p(token_seq),
+          _p(seq_slot), _p(page_table), c_int(page_table.shape[1]), _p(kcache), _p(vcache), c_int(n), c_int(n_heads), c_int(n_kv_heads),
+          c_int(head_dim), c_int(page_size), c_int(style), c_int(rot), c_int(v_hd), _p(lam), _p(other),
+          c_int(0 if other is None else other.stride(0)), _stream())
+
+
 def rope_cache_write(qkv: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor, token_pos, token_seq,
                      seq_slot, page_table: torch.Tensor, kcache, vcache, *, n_heads: int,
                      n_kv_heads: int, head_dim: int, page_size: int, style: int, write_kv: bool,
@@ -795,14 +834,16 @@ def moe_route(x: torch.Tensor, router: torch.Tensor, correction: torch.Tensor | 
               weights: torch.Tensor, *, top: int, groups: int = 1, keep: int = 1,
               gate_weight: torch.Tensor | None = None, gate_out: torch.Tensor | None = None,
               softmax: bool = False, normalise: bool = True, split: int = 1, split_sums: torch.Tensor | None = None,
-              split_count: torch.Tensor | None = None, group_max: bool = False, bias: torch.Tensor | None = None) -> None:
+              split_count: torch.Tensor | None = None, group_max: bool = False, bias: torch.Tensor | None = None,
+              always: int = 0) -> None:
     """Per token the `top` experts with the largest sigmoid(router x) + correction among the `keep` best of
     `groups` groups (a group's score: the sum of its two largest, or with group_max its largest alone; correction None:
     zero), ids int32 [T, top], and their weights
     float32 [T, top] (the plain sigmoid scores, normalised).  gate_weight float32 [width]: gate_out[t] =
     sigmoid(gate_weight . x_t) as well.  softmax: the scores are softmax(router x) over all experts instead of
     sigmoids; normalise False: the weights are the chosen scores as they are.  bias float32 [experts]: added to
-    router x before the sigmoid or softmax.  split > 1 (steps of fewer than 296
+    router x before the sigmoid or softmax.  always: so many ids from `experts` on that every token has after its chosen ones,
+    with weight 1 (ids and weights are then [T, top + always]).  split > 1 (steps of fewer than 296
     tokens): the router's rows are cut over that many blocks per token, which leave their sums in split_sums (float32
     [T, experts + 1]) and count themselves in split_count (int32 [T], zero before the call and after it)."""
     _need_cuda(x, router, correction, ids, weights, gate_weight, gate_out, bias)
@@ -812,8 +853,8 @@ def moe_route(x: torch.Tensor, router: torch.Tensor, correction: torch.Tensor | 
           and (correction is None or (correction.dtype == torch.float32 and correction.numel() == experts)), "moe_route: router and correction")
     if bias is not None:
         _f32_vec(bias, experts, "moe_route: bias")
-    _need(ids.dtype == torch.int32 and ids.is_contiguous() and ids.numel() >= n * top and weights.dtype == torch.float32
-          and weights.is_contiguous() and weights.numel() >= n * top, "moe_route: ids int32 and weights float32 [T, top]")
+    _need(ids.dtype == torch.int32 and ids.is_contiguous() and ids.numel() >= n * (top + always) and weights.dtype == torch.float32
+          and weights.is_contiguous() and weights.numel() >= n * (top + always), "moe_route: ids int32 and weights float32 [T, top]")
     _need((gate_weight is None) == (gate_out is None), "moe_route: gate weight and output go together")
     if gate_weight is not None:
         _need(gate_weight.dtype == torch.float32 and gate_weight.is_contiguous() and gate_weight.numel() == width
@@ -825,7 +866,7 @@ def moe_route(x: torch.Tensor, router: torch.Tensor, correction: torch.Tensor | 
               and split_count.numel() >= n, "moe_route: rows cut over blocks need few tokens, float32 sums and int32 counters")
     _call("moe", "ri_moe_route", _p(x), c_int(dtype_code(x.dtype)), _p(router), _p(correction), _p(bias), _p(gate_weight), _p(ids),
           _p(weights), _p(gate_out), c_int(n), c_int(width), c_int(experts), c_int(top), c_int(groups), c_int(keep),
-          c_int((1 if softmax else 0) | (0 if normalise else 2) | (4 if group_max else 0)), c_int(max(1, split)), _p(split_sums if split > 1 else None),
+          c_int((1 if softmax else 0) | (0 if normalise else 2) | (4 if group_max else 0)), c_int(always), c_int(max(1, split)), _p(split_sums if split > 1 else None),
           _p(split_count if split > 1 else None), _stream())
 
 
@@ -922,7 +963,8 @@ def latent_prepare(proj: torch.Tensor, cos, sin, latent_weight, eps: float, toke
                    cache, q_nope: torch.Tensor, q_wide: torch.Tensor, offsets, order, tiles, n_tiles, *, n_heads: int,
                    head_dim: int, rot_dim: int, rank: int, rot_dims: int, style: int, page_size: int, write_kv: bool,
                    tile_rows: int) -> None:
-    """From the projection [T, heads * (head_dim + rot_dim) (+ rank + rot_dim ...)]: the heads' unrotated query
+    """From the projection [T, heads * (head_dim + rot_dim) (+ rank + rot_dim ...)] (in the run dtype, or float32 accumulators of a
+    K-split projection, which are left zeroed): the heads' unrotated query
     parts head by head into q_nope [heads, T, head_dim], their rotated parts into the last rot_dim channels of
     q_wide [T, heads, rank + rot_dim]; with write_kv the RMS-normalised latent (times latent_weight) and the rotated
     key part into the token's row of `cache` [pages, 1, page_size, rank + rot_dim]; and the lists of the per-head
@@ -933,21 +975,23 @@ def latent_prepare(proj: torch.Tensor, cos, sin, latent_weight, eps: float, toke
     wide = rank + rot_dim
     need_cols = n_heads * (head_dim + rot_dim) + (wide if write_kv else 0)
     _need(proj.is_contiguous() and proj.shape[1] >= need_cols, "latent_prepare: the projection holds too few columns")
-    _need(q_nope.dtype == proj.dtype and q_wide.dtype == proj.dtype and q_nope.is_contiguous() and q_wide.is_contiguous()
+    zeroed = proj.dtype != q_wide.dtype
+    _need(proj.dtype in (q_wide.dtype, torch.float32), "latent_prepare: the projection must be float32 or of the run dtype")
+    _need(q_nope.dtype == q_wide.dtype and q_nope.is_contiguous() and q_wide.is_contiguous()
           and q_nope.numel() == n * n_heads * head_dim and q_wide.numel() == n * n_heads * wide, "latent_prepare: query buffers")
     _need(cos.dtype == torch.float32 and sin.dtype == torch.float32 and cos.shape[1] == rot_dims // 2 and cos.is_contiguous()
           and sin.is_contiguous() and 0 < rot_dims <= rot_dim and rot_dims % 2 == 0, "latent_prepare: rotation tables")
     if write_kv:
         _need(latent_weight is not None and latent_weight.dtype == torch.float32 and latent_weight.numel() == rank,
               "latent_prepare: the latent's norm weight must be float32 [rank]")
-        _need(cache.dtype == proj.dtype and cache.is_contiguous() and tuple(cache.shape[1:]) == (1, page_size, wide),
+        _need(cache.dtype == q_wide.dtype and cache.is_contiguous() and tuple(cache.shape[1:]) == (1, page_size, wide),
               "latent_prepare: cache shape")
     per_head = -(-n // tile_rows)
     for t in (offsets, order, tiles, n_tiles):
         _need(t.dtype == torch.int32 and t.is_contiguous(), "latent_prepare: int32 lists")
     _need(offsets.numel() >= n_heads + 1 and order.numel() >= n_heads * n and tiles.numel() >= 2 * n_heads * per_head,
           "latent_prepare: lists too small")
-    _call("latent", "ri_latent_prepare", _p(proj), c_int(dtype_code(proj.dtype)), c_int(proj.shape[1]), _p(cos), _p(sin),
+    _call("latent", "ri_latent_prepare", _p(proj), c_int(1 if zeroed else 0), c_int(dtype_code(q_wide.dtype)), c_int(proj.shape[1]), _p(cos), _p(sin),
           _p(latent_weight), c_float(eps), _p(token_pos), _p(token_seq), _p(seq_slot), _p(page_table),
           c_int(page_table.shape[1]), _p(cache), _p(q_nope), _p(q_wide), _p(offsets), _p(order), _p(tiles), _p(n_tiles),
           c_int(n), c_int(n_heads), c_int(head_dim), c_int(rot_dim), c_int(rank), c_int(rot_dims), c_int(style),
@@ -1078,13 +1122,16 @@ def stream_update(stream_x: torch.Tensor, *, branch=None, branch_bias=None, post
 
 
 MAX_STREAMS = 16             # parallel streams `streams_step` takes
+MAX_SUMMED_EXPERTS = 32      # rows of a token it sums
 
 
-def streams_step(x: torch.Tensor, streams: int, *, branch=None, scale=None, mix=None, write=None, read=None, norm=None,
-                 eps: float = 0.0, out=None, rows=None) -> None:
+def streams_step(x: torch.Tensor, streams: int, *, branch=None, experts: dict | None = None, scale=None, mix=None, write=None,
+                 read=None, norm=None, eps: float = 0.0, out=None, rows=None) -> None:
     """One pass over `streams` parallel hidden streams x (float32 [T, streams * n], a token's streams side by side).  With
     `branch` (float32 [T, n], left zeroed): x_t <- sum_s mix[s, t] x_s + write[t] * branch * scale, all streams at once from
-    the old ones (mix float32 [from, to], write float32 [streams], scale float32 [n] or None).  With `out`:
+    the old ones (mix float32 [from, to], write float32 [streams], scale float32 [n] or None).  `experts` in place of a branch:
+    a dict y (float32 rows [pairs, n]), weights (float32 [T, top]), top, place (int32 [T * top]: a pair's row; None: its own
+    number), shared (float32 [T, n] or None), factor: branch = factor (sum_c weights[t, c] y[place[t top + c]] + shared).  With `out`:
     out = u / sqrt(mean(u^2) + eps) * norm of u = sum_s read[s] x_s, the streams as just written (read None: the plain sum;
     norm None: u itself); `rows` (int32, without a branch) picks the tokens that are read."""
     _need_cuda(x, branch, scale, mix, write, read, norm, out, rows)
@@ -1094,6 +1141,19 @@ def streams_step(x: torch.Tensor, streams: int, *, branch=None, scale=None, mix=
     if branch is not None:
         _need(branch.dtype == torch.float32 and branch.is_contiguous() and tuple(branch.shape) == (t, n) and rows is None,
               "streams_step: branch must be float32 [T, n], without chosen rows")
+    y = weights = place = shared = None
+    top, factor = 0, 1.0
+    if experts is not None:
+        y, weights, top, place, shared = (experts[k] for k in ("y", "weights", "top", "place", "shared"))
+        factor = experts["factor"]
+        _need_cuda(y, weights, place, shared)
+        _need(branch is None and rows is None and y.dtype == torch.float32 and y.is_contiguous() and y.shape[1] == n
+              and weights.dtype == torch.float32 and weights.is_contiguous() and weights.numel() >= t * top
+              and (place is None or (place.dtype == torch.int32 and place.is_contiguous() and place.numel() >= t * top))
+              and (place is not None or y.shape[0] >= t * top), "streams_step: the experts' rows, weights and places")
+        _need(shared is None or (shared.dtype == torch.float32 and shared.is_contiguous() and tuple(shared.shape) == (t, n)),
+              "streams_step: shared must be float32 [T, n]")
+    if branch is not None or experts is not None:
         _f32_vec(mix, streams * streams, "streams_step: mix"); _f32_vec(write, streams, "streams_step: write")
         if scale is not None:
             _f32_vec(scale, n, "streams_step: scale")
@@ -1110,7 +1170,8 @@ def streams_step(x: torch.Tensor, streams: int, *, branch=None, scale=None, mix=
         _f32_vec(read, streams, "streams_step: read")
     if norm is not None:
         _f32_vec(norm, n, "streams_step: norm")
-    _call("parallel_streams", "ri_streams_step", _p(x), _p(branch), _p(scale), _p(mix), _p(write), _p(read), _p(norm), c_float(eps),
+    _call("parallel_streams", "ri_streams_step", _p(x), _p(branch), _p(y), _p(weights), _p(place), _p(shared),
+          c_float(factor), c_int(top), _p(scale), _p(mix), _p(write), _p(read), _p(norm), c_float(eps),
           _p(rows), _p(out), c_int(dtype), c_int(n_rows), c_int(streams), c_int(n), _stream())
 
 

@@ -109,6 +109,7 @@ def time_parts(engine, s: dict, lens_before: list, new_tokens: int, peaks: dict,
     att, cache3 = blocks[3].mixer, engine.cache.layer(3)
     hd, vhd, heads, kv = s["hd"], s["vd"], s["heads"], s["kv"]
     ctx.extras["first_values"] = (torch.randn(n, att.w_qkv.n, device=dev).to(bf), att.q_dim + att.kv_dim, att.v_dim)
+    first_rows = ctx.extras["first_values"][0]
     out["attention_mixer_ms"] = round(timer(lambda: att.forward(x, residual, ctx, cache3, True)), 4)
     causal = sum(p + 1 for before in lens_before for p in range(before, before + new_tokens))
     keys = sum(before + new_tokens for before in lens_before)
@@ -118,9 +119,12 @@ def time_parts(engine, s: dict, lens_before: list, new_tokens: int, peaks: dict,
     row("attention", ms, 2.0 * (hd + vhd) * causal * heads, keys * kv * (hd + vhd) * 2 + n * heads * (hd + vhd) * 2)
     ms = timer(lambda: att.position.apply_normed_and_store(
         qkv, ctx, cache3, n_heads=heads, n_kv_heads=kv, head_dim=hd, write_kv=True, q_weight=att.q_norm, k_weight=att.k_norm, eps=1e-5,
-        v_head_dim=vhd, value_mix=(att.value_lambda, ctx.extras["first_values"][0], att.q_dim + att.kv_dim)))
+        v_head_dim=vhd, value_mix=(att.value_lambda, first_rows, att.q_dim + att.kv_dim)))
     row("norm_rotate_blend_store", ms, 0.0, n * (2 * heads * hd + 2 * kv * hd + 3 * kv * vhd) * 2)
-    row("qkv_projection", timer(lambda: linear.project(x, att.w_qkv, qkv, ctx)), 2.0 * n * att.w_qkv.n * width,
+    qkv_acc = torch.zeros(n, att.w_qkv.n, dtype=f32, device=dev)
+    project = ((lambda: linear.accumulate_split(x, att.w_qkv, qkv_acc, ctx)) if linear.wants_split(x, att.w_qkv)      # as the part calls it
+               else (lambda: linear.project(x, att.w_qkv, qkv, ctx)))
+    row("qkv_projection", timer(project), 2.0 * n * att.w_qkv.n * width,
         att.w_qkv.n * width * 2 + n * (width + att.w_qkv.n) * 2)
 
     # ---- the delta rule (layer 2) ------------------------------------------------------------------------------------------------

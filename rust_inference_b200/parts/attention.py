@@ -293,18 +293,25 @@ class GQAttention(Mixer):
             qkv = ctx.buffer("q_rot", (n, self.q_dim), self.dtype)
             from_acc(acc, self.b_qkv, qkv, ctx, cache_layer, n_heads=self.n_heads, n_kv_heads=self.n_kv_heads,
                      head_dim=self.head_dim, write_kv=writes_cache)
+        elif (special and not self.values_from_keys and not self.head_gate and not self.out_gate and writes_cache and self.own_kv
+              and linear.wants_split(x, self.w_qkv) and hasattr(self.position, "apply_normed_and_store_from_accumulators")):
+            # the same for heads that are normed, or whose values are blended
+            acc = ctx.zeroed_buffer("qkv_acc", (n, width), torch.float32)
+            linear.accumulate_split(x, self.w_qkv, acc, ctx)
+            qkv = ctx.buffer("q_rot", (n, self.q_dim), self.dtype)
+            keep = ctx.buffer("first_values", (n, self.v_dim), self.dtype) if self.value_mix == "first" else None
+            self.position.apply_normed_and_store_from_accumulators(
+                acc, self.b_qkv, qkv, ctx, cache_layer, n_heads=self.n_heads, n_kv_heads=self.n_kv_heads, head_dim=self.head_dim,
+                q_weight=self.q_norm, k_weight=self.k_norm, eps=self.qk_norm_eps if self.qk_norm_eps is not None else 0.0,
+                v_head_dim=self.v_head_dim, v_keep=keep, value_mix=self._blend(ctx, n, (keep, 0)))
         else:
             # values that later layers of the step blend in stay where they were projected: in a buffer that layers do not share
             qkv = ctx.buffer("qkv" if self.value_mix != "first" else "qkv_first_values", (n, width), self.dtype)
             linear.project(x, self.w_qkv, qkv, ctx, bias=self.b_qkv)
             extra = {} if usual else {"v_head_dim": self.v_head_dim}
-            if self.value_mix == "first":
-                ctx.extras["first_values"] = (qkv, self.q_dim + self.kv_dim, self.v_dim)
-            elif self.value_mix == "mixed":
-                first = ctx.extras.get("first_values")
-                if first is None or first[0].shape[0] != n or first[2] != self.v_dim:
-                    raise RuntimeError("blended values: no layer before this one has kept values of the same size in this step")
-                extra["value_mix"] = (self.value_lambda, first[0], first[1])
+            blend = self._blend(ctx, n, (qkv, self.q_dim + self.kv_dim))
+            if blend is not None:
+                extra["value_mix"] = blend
             if special:
                 # norm of the heads, rotation and cache write as one kernel (the position encoding's)
                 self.position.apply_normed_and_store(
@@ -317,6 +324,18 @@ class GQAttention(Mixer):
                                               n_kv_heads=self.n_kv_heads, head_dim=self.head_dim,
                                               write_kv=writes_cache and self.own_kv, **extra)
         self._attend(qkv, gate_col, residual, ctx, cache_layer)
+
+    def _blend(self, ctx, n, own):
+        """What the values are blended with, (lambda, rows, column), or None.  `own`: rows and column of the layer's own projected
+        values, which later layers of the step read if this one is the first."""
+        if self.value_mix == "first":
+            ctx.extras["first_values"] = (*own, self.v_dim)
+        if self.value_mix != "mixed":
+            return None
+        first = ctx.extras.get("first_values")
+        if first is None or first[0].shape[0] != n or first[2] != self.v_dim:
+            raise RuntimeError("blended values: no layer before this one has kept values of the same size in this step")
+        return self.value_lambda, first[0], first[1]
 
     def _attend(self, qkv, gate_col, residual, ctx, cache_layer):
         """Attention over the cache, gates and the output projection; the queries are qkv's first columns."""

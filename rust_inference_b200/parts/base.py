@@ -81,6 +81,11 @@ class FeedForward(Part):
         """residual += ff(x)."""
         raise NotImplementedError
 
+    def forward_unsummed(self, x: torch.Tensor, ctx):
+        """For arrangements whose pass over the stream can sum routed experts itself: ff(x) as the `experts` argument of
+        `ops.streams_step`, or None (nothing has run: the part has no such form, and `forward` is to be called)."""
+        return None
+
 
 class Embedding(Part):
     """Token ids -> the float32 hidden stream."""

@@ -140,8 +140,13 @@ class LatentAttention(Mixer):
         pos = self.position
         if pos.cos is None or pos.cos.shape[0] < ctx.max_len:
             raise RuntimeError("rope tables do not cover the step's positions; call prepare() first")
-        proj = ctx.buffer("latent_proj", (n, self.w_in.n), self.dtype)
-        linear.project(x, self.w_in, proj, ctx)
+        if not self.gated and linear.wants_split(x, self.w_in):
+            # a small step: the projection is split over K into float32 accumulators, which the preparing kernel reads and clears
+            proj = ctx.zeroed_buffer("latent_proj_acc", (n, self.w_in.n), torch.float32)
+            linear.accumulate_split(x, self.w_in, proj, ctx)
+        else:
+            proj = ctx.buffer("latent_proj", (n, self.w_in.n), self.dtype)
+            linear.project(x, self.w_in, proj, ctx)
 
         fast = False
         if self.dtype == torch.bfloat16:

@@ -158,6 +158,17 @@ class RotaryEncoding(PositionEncoding):
                                     write_kv=write_kv, rot_dims=self.rot_dims, v_head_dim=v_head_dim,
                                     values_from_keys=values_from_keys, value_mix=value_mix)
 
+    def apply_normed_and_store_from_accumulators(self, acc, bias, q_out, ctx, cache_layer, *, n_heads, n_kv_heads, head_dim, q_weight,
+                                                 k_weight, eps, v_head_dim=None, value_mix=None, v_keep=None):
+        """`apply_normed_and_store` from float32 accumulators of a K-split projection (bias not yet added): q goes to q_out, the
+        projected values into v_keep as well where one is given, and `acc` is left zeroed."""
+        if self.cos is None or self.cos.shape[0] < ctx.max_len:
+            raise RuntimeError("rope tables do not cover the step's positions; call prepare() first")
+        ops.rope_normed_cache_write_acc(acc, bias, q_out, self.cos, self.sin, q_weight, k_weight, eps, ctx.token_pos, ctx.token_seq,
+                                        ctx.seq_slot, ctx.page_table, cache_layer.k, cache_layer.v, n_heads=n_heads,
+                                        n_kv_heads=n_kv_heads, head_dim=head_dim, page_size=ctx.page_size, style=self.style,
+                                        rot_dims=self.rot_dims, v_head_dim=v_head_dim, value_mix=value_mix, v_keep=v_keep)
+
     def apply_and_store_from_accumulators(self, acc, bias, q_out, ctx, cache_layer, *, n_heads, n_kv_heads,
                                           head_dim, write_kv):
         """The same from float32 accumulators of a K-split projection (bias not yet added): q goes

@@ -69,6 +69,12 @@ class RoutedExperts(FeedForward):
         self.n_experts, self.top, self.expert_size = n_experts, top, expert_size
         self.n_groups, self.group_keep = n_groups, group_keep
         self.shared_size = shared_size
+        # so many slices of an expert's width a shared expert without a gate of its own consists of, where it is a whole number
+        # of them and the experts' activation is its own (0: it always runs as matrices of its own)
+        self.in_lists = 0
+        if shared_size is not None and not self.shared_gate and not self.identity and expert_form is None and shared_form is None:
+            slices = shared_size // expert_size
+            self.in_lists = slices if slices * expert_size == shared_size and slices <= self.MOST_SLICES else 0
         self.names = dict(self._NAMES, **(names or {}))
         self.router = self.correction = self.w_gate = self.w_up = self.w_down = None
         self.shared = self.shared_mix = None
@@ -110,11 +116,15 @@ class RoutedExperts(FeedForward):
         self.router = tensors[nm["router"]].contiguous()
         self.correction = tensors[nm["correction"]].contiguous() if self.has_correction else None
         self.router_bias = tensors[nm["router_bias"]].contiguous() if self.has_router_bias else None
-        self.w_gate = torch.stack([tensors[nm["gate"].format(e=e)] for e in range(n)]).contiguous()
-        self.w_up = torch.stack([tensors[nm["up"].format(e=e)] for e in range(n)]).contiguous()
-        self.w_down = torch.stack([tensors[nm["down"].format(e=e)] for e in range(n)]).contiguous()
+        # an ungated shared expert that is a whole number of experts wide stands behind the experts as that many slices
+        slices = lambda key: (tensors[nm["shared_" + key]].chunk(self.in_lists, dim=1 if key == "down" else 0) if self.in_lists else ())
+        stack = lambda key: torch.stack([tensors[nm[key].format(e=e)] for e in range(n)] + list(slices(key))).contiguous()
+        self.w_gate, self.w_up, self.w_down = stack("gate"), stack("up"), stack("down")
         if self.shared_size is not None:
-            self.shared = tuple(linear.Weight(tensors[nm[k]]) for k in ("shared_gate", "shared_up", "shared_down"))
+            # (its gate and up rows are those slices' storage; its down matrix lies the other way round and is kept twice)
+            whole = lambda w, key: w[n:].view(self.shared_size, -1) if self.in_lists else tensors[nm["shared_" + key]]
+            self.shared = (linear.Weight(whole(self.w_gate, "gate")), linear.Weight(whole(self.w_up, "up")),
+                           linear.Weight(tensors[nm["shared_down"]]))
             if self.shared_gate:
                 self.shared_mix = tensors[nm["shared_mix"]].reshape(-1).contiguous()
 
@@ -139,6 +149,7 @@ class RoutedExperts(FeedForward):
     # expert, their weights streamed by TMA) when the sizes allow; the FFMA form is the 32-bit path and
     # the fallback for other sizes
     TENSOR_CORE_MIN_TOKENS = 0
+    SHARED_IN_LISTS_TOKENS, MOST_SLICES = 64, 8     # steps of up to so many tokens; slices of a shared expert
     GATHER_IN_ARRANGE_PAIRS = 256       # up to so many (token, choice) pairs the arranging block also gathers their rows
     ROUTE_SPLIT_TOKENS, ROUTE_SPLIT_BLOCKS, ROUTE_SPLIT_MOST = 64, 148, 16     # steps of up to 64 tokens: the router's rows
     #                                     over up to 16 blocks per token, about one block per SM in all
@@ -163,13 +174,31 @@ class RoutedExperts(FeedForward):
                     split_count=ctx.zeroed_buffer("moe_route_count", (n,), torch.int32))
 
     def forward(self, x, residual, ctx):
-        n, h, top, experts = x.shape[0], self.hidden_size, self.top, self.n_experts
+        r = self._run(x, ctx)
+        # ids at or beyond the experts with tensors were left out of the lists: their rows are the input itself
+        through = dict(ids=r["ids"], x=x, n_real=self.n_experts) if self.identity else {}
+        ops.moe_combine(residual, r["y"], r["weights"], top=r["top"], shared_y=r["shared"], gate=r["gate"], place=r["place"],
+                        scale=self.out_scale, **through)
+
+    def forward_unsummed(self, x, ctx):
+        if self.identity or self.shared_mix is not None or self.top + self.in_lists > ops.MAX_SUMMED_EXPERTS:
+            return None
+        r = self._run(x, ctx)
+        return {**{k: r[k] for k in ("y", "weights", "top", "place", "shared")}, "factor": self.out_scale}
+
+    def _run(self, x, ctx) -> dict:
+        """Everything up to the sum: the experts' rows y, a token's weights and the places of its rows, the shared expert's result."""
+        n, h, experts = x.shape[0], self.hidden_size, self.n_experts
+        # a step of few tokens lists the shared expert's slices as experts that every token uses
+        extra = self.in_lists if n <= self.SHARED_IN_LISTS_TOKENS and self._on_tensor_cores(x) else 0
+        chosen, top = self.top, self.top + extra
+        listed = experts + extra
         pairs = n * top
         ids = ctx.buffer("moe_ids", (n, top), torch.int32)
         weights = ctx.buffer("moe_weights", (n, top), torch.float32)
         gate = ctx.buffer("moe_shared_gate", (n,), torch.float32) if self.shared_mix is not None else None
         cut = self.route_cut(n, ctx)
-        ops.moe_route(x, self.router, self.correction, ids, weights, top=top, groups=self.n_groups,
+        ops.moe_route(x, self.router, self.correction, ids, weights, top=chosen, always=extra, groups=self.n_groups,
                       keep=self.group_keep, gate_weight=self.shared_mix, gate_out=gate,
                       softmax=self.router_kind == "softmax", normalise=self.normalise, group_max=self.group_max, bias=self.router_bias, **cut)
         fast = self._on_tensor_cores(x)
@@ -178,38 +207,36 @@ class RoutedExperts(FeedForward):
             rows = tcgen05.GROUPED_TILE_ROWS
         else:
             rows = ops.moe_tile_rows()
-        offsets = ctx.buffer("moe_offsets", (experts + 1,), torch.int32)
+        offsets = ctx.buffer("moe_offsets", (listed + 1,), torch.int32)
         order = ctx.buffer("moe_order", (pairs,), torch.int32)
-        tiles = ctx.buffer("moe_tiles", (2 * (-(-pairs // rows) + experts),), torch.int32)
+        tiles = ctx.buffer("moe_tiles", (2 * (-(-pairs // rows) + listed),), torch.int32)
         n_tiles = ctx.buffer("moe_n_tiles", (1,), torch.int32)
         place = ctx.buffer("moe_place", (pairs,), torch.int32) if fast else None
         # an expert's rows consecutive: the activations are gathered into the lists' order (by the arranging
         # kernel itself when the pairs are few); act and y stay in that order
         xs = ctx.buffer("moe_x_sorted", (pairs, h), self.dtype) if fast else None
         small = fast and pairs <= self.GATHER_IN_ARRANGE_PAIRS
-        ops.moe_arrange(ids, pairs, experts, rows, offsets, order, tiles, n_tiles, place,
+        ops.moe_arrange(ids, pairs, listed, rows, offsets, order, tiles, n_tiles, place,
                         gather=(x, xs, top) if small else None)
         act = ctx.buffer("moe_act", (pairs, self.expert_size), self.dtype)
         y = ctx.buffer("moe_y", (pairs, h), torch.float32)
+        w_gate, w_up, w_down = (w[:listed] for w in (self.w_gate, self.w_up, self.w_down))
         if fast:
             if not small:
                 ops.moe_gather(x, xs, order, n_pairs=pairs, top=top,
-                               listed=offsets[experts:experts + 1] if self.identity else None)
-            tcgen05.grouped_gemm(xs, self.w_gate, self.w_up, act, offsets, tiles, n_tiles, n_pairs=pairs,
+                               listed=offsets[listed:listed + 1] if self.identity else None)
+            tcgen05.grouped_gemm(xs, w_gate, w_up, act, offsets, tiles, n_tiles, n_pairs=pairs,
                                  gate_form=self.expert_form)
-            tcgen05.grouped_gemm(act, self.w_down, None, y, offsets, tiles, n_tiles, n_pairs=pairs)
+            tcgen05.grouped_gemm(act, w_down, None, y, offsets, tiles, n_tiles, n_pairs=pairs)
         else:
-            ops.moe_grouped_simt(x, self.w_gate, self.w_up, act, offsets, order, tiles, n_tiles, n_pairs=pairs, top=top,
+            ops.moe_grouped_simt(x, w_gate, w_up, act, offsets, order, tiles, n_tiles, n_pairs=pairs, top=top,
                                  gate_form=self.expert_form)
-            ops.moe_grouped_simt(act, self.w_down, None, y, offsets, order, tiles, n_tiles, n_pairs=pairs, top=top)
+            ops.moe_grouped_simt(act, w_down, None, y, offsets, order, tiles, n_tiles, n_pairs=pairs, top=top)
         shared_y = None
-        if self.shared is not None:
+        if self.shared is not None and not extra:
             w_gate, w_up, w_down = self.shared
             sact = ctx.buffer("moe_shared_act", (n, self.shared_size), self.dtype)
             linear.gated(x, w_gate, w_up, sact, ctx, form=self.shared_form)
             shared_y = ctx.buffer("moe_shared_y", (n, h), torch.float32)
             linear.logits(sact, w_down, shared_y, ctx)
-        # ids at or beyond the experts with tensors were left out of the lists: their rows are the input itself
-        through = dict(ids=ids, x=x, n_real=experts) if self.identity else {}
-        ops.moe_combine(residual, y, weights, top=top, shared_y=shared_y, gate=gate, place=place, scale=self.out_scale,
-                        **through)
+        return dict(y=y, weights=weights, top=top, place=place, shared=shared_y, gate=gate, ids=ids)

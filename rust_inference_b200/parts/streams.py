@@ -62,14 +62,14 @@ class LayerScale(Part):
 
 
 class PendingWrite:
-    """A sublayer's result that has not reached the streams yet (`branch`, an accumulator, with its link and scale): the next
-    sublayer's pass over the streams takes it along, or `apply` writes it."""
+    """A sublayer's result that has not reached the streams yet (`result`: an accumulator as `branch`, or `experts`' rows; with
+    its link and scale): the next sublayer's pass over the streams takes it along, or `apply` writes it."""
 
-    def __init__(self, branch, link, scale):
-        self.branch, self.link, self.scale = branch, link, scale
+    def __init__(self, result: dict, link, scale):
+        self.result, self.link, self.scale = result, link, scale
 
     def kwargs(self) -> dict:
-        return dict(branch=self.branch, scale=None if self.scale is None else self.scale.weight, mix=self.link.mix,
+        return dict(self.result, scale=None if self.scale is None else self.scale.weight, mix=self.link.mix,
                     write=self.link.write_scaled)
 
     def apply(self, stream) -> None:
@@ -84,7 +84,7 @@ class ParallelStreams(Arrangement):
 
     The stream tensor is [T, streams * hidden], a token's streams side by side.  A sublayer adds into a zeroed float32
     buffer; writing that into the streams, reading them for the next sublayer and the norm are one pass
-    (`ops.streams_step`), also across layers: what the layer's last sublayer leaves is taken along by the next layer, or
+    (`ops.streams_step`), also across layers; routed experts' rows are summed in that pass: what the layer's last sublayer leaves is taken along by the next layer, or
     written by the model where something else looks at the streams (`ctx.settle`)."""
 
     ROLES = {"mixer": "mixer", "feed_forward": "feed_forward", "mixer_norm": "norm", "feed_forward_norm": "norm",
@@ -118,9 +118,11 @@ class ParallelStreams(Arrangement):
         branch = ctx.zeroed_buffer("branch", shape, torch.float32)
         self._enter(residual, ctx.take_pending(), self.mixer_link, self.mixer_norm, normed, ctx)
         self.mixer.forward(normed, branch, ctx, cache_layer, writes_cache)
-        pending = PendingWrite(branch, self.mixer_link, self.mixer_scale)
+        pending = PendingWrite({"branch": branch}, self.mixer_link, self.mixer_scale)
         if self.feed_forward is not None:
             self._enter(residual, pending, self.feed_forward_link, self.feed_forward_norm, normed, ctx)
-            self.feed_forward.forward(normed, branch, ctx)
-            pending = PendingWrite(branch, self.feed_forward_link, self.feed_forward_scale)
+            experts = self.feed_forward.forward_unsummed(normed, ctx)
+            if experts is None:
+                self.feed_forward.forward(normed, branch, ctx)
+            pending = PendingWrite({"branch": branch} if experts is None else {"experts": experts}, self.feed_forward_link, self.feed_forward_scale)
         ctx.leave_pending(pending)

@@ -121,6 +121,29 @@ def test_streams_step_refuses():
         ops.streams_step(x, 2)
 
 
+@pytest.mark.parametrize("streams,width,top,n", [(2, 96, 1, 5), (3, 130, 4, 9), (2, 512, 6, 400), (4, 4096, 3, 7), (1, 64, 12, 300), (6, 72, 2, 3)])
+def test_streams_step_sums_experts_rows(streams, width, top, n):
+    """What routed experts leave (rows in the order of their lists, weights, a shared result, a factor) summed in the pass that
+    writes the streams; rows in the pairs' own order; without a shared result."""
+    from rust_inference_b200.kernels import ops
+    g = torch.Generator().manual_seed(streams * width)
+    mix, write, read = torch.randn(streams, streams, generator=g), torch.randn(streams, generator=g), torch.randn(streams, generator=g)
+    scale, norm = 1 + 0.3 * torch.randn(width, generator=g), 1 + 0.3 * torch.randn(width, generator=g)
+    x, y = torch.randn(n, streams, width, generator=g), torch.randn(n * top, width, generator=g)
+    weights, shared = torch.rand(n, top, generator=g), torch.randn(n, width, generator=g)
+    order = torch.randperm(n * top, generator=g)
+    for place, with_shared, factor in ((order, True, 0.7), (None, True, 1.0), (order, False, 1.0)):
+        rows = (y[place] if place is not None else y).view(n, top, width).double()
+        total = factor * ((weights.double()[:, :, None] * rows).sum(1) + (shared.double() if with_shared else 0.0))
+        new = pp.write_streams(x.double().transpose(0, 1), mix.double(), write.double(), total * scale.double(), 1.0)
+        dx, out = d(x.reshape(n, -1)).clone(), torch.empty(n, width, device=DEV)
+        ops.streams_step(dx, streams, experts=dict(y=d(y), weights=d(weights), top=top, place=None if place is None else d(place.int()),
+                                                   shared=d(shared) if with_shared else None, factor=factor),
+                         scale=d(scale), mix=d(mix), write=d(write), read=d(read), norm=d(norm), eps=1e-5, out=out)
+        assert rel_err(dx, new.transpose(0, 1).reshape(n, -1)) < 3e-5
+        assert rel_err(out, pp.rms_norm(pp.read_streams(new, read.double()), norm.double(), 1e-5)) < 3e-5
+
+
 @pytest.mark.parametrize("dtype", [F32, BF16])
 @pytest.mark.parametrize("width,copies", [(72, 3), (30, 2), (512, 4)])
 def test_embedding_into_several_streams(dtype, width, copies):
@@ -349,6 +372,33 @@ def test_latent_attention_in_runs_of_keys(rank, rot_dim, heads, size):
             assert rel_err(out.float().reshape(-1, rank), want.float().reshape(-1, rank)) < 3e-2, (starts, splits)
 
 
+@pytest.mark.parametrize("kind", ["latent", "attention"])
+def test_projections_split_over_k(kind):
+    """A width whose small steps cut the projection over K into float32 accumulators: single tokens and portions that go that way
+    against whole prompts that do not, and the accumulators zeroed again."""
+    from rust_inference_b200.kernels import linear
+    width, n = 1536, 300
+    if kind == "latent":
+        layers = [gm.layer("latent", gm.latent(heads=4, dim=32, rot_dim=16, vdim=24, rank=64, scale=0.15, size=50))]
+    else:
+        layers = [gm.layer("attention", gm.attention(heads=4, kv=2, dim=64, vdim=32, scale=0.125, dims=32, scaling=(4.0, 1.0, 4.0, 50.0), mix=True)),
+                  gm.layer("attention", gm.attention(heads=2, kv=2, dim=24, vdim=32, scale=0.2, dims=24, mix=True))]
+    made, W = _parts(layers, BF16, width, 6)
+    parts = [p[0] for p in made]
+    x = [torch.randn(n, width, generator=torch.Generator().manual_seed(3 + i)).to(BF16) for i in range(len(parts))]
+    for part in parts:
+        w = part.w_in if kind == "latent" else part.w_qkv
+        assert linear.wants_split(d(x[0][:1]), w) and not linear.wants_split(d(x[0]), w)
+    caches, ws, shared = [_cache(p, BF16) for p in parts], _workspace(), {}
+    want = [pp.latent_attention(t.double(), W, f"l{i}.mix.", L["mixer"], 1e-5) if kind == "latent"
+            else pp.attention(t.double(), W, f"l{i}.mix.", L["mixer"], 1e-5, shared) for i, (t, L) in enumerate(zip(x, layers))]
+    for portions in ([n], [270, 1], [1, 2, 200, 30, 1], [64, 2]):
+        for got, w in zip(_both(parts, caches, x, portions, BF16, ws), want):
+            assert rel_err(got, w) < PART_TOL[BF16], portions
+    acc = ws.get_zeroed("latent_proj_acc" if kind == "latent" else "qkv_acc", (256, 512), F32)
+    assert float(acc.abs().max()) == 0.0
+
+
 @pytest.mark.parametrize("dtype", [F32, BF16])
 @pytest.mark.parametrize("heads,kv,dim,vdim,conv", [(4, 2, 16, 24, 3), (1, 1, 40, 72, 1), (6, 3, 64, 64, 4), (2, 1, 128, 64, 2), (3, 3, 9, 7, 5)])
 def test_delta_rule_alone(dtype, heads, kv, dim, vdim, conv):
@@ -385,14 +435,20 @@ def test_a_state_remembers_a_far_token():
 
 
 @pytest.mark.parametrize("dtype", [F32, BF16])
-@pytest.mark.parametrize("experts,top,ff,shared", [(6, 3, 24, 40), (8, 2, 64, 96), (12, 5, 40, 8), (1, 1, 16, 24), (4, 4, 20, None), (9, 1, 96, 96)])
+@pytest.mark.parametrize("experts,top,ff,shared", [(6, 3, 24, 40), (8, 2, 64, 96), (12, 5, 40, 8), (1, 1, 16, 24), (4, 4, 20, None), (9, 1, 96, 96), (8, 3, 32, 96),
+                                                    (5, 2, 16, 128), (3, 2, 8, 80)])
 def test_experts_as_a_part(dtype, experts, top, ff, shared):
-    """The mixture against the plain one for 1, 7, 300 and 1,100 tokens, routed freely (both get the same rounded input)."""
+    """The mixture against the plain one for 1, 7, 64, 65, 300 and 1,100 tokens, routed freely (both get the same rounded input): a
+    shared expert as matrices of its own and, in small steps where it is a whole number of experts wide, as slices in the
+    experts' lists; the tensors come back as they were."""
     width = 128
     mlp = gm.moe(experts=experts, top=top, ff=ff, shared=shared)
     parts, W = _parts([gm.layer("delta", gm.delta(heads=1, kv=1, dim=8, vdim=8, conv=1), mlp)], dtype, width, experts + top)
     part, ws = parts[0][1], _workspace()
-    for n in (1, 7, 300, 1100):
+    assert part.in_lists == (shared // ff if shared and shared % ff == 0 and shared // ff <= part.MOST_SLICES else 0)
+    for name, t in part.get_tensors().items():
+        assert torch.equal(t.double().cpu().reshape(W["l0.mlp." + name].shape), W["l0.mlp." + name]), name
+    for n in (1, 7, 64, 65, 300, 1100):
         x = torch.randn(n, width, generator=torch.Generator().manual_seed(n)).to(dtype)
         got = torch.zeros(n, width, device=DEV)
         part.forward(d(x), got, _Scratch(ws, dtype))
