@@ -74,12 +74,14 @@ template <> __device__ __forceinline__ void load4_f32<__nv_bfloat16>(const __nv_
 // tokens read them: every block leaves its rows' sums in `split_sums` ([tokens, experts + 1], float32) and takes a ticket
 // from the token's counter in `split_count` (int32, zero before and after the kernel); the block that draws the last
 // ticket reads all sums back and makes the token's choice.
+// `given` (float32 [tokens, terms * given_rows]): the rows' sums come from a product of its own (router rows, then the
+// gate's, as the sum of so many terms), and only the choice is made here.
 template <typename T, bool VEC, int TOK>
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
 moe_route_kernel(const T* x, const float* __restrict__ router, const float* __restrict__ correction, const float* __restrict__ bias,
                  const float* __restrict__ gate_w, int* __restrict__ ids, float* __restrict__ weights,
                  float* __restrict__ gate_out, int n_tokens, int width, int experts, int top, int groups, int keep,
-                 int per_block, int form, int always, float* split_sums, int* split_count) {
+                 int per_block, int form, int always, const float* given, int given_rows, int terms, float* split_sums, int* split_count) {
     extern __shared__ float smem[];
     __shared__ int last_ticket;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -104,7 +106,14 @@ moe_route_kernel(const T* x, const float* __restrict__ router, const float* __re
             gate_out[tok0 + k] = s;
         }
     };
-    for (int e = row_lo + warp; e < row_hi; e += ROUTE_WARPS) {
+    if (given != nullptr)
+        for (int i = threadIdx.x; i < n_here * n_rows; i += blockDim.x) {
+            const float* g = given + (size_t)(tok0 + i / n_rows) * terms * given_rows + i % n_rows;
+            float a = 0.f;
+            for (int j = terms - 1; j >= 0; --j) a += g[(size_t)j * given_rows];      // the smallest term first
+            place(i / n_rows, i % n_rows, a);
+        }
+    for (int e = row_lo + warp; given == nullptr && e < row_hi; e += ROUTE_WARPS) {
         const float* w = e < experts ? router + (size_t)e * width : gate_w;
         float acc[TOK];
 #pragma unroll
@@ -411,13 +420,15 @@ __global__ void moe_combine_kernel(float* residual, const float* y, const float*
 
 // form: bit 0 softmax scores instead of sigmoid ones, bit 1 weights not divided by their sum, bit 2 a group counts by its
 // largest score instead of the sum of its two largest.  correction and bias may be null.
+// given (or null): the rows' sums as `terms` terms side by side, float32 [n_tokens, terms * given_rows] (then router, x and
+// gate_w's values are not read).
 // always > 0: a token's ids are its top chosen ones and then experts, experts + 1, .. (so many, with weight 1): rows of ids and
 // weights hold top + always entries.
 // split > 1 (steps of up to ROUTE_SPLIT_TOKENS tokens): the router's rows are cut over that many blocks per token;
 // split_sums: float32 [n_tokens, experts + 1] scratch, split_count: int32 [n_tokens], zero before the call and after it.
 RI_API int ri_moe_route(const void* x, int dtype, const float* router, const float* correction, const float* bias, const float* gate_w,
                         int* ids, float* weights, float* gate_out, int n_tokens, int width, int experts, int top,
-                        int groups, int keep, int form, int always, int split, float* split_sums, int* split_count,
+                        int groups, int keep, int form, int always, const float* given, int given_rows, int terms, int split, float* split_sums, int* split_count,
                         cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (always < 0) return fail("moe_route: %d ids that every token has", always);
@@ -427,6 +438,8 @@ RI_API int ri_moe_route(const void* x, int dtype, const float* router, const flo
     if ((long long)keep * (experts / groups) < top)
         return fail("moe_route: %d groups of %d experts cannot give %d choices", keep, experts / groups, top);
     // few tokens: one per block, so that the router's rows are shared out over more SMs
+    if (given != nullptr && (split > 1 || terms < 1 || given_rows < experts + (gate_w != nullptr ? 1 : 0)))
+        return fail("moe_route: %d terms of the sums of %d rows", terms, given_rows);
     const int per_block = n_tokens >= 148 * ROUTE_TOKENS ? ROUTE_TOKENS : (n_tokens >= 2 * 148 ? 2 : 1);
     if (split > 1 && (per_block != 1 || split_sums == nullptr || split_count == nullptr || split > 65535))
         return fail("moe_route: rows cut over %d blocks need one token per block and their scratch", split);
@@ -438,7 +451,7 @@ RI_API int ri_moe_route(const void* x, int dtype, const float* router, const flo
     cudaError_t e;
 #define RI_ROUTE_N(T, V, N) launch_dependent(moe_route_kernel<T, V, N>, blocks, ROUTE_WARPS * 32, smem, stream, (const T*)x, \
                                              router, correction, bias, gate_w, ids, weights, gate_out, n_tokens, width, experts, top,   \
-                                             groups, keep, per_block, form, always, split_sums, split_count)
+                                             groups, keep, per_block, form, always, given, given_rows, terms, split_sums, split_count)
 #define RI_ROUTE(T, V) (per_block == 1 ? RI_ROUTE_N(T, V, 1) : per_block == 2 ? RI_ROUTE_N(T, V, 2) : RI_ROUTE_N(T, V, ROUTE_TOKENS))
     if (dtype == RI_F32) e = vec ? RI_ROUTE(float, true) : RI_ROUTE(float, false);
     else if (dtype == RI_BF16) e = vec ? RI_ROUTE(__nv_bfloat16, true) : RI_ROUTE(__nv_bfloat16, false);

@@ -189,7 +189,7 @@ def time_parts(engine, kind: str, s: dict, lens_before: list, new_tokens: int, p
                                                          n_pairs=pairs, top=top))
         out["route_ms"] = round(timer(lambda: ops.moe_route(x, ff.router, ff.correction, ids, wts, top=top, groups=s["groups"],
                                                             keep=s["keep"], gate_weight=ff.shared_mix, gate_out=gate,
-                                                            **ff.route_cut(n, ctx))), 4)
+                                                            **ff.route_cut(x, ctx))), 4)
         out["arrange_ms"] = round(timer(lambda: ops.moe_arrange(ids, pairs, experts, rows, offsets, order, tiles, n_tiles, place)), 4)
         if fast:
             out["gather_ms"] = round(timer(lambda: ops.moe_gather(x, xs, order, n_pairs=pairs, top=top)), 4)

@@ -155,7 +155,7 @@ def time_parts(engine, s: dict, lens_before: list, new_tokens: int, peaks: dict,
     ids = torch.empty(n, top, dtype=torch.int32, device=dev)
     wts = torch.empty(n, top, dtype=f32, device=dev)
     route = lambda: ops.moe_route(x, mx.router, None, ids, wts, top=top, groups=mx.n_groups, keep=mx.group_keep, softmax=True,
-                                  normalise=False, group_max=True, **mx.route_cut(n, ctx))
+                                  normalise=False, group_max=True, **mx.route_cut(x, ctx))
     row("router", timer(route), 0.0, experts * width * 4 + n * width * 2, fp32_flops=2.0 * n * experts * width)
     used = int(torch.unique(ids).numel())
     if not mx._on_tensor_cores(x):

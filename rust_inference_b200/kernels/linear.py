@@ -31,6 +31,9 @@ def _use_tensor_cores(x: torch.Tensor, w: Weight) -> bool:
     return tcgen05.supports(x, w)
 
 
+on_tensor_cores = _use_tensor_cores      # for callers that choose their path by it
+
+
 def project(x, w: Weight, out, ctx, bias=None):
     """out<run dtype> = x W^T + bias."""
     if _use_tensor_cores(x, w):

@@ -835,7 +835,7 @@ def moe_route(x: torch.Tensor, router: torch.Tensor, correction: torch.Tensor | 
               gate_weight: torch.Tensor | None = None, gate_out: torch.Tensor | None = None,
               softmax: bool = False, normalise: bool = True, split: int = 1, split_sums: torch.Tensor | None = None,
               split_count: torch.Tensor | None = None, group_max: bool = False, bias: torch.Tensor | None = None,
-              always: int = 0) -> None:
+              always: int = 0, sums: tuple | None = None) -> None:
     """Per token the `top` experts with the largest sigmoid(router x) + correction among the `keep` best of
     `groups` groups (a group's score: the sum of its two largest, or with group_max its largest alone; correction None:
     zero), ids int32 [T, top], and their weights
@@ -843,7 +843,8 @@ def moe_route(x: torch.Tensor, router: torch.Tensor, correction: torch.Tensor | 
     sigmoid(gate_weight . x_t) as well.  softmax: the scores are softmax(router x) over all experts instead of
     sigmoids; normalise False: the weights are the chosen scores as they are.  bias float32 [experts]: added to
     router x before the sigmoid or softmax.  always: so many ids from `experts` on that every token has after its chosen ones,
-    with weight 1 (ids and weights are then [T, top + always]).  split > 1 (steps of fewer than 296
+    with weight 1 (ids and weights are then [T, top + always]).  sums = (t, terms): router x, then gate_weight . x, already
+    formed, as the sum of `terms` pieces of t, float32 [T, terms * rows] side by side (rows at least experts, + 1 with a gate).  split > 1 (steps of fewer than 296
     tokens): the router's rows are cut over that many blocks per token, which leave their sums in split_sums (float32
     [T, experts + 1]) and count themselves in split_count (int32 [T], zero before the call and after it)."""
     _need_cuda(x, router, correction, ids, weights, gate_weight, gate_out, bias)
@@ -859,6 +860,11 @@ def moe_route(x: torch.Tensor, router: torch.Tensor, correction: torch.Tensor | 
     if gate_weight is not None:
         _need(gate_weight.dtype == torch.float32 and gate_weight.is_contiguous() and gate_weight.numel() == width
               and gate_out.dtype == torch.float32 and gate_out.numel() >= n, "moe_route: gate")
+    if sums is not None:
+        t, terms = sums
+        _need_cuda(t)
+        _need(split == 1 and t.dtype == torch.float32 and t.is_contiguous() and t.shape[0] == n and t.shape[1] % terms == 0
+              and t.shape[1] // terms >= experts + (0 if gate_weight is None else 1), "moe_route: sums must be float32 [T, terms * rows]")
     if split > 1:
         _need_cuda(split_sums, split_count)
         _need(n < 296 and split_sums is not None and split_sums.dtype == torch.float32 and split_sums.is_contiguous()
@@ -866,7 +872,9 @@ def moe_route(x: torch.Tensor, router: torch.Tensor, correction: torch.Tensor | 
               and split_count.numel() >= n, "moe_route: rows cut over blocks need few tokens, float32 sums and int32 counters")
     _call("moe", "ri_moe_route", _p(x), c_int(dtype_code(x.dtype)), _p(router), _p(correction), _p(bias), _p(gate_weight), _p(ids),
           _p(weights), _p(gate_out), c_int(n), c_int(width), c_int(experts), c_int(top), c_int(groups), c_int(keep),
-          c_int((1 if softmax else 0) | (0 if normalise else 2) | (4 if group_max else 0)), c_int(always), c_int(max(1, split)), _p(split_sums if split > 1 else None),
+          c_int((1 if softmax else 0) | (0 if normalise else 2) | (4 if group_max else 0)), c_int(always),
+          _p(None if sums is None else sums[0]), c_int(0 if sums is None else sums[0].shape[1] // sums[1]),
+          c_int(0 if sums is None else sums[1]), c_int(max(1, split)), _p(split_sums if split > 1 else None),
           _p(split_count if split > 1 else None), _stream())
 
 

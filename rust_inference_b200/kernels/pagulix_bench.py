@@ -66,10 +66,9 @@ def time_parts(engine, s: dict, lens_before: list, new_tokens: int, peaks: dict,
     S, link, norm, scale = s["streams"], blocks[0].feed_forward_link, blocks[0].feed_forward_norm, blocks[0].mixer_scale
     streams = torch.randn(n, S * width, device=dev)
     branch, normed = torch.zeros(n, width, device=dev), torch.empty(n, width, dtype=bf, device=dev)
-    row("streams_write_read_norm", timer(lambda: ops.streams_step(
-        streams, S, branch=branch, scale=scale.weight, mix=link.mix, write=link.write_scaled, read=link.read, norm=norm.factor, eps=norm.eps,
-        out=normed)), 0.0, n * width * (8 * S + 8 + 2) + width * 8)
-    del streams
+    border = dict(scale=scale.weight, mix=link.mix, write=link.write_scaled, read=link.read, norm=norm.factor, eps=norm.eps, out=normed)
+    row("streams_write_read_norm", timer(lambda: ops.streams_step(streams, S, branch=branch, **border)), 0.0,
+        n * width * (8 * S + 8 + 2) + width * 8)
 
     # ---- latent attention over a window (layer 0) ------------------------------------------------------------------------
     lat, cache0 = blocks[0].mixer, engine.cache.layer(0)
@@ -155,35 +154,42 @@ def time_parts(engine, s: dict, lens_before: list, new_tokens: int, peaks: dict,
     # ---- experts -------------------------------------------------------------------------------------------------------------------
     mx = blocks[0].feed_forward
     out["experts_feed_forward_ms"] = round(timer(lambda: mx.forward(x, residual, ctx)), 4)
-    top, experts, f, shared = mx.top, mx.n_experts, mx.expert_size, mx.shared_size
+    # a step of few tokens lists the shared expert's slices as experts that every token uses; else they are matrices of their own
+    extra = mx.in_lists if n <= mx.SHARED_IN_LISTS_TOKENS else 0
+    chosen, top, experts, f, shared = mx.top, mx.top + extra, mx.n_experts + extra, mx.expert_size, mx.shared_size
     pairs = n * top
     ids, wts = torch.empty(n, top, dtype=torch.int32, device=dev), torch.empty(n, top, dtype=f32, device=dev)
-    row("router", timer(lambda: ops.moe_route(x, mx.router, None, ids, wts, top=top, softmax=True, bias=mx.router_bias, **mx.route_cut(n, ctx))),
-        0.0, experts * width * 4 + n * width * 2, fp32_flops=2.0 * n * experts * width)
+    row("router", timer(lambda: ops.moe_route(x, mx.router, None, ids, wts, top=chosen, always=extra, softmax=True, bias=mx.router_bias,
+                                              **mx.route_cut(x, ctx))),
+        0.0, mx.n_experts * width * 4 + n * width * 2, fp32_flops=2.0 * n * mx.n_experts * width)
     used = int(torch.unique(ids).numel())
     if not mx._on_tensor_cores(x):
         raise RuntimeError("the benchmark's experts run on the tensor cores")
     offsets, order, tiles, n_tiles, place = i32(experts + 1), i32(pairs), i32(2 * (-(-pairs // tile_rows) + experts)), i32(1), i32(pairs)
     arrange = lambda: ops.moe_arrange(ids, pairs, experts, tile_rows, offsets, order, tiles, n_tiles, place)
     arrange()
-    y = torch.empty(pairs, width, dtype=f32, device=dev)
+    y = torch.randn(pairs, width, dtype=f32, device=dev)
     acts = torch.empty(pairs, f, dtype=bf, device=dev)
     xs = torch.zeros(pairs, width, dtype=bf, device=dev)
     gather = lambda: ops.moe_gather(x, xs, order, n_pairs=pairs, top=top)
     gather()
-    ms_up = timer(lambda: tcgen05.grouped_gemm(xs, mx.w_gate, mx.w_up, acts, offsets, tiles, n_tiles, n_pairs=pairs))
-    ms_down = timer(lambda: tcgen05.grouped_gemm(acts, mx.w_down, None, y, offsets, tiles, n_tiles, n_pairs=pairs))
+    w_gate, w_up, w_down = mx.w_gate[:experts], mx.w_up[:experts], mx.w_down[:experts]
+    ms_up = timer(lambda: tcgen05.grouped_gemm(xs, w_gate, w_up, acts, offsets, tiles, n_tiles, n_pairs=pairs))
+    ms_down = timer(lambda: tcgen05.grouped_gemm(acts, w_down, None, y, offsets, tiles, n_tiles, n_pairs=pairs))
     out["gather_ms"], out["arrange_ms"] = round(timer(gather), 4), round(timer(arrange), 4)
     row("experts_gate_up", ms_up, 2.0 * pairs * 2 * f * width, used * 2 * f * width * 2 + pairs * (width + f) * 2)
     row("experts_down", ms_down, 2.0 * pairs * f * width, used * f * width * 2 + pairs * (f * 2 + width * 4))
-    w_gate, w_up, w_down = mx.shared
-    sact, shared_y = torch.empty(n, shared, dtype=bf, device=dev), torch.empty(n, width, dtype=f32, device=dev)
-    row("shared_gate_up", timer(lambda: linear.gated(x, w_gate, w_up, sact, ctx)), 2.0 * n * 2 * shared * width,
-        2 * shared * width * 2 + n * (width + shared) * 2)
-    row("shared_down", timer(lambda: linear.logits(sact, w_down, shared_y, ctx)), 2.0 * n * shared * width,
-        shared * width * 2 + n * (shared * 2 + width * 4))
-    row("combine", timer(lambda: ops.moe_combine(residual, y, wts, top=top, shared_y=shared_y, place=place)), 0.0,
-        pairs * width * 4 + n * width * 12 + pairs * 8)
+    shared_y = None
+    if not extra:
+        w_gate, w_up, w_down = mx.shared
+        sact, shared_y = torch.empty(n, shared, dtype=bf, device=dev), torch.empty(n, width, dtype=f32, device=dev)
+        row("shared_gate_up", timer(lambda: linear.gated(x, w_gate, w_up, sact, ctx)), 2.0 * n * 2 * shared * width,
+            2 * shared * width * 2 + n * (width + shared) * 2)
+        row("shared_down", timer(lambda: linear.logits(sact, w_down, shared_y, ctx)), 2.0 * n * shared * width,
+            shared * width * 2 + n * (shared * 2 + width * 4))
+    left = dict(y=y, weights=wts, top=top, place=place, shared=shared_y, factor=1.0)
+    row("experts_sum_streams_write_read_norm", timer(lambda: ops.streams_step(streams, S, experts=left, **border)), 0.0,
+        pairs * (width * 4 + 8) + n * width * (8 * S + 2 + (0 if extra else 4)) + width * 8)
     out["experts_used"] = used
     engine.workspace.rezero()
     for slot in slots:
@@ -192,7 +198,7 @@ def time_parts(engine, s: dict, lens_before: list, new_tokens: int, peaks: dict,
 
 
 # how far each kernel of the design is from its roofline, over the like kernel of the closest model
-LIKE = {"streams_write_read_norm": ("dense", "rms_norm"), "latent_attention": ("vadodra", "latent_attention"),
+LIKE = {"streams_write_read_norm": ("dense", "rms_norm"), "experts_sum_streams_write_read_norm": ("dense", "rms_norm"), "latent_attention": ("vadodra", "latent_attention"),
         "latent_prepare": ("vadodra", "latent_prepare"), "queries_into_latent": ("vadodra", "queries_into_latent"),
         "latents_to_values": ("vadodra", "latents_to_values"), "latent_gate": ("vadodra", "latent_gate"),
         "attention": ("dense", "attention"), "norm_rotate_blend_store": ("vadodra", "norm_rotate_store"),
@@ -243,9 +249,10 @@ def main(sizes: str, peaks: dict, peak_source: str, *, prefill_tokens: int = 204
     ratios = {}
     for phase in ("prefill_parts", "decode_parts"):
         for name, (model, other) in LIKE.items():
-            ratios[f"{phase[:-6]}.{name} (over {model} {other})"] = round(
-                result["pagulix"][phase][name]["x_roofline"] / result[model][phase][other]["x_roofline"], 2)
-        for name, other in (("router", "route_ms"), ("combine", "combine_ms")):
+            if name in result["pagulix"][phase]:
+                ratios[f"{phase[:-6]}.{name} (over {model} {other})"] = round(
+                    result["pagulix"][phase][name]["x_roofline"] / result[model][phase][other]["x_roofline"], 2)
+        for name, other in (("router", "route_ms"),):
             ratios[f"{phase[:-6]}.{name} ms (over lulisun {name} ms)"] = round(
                 result["pagulix"][phase][name]["ms"] / max(result["lulisun"][phase][other], 1e-6), 2)
     result["x_roofline_over_like"] = ratios

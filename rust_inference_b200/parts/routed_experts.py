@@ -77,7 +77,7 @@ class RoutedExperts(FeedForward):
             self.in_lists = slices if slices * expert_size == shared_size and slices <= self.MOST_SLICES else 0
         self.names = dict(self._NAMES, **(names or {}))
         self.router = self.correction = self.w_gate = self.w_up = self.w_down = None
-        self.shared = self.shared_mix = None
+        self.shared = self.shared_mix = self.w_router = None
 
     @staticmethod
     def _form(form, device):
@@ -116,6 +116,8 @@ class RoutedExperts(FeedForward):
         self.router = tensors[nm["router"]].contiguous()
         self.correction = tensors[nm["correction"]].contiguous() if self.has_correction else None
         self.router_bias = tensors[nm["router_bias"]].contiguous() if self.has_router_bias else None
+        self.shared_mix = tensors[nm["shared_mix"]].reshape(-1).contiguous() if self.shared_size is not None and self.shared_gate else None
+        self.w_router, self.router_terms = self._router_matrix()
         # an ungated shared expert that is a whole number of experts wide stands behind the experts as that many slices
         slices = lambda key: (tensors[nm["shared_" + key]].chunk(self.in_lists, dim=1 if key == "down" else 0) if self.in_lists else ())
         stack = lambda key: torch.stack([tensors[nm[key].format(e=e)] for e in range(n)] + list(slices(key))).contiguous()
@@ -125,8 +127,20 @@ class RoutedExperts(FeedForward):
             whole = lambda w, key: w[n:].view(self.shared_size, -1) if self.in_lists else tensors[nm["shared_" + key]]
             self.shared = (linear.Weight(whole(self.w_gate, "gate")), linear.Weight(whole(self.w_up, "up")),
                            linear.Weight(tensors[nm["shared_down"]]))
-            if self.shared_gate:
-                self.shared_mix = tensors[nm["shared_mix"]].reshape(-1).contiguous()
+
+    def _router_matrix(self):
+        """The router's rows (and the shared expert's gate row) for bfloat16 runs as bfloat16 matrices that add up to them, one
+        below the other: a float32 number is the sum of three bfloat16 ones (8 bits of its 24 each), and one that is stored as
+        bfloat16 is the first of them alone.  Products of a bfloat16 input with bfloat16 weights are exact in float32, so a
+        tensor-core product with float32 accumulators forms the same 32-bit logits as the float32 rows would."""
+        if self.dtype != torch.bfloat16:
+            return None, 0
+        rows = self.router if self.shared_mix is None else torch.cat([self.router, self.shared_mix[None]], dim=0)
+        rest, terms = torch.cat([rows, rows.new_zeros(-len(rows) % 8, rows.shape[1])], dim=0), []
+        while len(terms) < 3 and (not terms or bool(rest.any())):
+            terms.append(rest.to(torch.bfloat16))
+            rest = rest - terms[-1].float()
+        return linear.Weight(torch.cat(terms, dim=0)), len(terms)
 
     def get_tensors(self):
         nm = self.names
@@ -151,6 +165,7 @@ class RoutedExperts(FeedForward):
     TENSOR_CORE_MIN_TOKENS = 0
     SHARED_IN_LISTS_TOKENS, MOST_SLICES = 64, 8     # steps of up to so many tokens; slices of a shared expert
     GATHER_IN_ARRANGE_PAIRS = 256       # up to so many (token, choice) pairs the arranging block also gathers their rows
+    ROUTE_PRODUCT_TOKENS = 256          # steps of at least so many tokens: the router's logits as a product
     ROUTE_SPLIT_TOKENS, ROUTE_SPLIT_BLOCKS, ROUTE_SPLIT_MOST = 64, 148, 16     # steps of up to 64 tokens: the router's rows
     #                                     over up to 16 blocks per token, about one block per SM in all
 
@@ -161,9 +176,15 @@ class RoutedExperts(FeedForward):
         return (tcgen05.grouped_supports(x.dtype, self.w_gate) and tcgen05.grouped_supports(x.dtype, self.w_down)
                 and self.hidden_size % 8 == 0)
 
-    def route_cut(self, n: int, ctx) -> dict:
-        """Keyword arguments of `ops.moe_route` for a step of n tokens: a step of few tokens cuts the router's rows over
-        several blocks per token, so that more SMs than tokens read them (scratch from the step's workspace)."""
+    def route_cut(self, x, ctx) -> dict:
+        """Keyword arguments of `ops.moe_route` for the step's input x: a step of few tokens cuts the router's rows over several
+        blocks per token, so that more SMs than tokens read them; one of many forms the logits as a product on the
+        tensor cores (scratch from the step's workspace)."""
+        n = x.shape[0]
+        if n >= self.ROUTE_PRODUCT_TOKENS and self.w_router is not None and linear.on_tensor_cores(x, self.w_router):
+            sums = ctx.buffer("moe_route_logits", (n, self.w_router.n), torch.float32)
+            linear.logits(x, self.w_router, sums, ctx)
+            return dict(sums=(sums, self.router_terms))
         outputs = self.router.shape[0] + (1 if self.shared_mix is not None else 0)
         if n > self.ROUTE_SPLIT_TOKENS:
             return {}
@@ -197,7 +218,7 @@ class RoutedExperts(FeedForward):
         ids = ctx.buffer("moe_ids", (n, top), torch.int32)
         weights = ctx.buffer("moe_weights", (n, top), torch.float32)
         gate = ctx.buffer("moe_shared_gate", (n,), torch.float32) if self.shared_mix is not None else None
-        cut = self.route_cut(n, ctx)
+        cut = self.route_cut(x, ctx)
         ops.moe_route(x, self.router, self.correction, ids, weights, top=chosen, always=extra, groups=self.n_groups,
                       keep=self.group_keep, gate_weight=self.shared_mix, gate_out=gate,
                       softmax=self.router_kind == "softmax", normalise=self.normalise, group_max=self.group_max, bias=self.router_bias, **cut)

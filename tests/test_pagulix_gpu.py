@@ -179,6 +179,36 @@ def test_router_with_a_bias():
             assert torch.allclose(got_w.cpu().double(), s.gather(1, got_ids.cpu().long()), rtol=2e-5, atol=1e-7)
 
 
+@pytest.mark.parametrize("gated,stored", [(False, BF16), (True, BF16), (False, F32), (True, F32)])
+def test_router_logits_as_a_product(gated, stored):
+    """A long bfloat16 step forms the router's logits on the tensor cores, from as many bfloat16 matrices as its rows need (one
+    where they are stored as bfloat16, three for float32 numbers): the same choices and weights as the float32 rows give, and
+    the shared expert's gate with them.  Logits differ by float32 rounding only."""
+    from rust_inference_b200.kernels import ops
+    from rust_inference_b200.parts.registry import lookup
+    width, n, experts, top = 200, 700, 11, 4
+    g = torch.Generator().manual_seed(5)
+    part = lookup("feed_forward", "routed_experts")(n_experts=experts, top=top, expert_size=16, shared_size=24, shared_gate=gated,
+                                                    router_kind="softmax", router_bias=True, correction=False, hidden_size=width,
+                                                    dtype=BF16, device=DEV)
+    T = {k: (torch.randn(ts.shape, generator=g) / (math.sqrt(ts.shape[-1]) if len(ts.shape) > 1 else 1.0)) for k, ts in part.tensor_specs().items()}
+    part.set_tensors({k: d(v.to(stored).float() if part.tensor_specs()[k].role == "vector" else v.to(BF16)) for k, v in T.items()})
+    assert part.router_terms == (1 if stored == BF16 else 3)
+    x = torch.randn(n, width, generator=g).to(BF16)
+    ctx = _Scratch(_workspace(), BF16)
+    cut = part.route_cut(d(x), ctx)
+    z = x.double() @ part.router.double().cpu().T
+    assert rel_err(cut["sums"][0].view(n, part.router_terms, -1)[:, :, :experts].sum(1), z) < 3e-6
+    ids, weights = pp.route(x.double(), part.router.double().cpu(), part.router_bias.double().cpu(), top)
+    got_ids, got_w, gate = torch.empty(n, top, dtype=torch.int32, device=DEV), torch.empty(n, top, device=DEV), torch.empty(n, device=DEV)
+    ops.moe_route(d(x), part.router, None, got_ids, got_w, top=top, softmax=True, bias=part.router_bias, gate_weight=part.shared_mix,
+                  gate_out=gate if gated else None, **cut)
+    assert torch.equal(got_ids.cpu().long(), ids)
+    assert torch.allclose(got_w.cpu().double(), weights, rtol=2e-5, atol=1e-7)
+    if gated:
+        assert torch.allclose(gate.cpu().double(), torch.sigmoid(x.double() @ part.shared_mix.double().cpu()), rtol=1e-5)
+
+
 # ---------------------------------------------------------------------------------------------------
 # parts alone, outside an engine
 # ---------------------------------------------------------------------------------------------------
