@@ -197,12 +197,27 @@ def time_parts(engine, s: dict, lens_before: list, new_tokens: int, peaks: dict,
     return out
 
 
+def dense_qkv(engine, s: dict, lens_before: list, new_tokens: int, peaks: dict, timer: Timer) -> dict:
+    """The dense decoder's q, k, v projection alone, as its mixer calls it."""
+    from . import linear
+    slots, ctx = _step_context(engine, lens_before, new_tokens, s["vocab"], 5)
+    n, w, dev = ctx.n_tokens, engine.model.layers[0].block.mixer.w_qkv, engine.device
+    x = (torch.randn(n, w.k, device=dev) * 0.5).to(torch.bfloat16)
+    split = linear.wants_split(x, w)
+    out = torch.zeros(n, w.n, dtype=torch.float32 if split else torch.bfloat16, device=dev)
+    ms = timer((lambda: linear.accumulate_split(x, w, out, ctx)) if split else (lambda: linear.project(x, w, out, ctx)))
+    ideal = _roofline_ms(2.0 * n * w.n * w.k, w.n * w.k * 2 + n * (w.k * 2 + w.n * out.element_size()), peaks)
+    for slot in slots:
+        engine.free_slot(slot)
+    return {"qkv_projection": {"ms": round(ms, 4), "roofline_ms": round(ideal, 6), "x_roofline": round(ms / ideal, 2)}}
+
+
 # how far each kernel of the design is from its roofline, over the like kernel of the closest model
 LIKE = {"streams_write_read_norm": ("dense", "rms_norm"), "experts_sum_streams_write_read_norm": ("dense", "rms_norm"), "latent_attention": ("vadodra", "latent_attention"),
         "latent_prepare": ("vadodra", "latent_prepare"), "queries_into_latent": ("vadodra", "queries_into_latent"),
         "latents_to_values": ("vadodra", "latents_to_values"), "latent_gate": ("vadodra", "latent_gate"),
         "attention": ("dense", "attention"), "norm_rotate_blend_store": ("vadodra", "norm_rotate_store"),
-        "qkv_projection": ("dense", "down"), "delta_projection": ("dense", "down"),
+        "qkv_projection": ("dense", "qkv_projection"), "delta_projection": ("dense", "down"),
         "delta_prepare": ("redodra", "delta_rule_prepare"), "delta_scan": ("redodra", "delta_rule_scan"),
         "delta_gated_norm": ("redodra", "delta_rule_gated_norm"), "experts_gate_up": ("lulisun", "experts_gate_up"),
         "experts_down": ("lulisun", "experts_down"), "shared_gate_up": ("dense", "gate_up"), "shared_down": ("dense", "down")}
@@ -242,6 +257,7 @@ def main(sizes: str, peaks: dict, peak_source: str, *, prefill_tokens: int = 204
             else:
                 r[phase] = arch_bench.time_parts(engine, "dense", s, before, new, peaks, timer)
                 r[phase].update(dense_norm_and_rope(engine, s, before, new, peaks, timer))
+                r[phase].update(dense_qkv(engine, s, before, new, peaks, timer))
         engine.check_device_status()
         result[kind] = r
         del engine

@@ -213,7 +213,7 @@ def test_router_logits_as_a_product(gated, stored):
 # parts alone, outside an engine
 # ---------------------------------------------------------------------------------------------------
 # heads, kv heads, dim, vdim, rotated channels
-ATTENTION_SIZES = [(4, 2, 16, 24, 8), (1, 1, 24, 24, 24), (5, 1, 12, 20, 4), (3, 3, 40, 9, 40), (4, 2, 64, 32, 32), (4, 1, 128, 64, 128), (8, 2, 128, 32, 64),
+ATTENTION_SIZES = [(4, 2, 16, 24, 8), (1, 1, 24, 24, 24), (5, 1, 12, 20, 4), (3, 3, 40, 9, 40), (4, 2, 64, 32, 32), (4, 1, 128, 64, 128), (6, 2, 128, 32, 96),
                    (4, 4, 64, 128, 16), (2, 1, 64, 64, 64), (6, 2, 128, 128, 48), (34, 2, 64, 32, 64), (2, 2, 96, 64, 96)]
 
 
@@ -308,7 +308,7 @@ def test_values_blended_with_the_first_layer_s(dtype, heads, kv, dim, vdim):
 
 # heads, dim, rotated part, vdim, rank, window
 LATENT_SIZES = [(3, 12, 8, 20, 40, 20), (1, 24, 24, 24, 24, 1), (4, 32, 64, 64, 64, 70), (8, 64, 32, 32, 256, 129), (2, 16, 32, 16, 128, 64),
-                (5, 9, 2, 7, 33, 65), (16, 32, 64, 32, 512, 40), (6, 32, 32, 32, 128, 33), (4, 40, 64, 24, 64, 200), (2, 128, 64, 128, 512, 100)]
+                (5, 9, 2, 7, 33, 65), (16, 32, 64, 32, 512, 40), (5, 48, 32, 40, 128, 33), (4, 40, 64, 24, 64, 200), (2, 128, 64, 128, 512, 100)]
 
 
 @pytest.mark.parametrize("dtype", [F32, BF16])
@@ -430,7 +430,7 @@ def test_projections_split_over_k(kind):
 
 
 @pytest.mark.parametrize("dtype", [F32, BF16])
-@pytest.mark.parametrize("heads,kv,dim,vdim,conv", [(4, 2, 16, 24, 3), (1, 1, 40, 72, 1), (6, 3, 64, 64, 4), (2, 1, 128, 64, 2), (3, 3, 9, 7, 5)])
+@pytest.mark.parametrize("heads,kv,dim,vdim,conv", [(4, 2, 16, 24, 3), (1, 1, 40, 72, 1), (8, 4, 64, 48, 3), (2, 1, 128, 64, 2), (3, 3, 9, 7, 5)])
 def test_delta_rule_alone(dtype, heads, kv, dim, vdim, conv):
     """With one decay per head and a silu gate: whole, in portions, token by token, in a slot another sequence has used."""
     width, n = 96, 150
@@ -737,10 +737,10 @@ def test_the_command_line_on_a_pagulix_folder(models):
 
 
 @pytest.mark.parametrize("kind,m", [("attention", gm.attention(heads=4, kv=2, dim=64, vdim=32, scale=0.125, dims=64)),
-                                    ("attention", gm.attention(heads=4, kv=2, dim=128, vdim=32, scale=0.08, dims=64)),
+                                    ("attention", gm.attention(heads=6, kv=2, dim=128, vdim=32, scale=0.08, dims=96)),
                                     ("attention", gm.attention(heads=4, kv=1, dim=128, vdim=64, scale=0.08, dims=64)),
                                     ("attention", gm.attention(heads=2, kv=2, dim=64, vdim=128, scale=0.125, dims=64)),
-                                    ("latent", gm.latent(heads=6, dim=32, rot_dim=32, vdim=32, rank=128, scale=0.125, size=100))])
+                                    ("latent", gm.latent(heads=5, dim=48, rot_dim=32, vdim=40, rank=128, scale=0.11, size=100))])
 def test_tensor_core_kernels_take_the_forms(kind, m, monkeypatch):
     """bfloat16 runs of these sizes never reach the generic kernel: prompts, portions and single tokens, whose pages are cut into
     one run, several by a second kernel and several as a cluster."""
